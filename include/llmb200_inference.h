@@ -108,7 +108,7 @@ int llmb200_state_connect(InferenceState *state, const void *all_handles, int wo
 
 /* Layer-by-layer construction (same conversions as inference_state_create). */
 typedef struct {
-    int model_type;                 /* MODEL_QWEN3 / MODEL_GEMMA3 */
+    int model_type;                 /* MODEL_QWEN3 / MODEL_GEMMA3 (others: inference_state_create_from_dir) */
     int d_model, n_q_heads, n_kv_heads, head_dim, intermediate_size, vocab_size, n_layers;
     int max_seq_len, use_fp16;
 } llmb200_config;
@@ -164,6 +164,19 @@ int llmb200_state_graph_kernels(InferenceState *state, int with_lm_head);
  * (interleaved rows g0,u0,g1,u1,...), 3 down, 4 LM head (layer ignored).
  * Returns the byte count, or 0 on error; buf may be NULL to query the size. */
 size_t llmb200_state_export_weight(InferenceState *state, int layer, int which, void *buf, size_t cap);
+
+/* A state for the model in a folder that holds config.json and model.safetensors; the model type is
+ * config.json's "architecture" (Morilorn). wtype: B200_WT_BF16 (bfloat16 matrices and products with fp32
+ * accumulation; norms, scores, softmax, gates and the residual stream in fp32) or B200_WT_F32 (everything in
+ * fp32). max_seq_len positions of cache, not clamped. NULL with a message on stderr on any failure. No
+ * counterpart in the reference, whose loaders fill the structures that inference_state_create takes. */
+InferenceState *inference_state_create_from_dir(const char *dir, int max_seq_len, int wtype);
+/* Feeds n tokens at the current position and advances it by n; logits of the places want[0..n_want), ascending
+ * indexes among the n tokens, are written to logits [n_want][vocab]. Works on every state: model types with a
+ * row path run a portion of several tokens in one pass over the weights, the others token by token. Returns 0,
+ * or a negative code with the position unchanged or, after a device error, undefined. */
+int inference_forward_tokens(InferenceState *state, const uint32_t *tokens, int n, const int *want, int n_want,
+                             float *logits);
 
 /* Batched decode state, built layer by layer (cfg->use_fp16 is ignored: weights
  * are binary16; cfg->max_seq_len is clamped to 4096). Sequences may have

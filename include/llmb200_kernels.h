@@ -15,6 +15,8 @@
  *   Q8_0  row r = cols int8 quants, then cols/32 binary16 scales; rows are
  *         row_stride bytes apart, row_stride = round_up(34*cols/32, 16).
  *   F16   row r = cols binary16 values; row_stride = round_up(2*cols, 16).
+ *   BF16  row r = cols bfloat16 values; row_stride = round_up(2*cols, 16).
+ *   F32   row r = cols fp32 values;     row_stride = round_up(4*cols, 16).
  * Values are exactly those of the reference's 34-byte block stream / half
  * array; only the placement differs, so that every 16-byte load of a row is
  * aligned and a warp reads 512 contiguous bytes.
@@ -33,8 +35,10 @@ extern "C" {
 #define B200_E_TOOLARGE (-2)
 #define B200_E_STATE    (-3)
 
-#define B200_WT_Q8  0
-#define B200_WT_F16 1
+#define B200_WT_Q8   0
+#define B200_WT_F16  1
+#define B200_WT_BF16 2
+#define B200_WT_F32  3
 
 #define B200_MAX_PEERS 8
 
@@ -47,6 +51,11 @@ size_t b200_packed_row_stride(int wtype, int cols);
 int b200_q8_pack(const float *d_src, long long ld, int rows, int cols,
                  void *d_dst, long long dst_row_stride, int dst_row0, int dst_row_step,
                  void *stream);
+/* fp32 rows -> bfloat16 (round to nearest even) or fp32 packed rows (wtype B200_WT_BF16 / B200_WT_F32). Any
+ * column count; the bytes of a row from cols up to dst_row_stride are written as zeros, so that a matrix
+ * can be given padding columns. No counterpart in the reference. */
+int b200_cast_pack(int wtype, const float *d_src, long long ld, int rows, int cols,
+                   void *d_dst, long long dst_row_stride, int dst_row0, int dst_row_step, void *stream);
 /* Same for F16 (src/nn/wmat.c:63-75). */
 int b200_f16_pack(const float *d_src, long long ld, int rows, int cols,
                   void *d_dst, long long dst_row_stride, int dst_row0, int dst_row_step,
@@ -71,12 +80,22 @@ int b200_q8_unpack_blocks(const void *d_packed, long long row_stride, int rows, 
  *                  block 0 stores h to resid_out; x = h
  *   B200_IN_EMBED  h = emb[tokens[*pos]][0..cols) * emb_scale; stored to
  *                  resid_out by block 0; x = h
- * then, if norm_gamma != NULL, x <- x * rsqrt(mean(x^2)+eps) * norm_gamma.
+ *   B200_IN_POSTNORM (BF16 / F32 weights) h = norm(in_vec) * slot_norm_gamma; block 0 stores h to
+ *                  post_copy (if not NULL); x = mix_in ? mix_in + *mix_coef * h : h, stored to
+ *                  resid_out by block 0 (if not NULL)
+ * then, if norm_gamma != NULL, x <- x * rsqrt(mean(x^2)+eps) * norm_gamma. With norm_groups > 1 the
+ * norms of BF16 / F32 launches treat that many equal consecutive parts of the vector separately;
+ * norm_dim (0 = cols) is the length they run over when the columns past it are padding.
  *
  * Output (out_mode):
  *   B200_OUT_STORE  out[p][out_offset + r] = y[r] for every peer p < n_out
  *   B200_OUT_GLU    rows come in (gate, up) pairs: out[0][out_offset + r/2] =
- *                   act(y[r]) * y[r+1], act = SiLU (0) or tanh-GELU (1)
+ *                   act(y[r]) * y[r+1], act = SiLU (0) or tanh-GELU (1). glu_rows > 0: only rows below
+ *                   it are pairs, row r above goes to out2[r - glu_rows] as it is
+ *   B200_OUT_GATED  (BF16 / F32 weights) out[0][r] = resid_alpha * out_resid[r]
+ *                   + sigmoid(out_gate[r] + out_gate_bias[r]) * y[r]
+ * BF16 / F32 launches can also cap what they store, y <- softcap * tanh(y / softcap), and form a depth
+ * sum for the rows they own, hist_out[r] = sum over j < hist_n of hist_coef[j] * hist[j * hist_stride + r].
  * With d_argmax_scratch != NULL (B200_OUT_STORE only) the launch also leaves
  * the largest y[r] and its row index plus out_offset (first one on ties, as
  * the reference's argmax) in *d_argmax_val[p] / *d_argmax_idx[p], p < n_argmax_out.
@@ -87,8 +106,8 @@ int b200_q8_unpack_blocks(const void *d_packed, long long row_stride, int rows, 
  * after its last store it writes E into signal_flags[p][signal_index], p < n_signal. A wait
  * that runs out sets *err = 1 and the kernel carries on without hanging.
  * ---------------------------------------------------------------------- */
-enum { B200_IN_VEC = 0, B200_IN_RESID = 1, B200_IN_EMBED = 2 };
-enum { B200_OUT_STORE = 0, B200_OUT_GLU = 1 };
+enum { B200_IN_VEC = 0, B200_IN_RESID = 1, B200_IN_EMBED = 2, B200_IN_POSTNORM = 3 };
+enum { B200_OUT_STORE = 0, B200_OUT_GLU = 1, B200_OUT_GATED = 2 };
 
 typedef struct b200_matvec_args {
     /* weights */
@@ -130,6 +149,13 @@ typedef struct b200_matvec_args {
     /* iterations of the bounded wait on d_wait_flags before the kernel gives up and sets *d_err = 1
      * (0 = default, about a second) */
     int spin_limit;
+    /* BF16 / F32 weights only (see above); all zero otherwise */
+    int norm_dim, norm_groups;
+    float *d_post_copy; const float *d_mix_in; const float *d_mix_coef;
+    const float *d_out_resid, *d_out_gate, *d_out_gate_bias; float resid_alpha;
+    const float *d_hist; int hist_n; long long hist_stride; const float *d_hist_coef; float *d_hist_out;
+    int glu_rows; float *d_out2;
+    float softcap;                 /* 0 = none */
 } b200_matvec_args;
 
 int b200_matvec(const b200_matvec_args *a, void *stream);
@@ -181,6 +207,89 @@ int    b200_attn_decode(const b200_attn_args *a, void *stream);
 #define B200_ATTN_STATIC_SCRATCH_FLOATS (1 << 18)      /* 1 MiB */
 #define B200_ATTN_STATIC_MAX_KV_HEADS   64
 int b200_attn_decode_static(const b200_attn_args *a, void *stream);
+
+/* ------------------------------------------------------------------------
+ * Latent attention: keys and values of all heads are linear maps of one low-rank vector per token, and
+ * one rotated key part is shared by the heads, so the cache holds kv_rank + rot_dim numbers a token.
+ *
+ *   q     head by head [dim unrotated | rot_dim rotated]
+ *   c     = rms_norm(dkv[0 .. kv_rank)) * dkv_gamma
+ *   kr    = rotate(dkv[kv_rank .. kv_rank + rot_dim))
+ *   score = scale * (q_unrotated . (W_uk c) + rotate(q_rotated) . kr)   over the visible positions
+ *   out   = sigmoid(gate) * sum softmax(score) (W_uv c)
+ *
+ * Rotation: the pair (2i, 2i+1), i < rot_dims/2, turns by the angle whose (cos, sin) d_rope holds,
+ * [max_seq][rot_dims/2][2]; the rest of the rotated part passes unchanged. Position i sees j with
+ * 0 <= i - j < window (window <= 0: every j <= i).
+ *
+ * With up8(n) = n rounded up to a multiple of 8: a cache row is [up8(kv_rank) | up8(rot_dim)] elements of
+ * the type `wtype` names (BF16 or F32), padding zero. d_w_uk_t: per head [kv_rank][up8(dim)] (the
+ * transposed map). d_w_kv: per head up8(dim) rows of W_uk and up8(vdim) rows of W_uv, up8(kv_rank)
+ * columns. All vectors of the decode form are fp32.
+ *
+ * Decode (b200_latent_decode, three launches): one new token at *d_pos. The query is moved into the latent
+ * space (q_lat = W_uk^T q), the scores and the weighted sum run over cache rows with all heads sharing
+ * the row loads, split over the sequence, and W_uv is applied once to the merged sum.
+ * Rows (b200_latent_rows_*): n_rows tokens from position pos0 on. _prep writes their cache rows and
+ * d_q_rows; the caller forms d_kv = cache rows x d_w_kv^T for positions kv_row0 .. pos0 + n_rows - 1;
+ * _attend runs the attention (BF16: tensor cores, F32: CUDA cores).
+ * ---------------------------------------------------------------------- */
+typedef struct b200_latent_args {
+    int wtype;
+    int heads, dim, rot_dim, rot_dims, vdim, kv_rank, window, max_seq;
+    float scale, eps;
+    const float *d_q, *d_dkv, *d_gate;   /* one token, or n_rows rows proj_ld floats apart */
+    const float *d_dkv_gamma, *d_rope;
+    void *d_cache;
+    const void *d_w_uk_t, *d_w_kv;
+    /* decode */
+    float *d_qlat;                       /* [heads][up8(kv_rank) + up8(rot_dim)] */
+    float *d_part;                       /* [heads][n_split][up8(kv_rank) + 8] */
+    float *d_out;                        /* [heads * vdim] */
+    const int *d_pos;
+    int n_split, use_pdl;
+    /* rows */
+    int n_rows, pos0, kv_row0;
+    long long proj_ld;
+    void *d_q_rows;                      /* [n_rows][heads][up8(dim) + up8(rot_dim)] */
+    const void *d_kv; long long kv_ld;   /* [pos0 + n_rows - kv_row0] rows of [heads][up8(dim) + up8(vdim)], kv_ld elements apart */
+    void *d_out_rows; long long out_ld;  /* [n_rows] rows of heads * vdim, out_ld elements apart */
+} b200_latent_args;
+
+/* Splits of the sequence worth launching for this shape (1 .. 256). */
+int b200_latent_splits(int heads, int window, int max_seq);
+int b200_latent_decode(const b200_latent_args *a, void *stream);
+int b200_latent_rows_prep(const b200_latent_args *a, void *stream);
+int b200_latent_rows_attend(const b200_latent_args *a, void *stream);
+
+/* ------------------------------------------------------------------------
+ * Row-wise steps of a prompt portion. Rows are ld floats apart; columns dim .. ld-1 are padding and are
+ * written as zeros. out_h (BF16 copies for the tensor-core products) may be NULL.
+ * ---------------------------------------------------------------------- */
+/* x[m] = scale * emb[tokens[m]], emb [vocab][ld]. */
+int b200_rows_embed(const float *emb, const uint32_t *tokens, int rows, int vocab, int ld, float scale,
+                    float *x, void *out_h, void *stream);
+/* z = alpha * x + sigmoid(gate + bias) * y; xn = grouped RMS norm of z times gamma, stored to `norm_out`;
+ * with hist_n > 0: out = sum over j < hist_n of coef[j] * hist[j][m] + coef[hist_n] * xn, else out = xn.
+ * hist[j] is [rows][ld], hist_stride floats apart. out may equal norm_out when hist_n == 0. */
+typedef struct b200_rows_postnorm_args {
+    const float *x, *y; long long y_ld;
+    const float *gate; long long gate_ld; const float *gate_bias;
+    const float *gamma;
+    float alpha, eps;
+    int rows, dim, ld, groups;
+    float *norm_out;
+    const float *hist; int hist_n; long long hist_stride; const float *coef;
+    float *out; void *out_h;
+} b200_rows_postnorm_args;
+int b200_rows_postnorm(const b200_rows_postnorm_args *a, void *stream);
+/* out[m] = grouped RMS norm of x[index[m]] times gamma; wtype: element type of out (BF16 or F32). */
+int b200_rows_norm(const float *x, const int *index, int rows, int dim, int ld, int groups, float eps,
+                   const float *gamma, int wtype, void *out, void *stream);
+/* out[m][i] = gelu_tanh(gu[m][2i]) * gu[m][2i+1], i < inter; out rows inter elements apart. */
+int b200_rows_gelu_mul(const float *gu, long long gu_ld, int rows, int inter, int wtype, void *out, void *stream);
+/* x <- cap * tanh(x / cap) over rows of dim floats, ld apart. */
+int b200_rows_softcap(float *x, int rows, int dim, long long ld, float cap, void *stream);
 
 /* Last tensor-parallel step of a token: waits for every rank's (value, index)
  * pair, takes the largest (lowest index on ties), stores it as tokens[pos+1]

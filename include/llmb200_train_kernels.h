@@ -38,6 +38,8 @@ typedef struct {
     float alpha;
     unsigned *d_err;     /* optional device word; the tensor-core kernel stores a non-zero code there when a
                             bounded wait runs out (the product is then incomplete) */
+    void *Ch; long long ldch;   /* b200_gemm_bf16 only: when not NULL the result is stored here as bfloat16 and C is
+                                   not written (R must be NULL) */
 } b200_gemm_args;
 
 /* CUDA-core version: any shape, any of the stride combinations above. */
@@ -54,6 +56,8 @@ int b200_gemm_tf32(const b200_gemm_args *a, void *stream);
  * 8), C and R stay fp32, accumulation is fp32. Half the operand bytes of the
  * TF32 form, which is what bounds the kernel. */
 int b200_gemm_f16(const b200_gemm_args *a, void *stream);
+/* The same kernel on bfloat16 operands (fp32's range, 8 significant bits; also kind::f16). */
+int b200_gemm_bf16(const b200_gemm_args *a, void *stream);
 /* dst[i] = binary16(src[i] * scale), round to nearest even: the operand copies
  * b200_gemm_f16 reads (gradients are scaled by a power of two into binary16's
  * range and the product scaled back through alpha). */

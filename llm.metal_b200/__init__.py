@@ -20,10 +20,10 @@ c_uint_p = C.POINTER(C.c_uint)
 c_u32_p = C.POINTER(C.c_uint32)
 
 B200_MAX_PEERS = 8
-B200_WT_Q8, B200_WT_F16 = 0, 1
-B200_IN_VEC, B200_IN_RESID, B200_IN_EMBED = 0, 1, 2
-B200_OUT_STORE, B200_OUT_GLU = 0, 1
-MODEL_QWEN3, MODEL_GEMMA3 = 0, 1
+B200_WT_Q8, B200_WT_F16, B200_WT_BF16, B200_WT_F32 = 0, 1, 2, 3
+B200_IN_VEC, B200_IN_RESID, B200_IN_EMBED, B200_IN_POSTNORM = 0, 1, 2, 3
+B200_OUT_STORE, B200_OUT_GLU, B200_OUT_GATED = 0, 1, 2
+MODEL_QWEN3, MODEL_GEMMA3, MODEL_MORILORN = 0, 1, 2
 LLMB200_HANDLE_BYTES = 64
 
 
@@ -55,6 +55,12 @@ class MatvecArgs(C.Structure):
         ("d_err", C.c_void_p),
         ("grid", C.c_int), ("use_pdl", C.c_int),
         ("d_in_copy", C.c_void_p), ("spin_limit", C.c_int),
+        ("norm_dim", C.c_int), ("norm_groups", C.c_int),
+        ("d_post_copy", C.c_void_p), ("d_mix_in", C.c_void_p), ("d_mix_coef", C.c_void_p),
+        ("d_out_resid", C.c_void_p), ("d_out_gate", C.c_void_p), ("d_out_gate_bias", C.c_void_p), ("resid_alpha", C.c_float),
+        ("d_hist", C.c_void_p), ("hist_n", C.c_int), ("hist_stride", C.c_longlong), ("d_hist_coef", C.c_void_p),
+        ("d_hist_out", C.c_void_p),
+        ("glu_rows", C.c_int), ("d_out2", C.c_void_p), ("softcap", C.c_float),
     ]
 
 
@@ -137,7 +143,29 @@ class GemmArgs(C.Structure):
                 ("B", C.c_void_p), ("b_row", C.c_longlong), ("b_col", C.c_longlong),
                 ("C", C.c_void_p), ("ldc", C.c_longlong),
                 ("R", C.c_void_p), ("ldr", C.c_longlong),
-                ("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("alpha", C.c_float), ("d_err", C.c_void_p)]
+                ("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("alpha", C.c_float), ("d_err", C.c_void_p),
+                ("Ch", C.c_void_p), ("ldch", C.c_longlong)]
+
+
+class LatentArgs(C.Structure):
+    """b200_latent_args (include/llmb200_kernels.h)."""
+    _fields_ = [("wtype", C.c_int)] + \
+               [(n, C.c_int) for n in ("heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank", "window", "max_seq")] + \
+               [("scale", C.c_float), ("eps", C.c_float)] + \
+               [(n, C.c_void_p) for n in ("d_q", "d_dkv", "d_gate", "d_dkv_gamma", "d_rope", "d_cache", "d_w_uk_t", "d_w_kv",
+                                          "d_qlat", "d_part", "d_out", "d_pos")] + \
+               [(n, C.c_int) for n in ("n_split", "use_pdl", "n_rows", "pos0", "kv_row0")] + \
+               [("proj_ld", C.c_longlong), ("d_q_rows", C.c_void_p), ("d_kv", C.c_void_p), ("kv_ld", C.c_longlong),
+                ("d_out_rows", C.c_void_p), ("out_ld", C.c_longlong)]
+
+
+class RowsPostnormArgs(C.Structure):
+    """b200_rows_postnorm_args (include/llmb200_kernels.h)."""
+    _fields_ = [("x", C.c_void_p), ("y", C.c_void_p), ("y_ld", C.c_longlong), ("gate", C.c_void_p), ("gate_ld", C.c_longlong),
+                ("gate_bias", C.c_void_p), ("gamma", C.c_void_p), ("alpha", C.c_float), ("eps", C.c_float),
+                ("rows", C.c_int), ("dim", C.c_int), ("ld", C.c_int), ("groups", C.c_int),
+                ("norm_out", C.c_void_p), ("hist", C.c_void_p), ("hist_n", C.c_int), ("hist_stride", C.c_longlong),
+                ("coef", C.c_void_p), ("out", C.c_void_p), ("out_h", C.c_void_p)]
 
 
 class WMat(C.Structure):
@@ -165,9 +193,11 @@ SYMBOLS_MAIN = {
     "llmb200_wmat.h": ["fast_metal_init", "fast_metal_shutdown", "metal_flush", "metal_buf_create", "metal_buf_from_data",
                        "metal_buf_free", "metal_buf_ptr", "wmat_create_q8", "wmat_create_f16", "wmat_free", "wmat_convert",
                        "norm_upload", "layers_convert_upload", "layers_free", "metal_enqueue_scale", "metal_enqueue_grpo_policy_grad"],
-    "llmb200_kernels.h": ["b200_packed_row_stride", "b200_q8_pack", "b200_f16_pack", "b200_q8_unpack_blocks", "b200_matvec",
+    "llmb200_kernels.h": ["b200_packed_row_stride", "b200_q8_pack", "b200_f16_pack", "b200_cast_pack", "b200_q8_unpack_blocks", "b200_matvec",
                           "b200_attn_scratch_floats", "b200_attn_decode", "b200_attn_decode_static", "b200_tp_argmax_finalize", "b200_token_plan", "b200_token_chunks", "b200_decode_token", "b200_lora_decode", "b200_argmax_rows",
-                          "b200_launch_count", "b200_launch_count_add"],
+                          "b200_launch_count", "b200_launch_count_add",
+                          "b200_latent_splits", "b200_latent_decode", "b200_latent_rows_prep", "b200_latent_rows_attend", "b200_rows_embed",
+                          "b200_rows_postnorm", "b200_rows_norm", "b200_rows_gelu_mul", "b200_rows_softcap"],
     "llmb200_inference.h": ["inference_state_create", "inference_state_create_gemma3", "inference_state_free",
                             "inference_generate", "inference_state_model_type", "inference_state_vocab_size",
                             "inference_state_reset", "inference_forward_token", "inference_state_load_eos",
@@ -177,10 +207,10 @@ SYMBOLS_MAIN = {
                             "llmb200_state_error", "llmb200_state_connect_loopback", "llmb200_state_run_device_steps", "llmb200_state_profile_token",
                             "llmb200_state_time_kind", "llmb200_state_step_trace",
                             "llmb200_state_weight_bytes", "llmb200_state_position", "llmb200_state_graph_kernels",
-                            "llmb200_state_export_weight", "llmb200_batch_begin", "llmb200_batch_load_layer",
+                            "llmb200_state_export_weight", "inference_state_create_from_dir", "inference_forward_tokens", "llmb200_batch_begin", "llmb200_batch_load_layer",
                             "llmb200_batch_finish", "llmb200_batch_set_eos", "llmb200_batch_generate",
                             "llmb200_batch_last_decode_ms", "llmb200_batch_graph_kernels", "llmb200_batch_logits", "llmb200_batch_free"],
-    "llmb200_train_kernels.h": ["b200_gemm_f32", "b200_gemm_tf32", "b200_gemm_f16", "b200_f32_to_f16", "b200_transpose_f16", "b200_lora_pack_f16", "b200_embed_rows", "b200_round_f16",
+    "llmb200_train_kernels.h": ["b200_gemm_f32", "b200_gemm_tf32", "b200_gemm_f16", "b200_gemm_bf16", "b200_f32_to_f16", "b200_transpose_f16", "b200_lora_pack_f16", "b200_embed_rows", "b200_round_f16",
                                 "b200_transpose_f32", "b200_rms_norm_rows", "b200_rms_norm_bwd_rows",
                                 "b200_qk_norm_rope", "b200_qk_norm_rope_bwd", "b200_attn_train_fwd",
                                 "b200_attn_train_bwd", "b200_silu_mul_rows", "b200_silu_mul_bwd_rows", "b200_lora_add", "b200_lora_pack", "b200_xty_skinny",
@@ -222,7 +252,7 @@ def lib():
         return _lib
     path = _build.LIB
     if not os.path.exists(path):
-        _build.build_main()
+        _build.build_main_locked()
     L = C.CDLL(path)
     vp, i, ll, sz, fl = C.c_void_p, C.c_int, C.c_longlong, C.c_size_t, C.c_float
     sig = {
@@ -278,9 +308,17 @@ def lib():
         "llmb200_state_weight_bytes": (C.c_ulonglong, [vp]), "llmb200_state_position": (i, [vp]),
         "llmb200_state_graph_kernels": (i, [vp, i]),
         "llmb200_state_export_weight": (sz, [vp, i, i, vp, sz]),
+        "inference_state_create_from_dir": (vp, [C.c_char_p, i, i]),
+        "inference_forward_tokens": (i, [vp, c_u32_p, i, c_int_p, i, c_float_p]),
+        "b200_cast_pack": (i, [i, vp, ll, i, i, vp, ll, i, i, vp]),
+        "b200_latent_splits": (i, [i, i, i]), "b200_latent_decode": (i, [C.POINTER(LatentArgs), vp]),
+        "b200_latent_rows_prep": (i, [C.POINTER(LatentArgs), vp]), "b200_latent_rows_attend": (i, [C.POINTER(LatentArgs), vp]),
+        "b200_rows_embed": (i, [vp, vp, i, i, i, fl, vp, vp, vp]), "b200_rows_postnorm": (i, [C.POINTER(RowsPostnormArgs), vp]),
+        "b200_rows_norm": (i, [vp, vp, i, i, i, i, fl, vp, i, vp, vp]), "b200_rows_gelu_mul": (i, [vp, ll, i, i, i, vp, vp]),
+        "b200_rows_softcap": (i, [vp, i, i, ll, fl, vp]),
         # ---- llmb200_train_kernels.h
         "b200_gemm_f32": (i, [C.POINTER(GemmArgs), vp]), "b200_gemm_tf32": (i, [C.POINTER(GemmArgs), vp]),
-        "b200_gemm_f16": (i, [C.POINTER(GemmArgs), vp]), "b200_f32_to_f16": (i, [vp, sz, fl, vp, vp]),
+        "b200_gemm_f16": (i, [C.POINTER(GemmArgs), vp]), "b200_gemm_bf16": (i, [C.POINTER(GemmArgs), vp]), "b200_f32_to_f16": (i, [vp, sz, fl, vp, vp]),
         "b200_transpose_f16": (i, [vp, i, i, vp, vp]),
         "b200_lora_pack_f16": (i, [vp, vp, vp, vp, vp, vp, i, i, i, i, i, fl, vp]),
         "b200_embed_rows": (i, [vp, vp, i, i, i, fl, vp, vp]),
@@ -371,6 +409,66 @@ def synth():
     S.llmb200_abi_layout.restype, S.llmb200_abi_layout.argtypes = i, [C.POINTER(sz), i]
     _synth = S
     return S
+
+
+class DirModel:
+    """A model folder (config.json, model.safetensors) opened through inference_state_create_from_dir: one live
+    sequence, fed in portions of any size, or greedy generation. Standard library only."""
+    DTYPES = {"bfloat16": B200_WT_BF16, "float32": B200_WT_F32}
+
+    def __init__(self, path, max_tokens, dtype="bfloat16"):
+        self.lib = lib()
+        self.state = self.lib.inference_state_create_from_dir(os.fsencode(path), max_tokens, self.DTYPES[dtype])
+        if not self.state:
+            raise RuntimeError(f"opening the model folder {path} failed")
+        self.vocab = self.lib.inference_state_vocab_size(self.state)
+
+    def close(self):
+        if self.state:
+            self.lib.inference_state_free(self.state)
+            self.state = None
+
+    def __enter__(self):
+        return self
+
+    def __exit__(self, *_):
+        self.close()
+
+    @property
+    def position(self):
+        return self.lib.llmb200_state_position(self.state)
+
+    def reset(self):
+        """Ends the live sequence: what it holds in the cache is given back."""
+        self.lib.inference_state_reset(self.state)
+
+    def feed(self, tokens, want=()):
+        """Runs `tokens` after what the sequence holds; the logits of the places `want` among them, in that
+        order, as one flat ctypes float array of len(want) * vocab."""
+        n = len(tokens)
+        order = sorted(set(want))
+        buf = (C.c_float * max(1, len(order) * self.vocab))()
+        rc = self.lib.inference_forward_tokens(self.state, (C.c_uint32 * n)(*tokens), n, (C.c_int * max(1, len(order)))(*order),
+                                               len(order), C.cast(buf, c_float_p))
+        if rc != 0:
+            raise RuntimeError(f"inference_forward_tokens failed with code {rc}")
+        if list(want) == order:
+            return buf
+        out = (C.c_float * max(1, len(want) * self.vocab))()
+        for i, w in enumerate(want):
+            k = order.index(w)
+            out[i * self.vocab:(i + 1) * self.vocab] = buf[k * self.vocab:(k + 1) * self.vocab]
+        return out
+
+    def generate(self, prompt, max_new, eos=None):
+        """Greedy continuation of a prompt through inference_generate (starts a new sequence)."""
+        if eos is not None:
+            self.lib.llmb200_state_set_eos(self.state, (C.c_int * max(1, len(eos)))(*eos), len(eos))
+        out = (C.c_uint32 * max_new)()
+        n = self.lib.inference_generate(self.state, (C.c_uint32 * len(prompt))(*prompt), len(prompt), out, max_new)
+        if n < 1:
+            raise RuntimeError("inference_generate failed")
+        return list(out[:n])
 
 
 # ---- the architectures the benchmarks and tests use ------------------------------------------------

@@ -6,6 +6,8 @@
 Sources are compiled only when they are newer than the library, so importing
 the package on a machine that received prebuilt libraries costs nothing.
 """
+import concurrent.futures
+import fcntl
 import os
 import shutil
 import subprocess
@@ -21,8 +23,9 @@ OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libllmb200.so")
 LIB_SYNTH = os.path.join(HERE, "libllmb200_synth.so")
 
-CU_SOURCES = ["pack.cu", "matvec.cu", "attention.cu", "decode_token.cu", "lora_decode.cu", "batch_kernels.cu", "gemm_f32.cu", "gemm_tf32.cu", "train_kernels.cu"]
-C_SOURCES = ["weights.c", "decode_engine.c", "sft_engine.c", "batch_engine.c"]
+CU_SOURCES = ["pack.cu", "matvec.cu", "attention.cu", "decode_token.cu", "lora_decode.cu", "batch_kernels.cu", "gemm_f32.cu", "gemm_tf32.cu", "train_kernels.cu",
+              "latent_attention.cu", "row_kernels.cu"]
+C_SOURCES = ["weights.c", "decode_engine.c", "sft_engine.c", "batch_engine.c", "json.c", "tensor_file.c", "model_dir.c", "latent_model.c"]
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC"]
@@ -64,21 +67,38 @@ def build_main(force=False, verbose=False):
         return LIB
     os.makedirs(OBJ, exist_ok=True)
     nvcc = _nvcc()
-    objs = []
-    for f in CU_SOURCES:
-        o = os.path.join(OBJ, f + ".o")
-        flags = NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else [])
-        out = _run([nvcc] + flags + ["-c", os.path.join(CSRC, f), "-o", o])
-        if verbose:
-            sys.stderr.write(out)
-        objs.append(o)
-    for f in C_SOURCES:
-        o = os.path.join(OBJ, f + ".o")
-        _run(["gcc", "-O2", "-std=gnu11", "-fPIC", "-Wall", "-Wno-unused-function",
-              "-I", os.path.join(CUDA_HOME, "include"), "-c", os.path.join(HOST, f), "-o", o])
-        objs.append(o)
-    _run([nvcc, "-shared", "-o", LIB] + objs + ["-cudart", "static", "-lm", "-lpthread", "-ldl", "-lrt"])
+    headers = _headers()
+
+    def compile_one(f):
+        """Compiles one source unless its object is newer than it and every header."""
+        cu = f.endswith(".cu")
+        src, o = os.path.join(CSRC if cu else HOST, f), os.path.join(OBJ, f + ".o")
+        if force or _newer(o, [src] + headers):
+            part = f"{o}.{os.getpid()}"
+            if cu:
+                out = _run([nvcc] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-c", src, "-o", part])
+                if verbose:
+                    sys.stderr.write(out)
+            else:
+                _run(["gcc", "-O2", "-std=gnu11", "-fPIC", "-Wall", "-Wno-unused-function",
+                      "-I", os.path.join(CUDA_HOME, "include"), "-c", src, "-o", part])
+            os.replace(part, o)
+        return o
+
+    with concurrent.futures.ThreadPoolExecutor(max(1, min(16, os.cpu_count() or 1))) as pool:
+        objs = list(pool.map(compile_one, CU_SOURCES + C_SOURCES))
+    part = f"{LIB}.{os.getpid()}"
+    _run([nvcc, "-shared", "-o", part] + objs + ["-cudart", "static", "-lm", "-lpthread", "-ldl", "-lrt"])
+    os.replace(part, LIB)                # a process that has the library mapped keeps its own copy
     return LIB
+
+
+def build_main_locked():
+    """build_main() for several processes that may find the library missing at the same time."""
+    os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        return build_main()
 
 
 def build_synth(force=False):

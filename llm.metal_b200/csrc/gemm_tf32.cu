@@ -1,7 +1,8 @@
 // Tensor-core GEMM for the frozen projections of the LoRA-SFT step (sm_100a only).
 //
 //   C[M,N] = alpha * A[M,K] * B[N,K]^T (+ R),  C, R fp32 row-major; A and B contiguous along k, either
-//   binary16 (b200_gemm_f16: tcgen05.mma kind::f16) or fp32 read as TF32 (b200_gemm_tf32: kind::tf32).
+//   binary16 or bfloat16 (b200_gemm_f16 / _bf16: tcgen05.mma kind::f16) or fp32 read as TF32 (b200_gemm_tf32:
+//   kind::tf32). The bfloat16 form can store C as bfloat16 instead.
 //
 // Replaces the reference's scalar tiled products f16_matmul / f16_matmul_nt
 // (shaders/q8_kernels.metal:383-435) for the seven projections and the LM head,
@@ -25,6 +26,7 @@
 #include "../../include/llmb200_train_kernels.h"
 
 #include <cuda.h>
+#include <cuda_bf16.h>
 #include <stdlib.h>
 #include <string.h>
 
@@ -46,10 +48,11 @@ struct EpiArgs {
     int bn;            // columns of the output tile = N of one tcgen05.mma (a multiple of 16, 64..256)
     int stages;        // ring slots
     int tmem_cols;     // tensor-memory columns to allocate: the power of two >= bn
-    int f16;           // 0: fp32 operands read as TF32 (32 per 128-byte row); 1: binary16 operands (64 per row)
+    int f16;           // 0: fp32 operands read as TF32 (32 per 128-byte row); 1 / 2: binary16 / bfloat16 operands (64 per row)
     int ksub;          // 128-byte-wide k sub-tiles per ring slot (each its own 128-byte-swizzled block)
     int splits;        // CTAs sharing one output tile along k (gridDim.z); 1 = none
     unsigned *flags;   // one turn counter per output tile, zero between launches
+    __nv_bfloat16 *Ch; long long ldch;   // bfloat16 result instead of C (never with splits > 1)
 };
 
 // Turn counters of the serial split-k epilogue (see the kernel): one word per output tile.
@@ -180,8 +183,8 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
     } else if (warp == 1) {
         if (lane == 0) {
             // instruction descriptor: D fp32, A and B TF32, both K-major, N = BN, M = 128
-            // (operand format field: 2 = TF32, 0 = F16; an MMA covers 32 bytes of k either way: 8 or 16 elements)
-            const uint32_t fmt = p.f16 ? 0u : 2u;
+            // (operand format field: 2 = TF32, 0 = F16, 1 = BF16; an MMA covers 32 bytes of k either way: 8 or 16 elements)
+            const uint32_t fmt = p.f16 == 0 ? 2u : p.f16 == 1 ? 0u : 1u;
             const uint32_t idesc = (1u << 4) | (fmt << 7) | (fmt << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
             bool ok = true;
             for (int kb = 0; kb < nkb && ok; ++kb) {
@@ -249,7 +252,27 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 const int cw = min(32, BN - c);                 // columns of this chunk that belong to the tile
                 uint32_t r[32];
                 tmem_ld32(tmem_base + ((uint32_t)lane_base << 16) + (uint32_t)c, r);
-                if (row < p.M) {
+                if (row < p.M && p.Ch) {
+                    __nv_bfloat16 *hrow = p.Ch + (long long)row * p.ldch + n0 + c;      // 16-byte aligned: checked by the host
+                    if (cw == 32 && n0 + c + 32 <= p.N) {
+#pragma unroll
+                        for (int j = 0; j < 32; j += 8) {
+                            uint4 v;
+                            uint32_t *vw = reinterpret_cast<uint32_t *>(&v);
+#pragma unroll
+                            for (int k = 0; k < 4; ++k) {
+                                const __nv_bfloat162 h = __floats2bfloat162_rn(p.alpha * __uint_as_float(r[j + 2 * k]),
+                                                                               p.alpha * __uint_as_float(r[j + 2 * k + 1]));
+                                vw[k] = *reinterpret_cast<const uint32_t *>(&h);
+                            }
+                            *reinterpret_cast<uint4 *>(hrow + j) = v;
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j)
+                            if (j < cw && n0 + c + j < p.N) hrow[j] = __float2bfloat16_rn(p.alpha * __uint_as_float(r[j]));
+                    }
+                } else if (row < p.M) {
                     if (vec && cw == 32 && n0 + c + 32 <= p.N) {
 #pragma unroll
                         for (int j = 0; j < 32; j += 4) {
@@ -331,7 +354,9 @@ bool make_map(CUtensorMap *map, const void *base, long long rows, long long K, l
     const cuuint64_t strides[1] = {(cuuint64_t)ld * (f16 ? 2 : 4)};
     const cuuint32_t box[2] = {(cuuint32_t)(f16 ? 2 * BK : BK), (cuuint32_t)box_rows};
     const cuuint32_t estr[2] = {1, 1};
-    return enc(map, f16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 2, const_cast<void *>(base),
+    const CUtensorMapDataType type = f16 == 0 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT32 : f16 == 1 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16
+                                                                                           : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    return enc(map, type, 2, const_cast<void *>(base),
                dims, strides, box, estr,
                CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
@@ -427,7 +452,8 @@ int launch(const CUtensorMap &ma, const CUtensorMap &mb, EpiArgs e, cudaStream_t
 
 static int gemm_tc(const b200_gemm_args *a, int f16, void *stream)
 {
-    if (!a || !a->A || !a->B || !a->C || a->M <= 0 || a->N <= 0 || a->K <= 0) return B200_E_BADARG;
+    if (!a || !a->A || !a->B || (!a->C && !a->Ch) || a->M <= 0 || a->N <= 0 || a->K <= 0) return B200_E_BADARG;
+    if (a->Ch && (f16 != 2 || a->R || (a->ldch & 7) || (reinterpret_cast<uintptr_t>(a->Ch) & 15))) return B200_E_BADARG;
     if (a->a_col != 1 || a->b_row != 1) return B200_E_UNSUPPORTED;
     const long long lda = a->a_row, ldb = a->b_col;
     const int gran = f16 ? 7 : 3;                                  // 16-byte granularity of rows and of k
@@ -437,7 +463,8 @@ static int gemm_tc(const b200_gemm_args *a, int f16, void *stream)
     if ((a->N + 63) / 64 > 65535) return B200_E_UNSUPPORTED;
 
     CUtensorMap ma, mb;
-    EpiArgs e = {a->C, a->ldc, a->R, a->ldr, a->M, a->N, a->K, a->alpha, a->d_err, 128, 0, 0, f16, 1, 1, nullptr};
+    EpiArgs e = {a->C, a->ldc, a->R, a->ldr, a->M, a->N, a->K, a->alpha, a->d_err, 128, 0, 0, f16, 1, 1, nullptr,
+                 static_cast<__nv_bfloat16 *>(a->Ch), a->ldch};
     // LLMB200_GEMM_BN=<n> overrides the tile width for experiments
     static int forced = -1;
     if (forced < 0) {
@@ -447,6 +474,7 @@ static int gemm_tc(const b200_gemm_args *a, int f16, void *stream)
     }
     pick_tile(a->M, a->N, a->K, f16, &e.bn, &e.ksub, &e.splits);
     if (forced >= 64) { e.bn = forced; e.splits = 1; }
+    if (e.Ch) e.splits = 1;
     if (!make_map(&ma, a->A, a->M, a->K, lda, BM, f16)) return B200_E_UNSUPPORTED;
     if (!make_map(&mb, a->B, a->N, a->K, ldb, e.bn, f16)) return B200_E_UNSUPPORTED;
     return launch(ma, mb, e, (cudaStream_t)stream);
@@ -454,3 +482,4 @@ static int gemm_tc(const b200_gemm_args *a, int f16, void *stream)
 
 extern "C" int b200_gemm_tf32(const b200_gemm_args *a, void *stream) { return gemm_tc(a, 0, stream); }
 extern "C" int b200_gemm_f16(const b200_gemm_args *a, void *stream) { return gemm_tc(a, 1, stream); }
+extern "C" int b200_gemm_bf16(const b200_gemm_args *a, void *stream) { return gemm_tc(a, 2, stream); }

@@ -1,0 +1,701 @@
+// Latent attention (sm_100a): keys and values of all heads are linear maps of one cached low-rank vector.
+//
+// Decode, three launches chained by programmatic dependent launch:
+//   latent_absorb  per head q_lat = scale * W_uk^T q (the weight slice of a block is in registers before the
+//                  previous kernel has finished); one extra block normalises the new token's latent, rotates its
+//                  key part and the queries, and writes the cache row
+//   latent_scores  split-sequence attention in the latent space: a block takes 32 cache rows at a time for eight
+//                  heads (one warp each), rows staged once in shared memory and used for the scores and for the
+//                  weighted sum; partial (sum, maximum, total) records per split
+//   latent_value   merges the splits of a head, applies W_uv and the output gate
+//
+// Prompt portions: latent_prep writes cache rows and rotated queries of all rows; keys and values are expanded
+// by a product the caller runs; latent_attend_bf16 is a tiled online-softmax attention on the tensor cores
+// (mma.sync m16n8k16, bfloat16 operands, fp32 scores, weights and sums), latent_attend_f32 the same sum in
+// fp32 on the CUDA cores.
+#include "stream_core.cuh"
+#include "../../include/llmb200_kernels.h"
+
+#include <cuda_bf16.h>
+
+extern unsigned long long g_b200_launches;
+
+namespace {
+
+constexpr int KT = 32;             // cache rows per tile of the decode scores = lanes of a warp
+constexpr int HB = 8;              // heads per block of the decode scores = warps
+constexpr int ABSORB_PASSES = 4;   // row passes whose weights a warp of latent_absorb holds in registers
+constexpr int VALUE_ROWS = 32;     // value rows per block of latent_value, four per warp
+constexpr int MAX_SPLITS = 256;
+
+__host__ __device__ __forceinline__ int up8(int n) { return (n + 7) & ~7; }
+
+template <int WT> struct Elem;
+template <> struct Elem<B200_WT_BF16> {
+    using T = __nv_bfloat16;
+    static constexpr int E = 8;
+    static __device__ __forceinline__ float dot(const uint4 &w, const float *x) { return dot8_bf16(w, x); }
+    static __device__ __forceinline__ void unpack(const uint4 &w, float *x)
+    {
+        const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const float2 f = bf16_pair(u[i]); x[2 * i] = f.x; x[2 * i + 1] = f.y; }
+    }
+};
+template <> struct Elem<B200_WT_F32> {
+    using T = float;
+    static constexpr int E = 4;
+    static __device__ __forceinline__ float dot(const uint4 &w, const float *x) { return dot4_f32(w, x); }
+    static __device__ __forceinline__ void unpack(const uint4 &w, float *x)
+    {
+        x[0] = __uint_as_float(w.x); x[1] = __uint_as_float(w.y); x[2] = __uint_as_float(w.z); x[3] = __uint_as_float(w.w);
+    }
+};
+
+// Element i of a rotated vector v whose first `dims` elements turn pairwise by the angles in rope (cos, sin).
+__device__ __forceinline__ float rotated(const float *v, int i, int dims, const float *rope)
+{
+    if (i >= dims) return v[i];
+    const float c = rope[i & ~1], s = rope[(i & ~1) + 1];
+    const float a = v[i & ~1], b = v[(i & ~1) + 1];
+    return (i & 1) ? b * c + a * s : a * c - b * s;
+}
+
+// The cache row of one token, by all threads of a block. `red` holds >= 33 floats.
+template <typename T>
+__device__ __forceinline__ void write_cache_row(const b200_latent_args &p, const float *dkv, int pos, float *red)
+{
+    const int R = p.kv_rank, R8 = up8(R), rot8 = up8(p.rot_dim);
+    T *row = static_cast<T *>(p.d_cache) + (size_t)pos * (R8 + rot8);
+    const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < R; i += blockDim.x) ss = fmaf(dkv[i], dkv[i], ss);
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)R + p.eps);
+    for (int i = threadIdx.x; i < R8; i += blockDim.x) row[i] = (T)(i < R ? p.d_dkv_gamma[i] * (dkv[i] * inv) : 0.0f);
+    for (int i = threadIdx.x; i < rot8; i += blockDim.x)
+        row[R8 + i] = (T)(i < p.rot_dim ? rotated(dkv + R, i, p.rot_dims, rope) : 0.0f);
+}
+
+// ------------------------------------------------------------------------------------------------ decode
+
+template <int WT>
+__global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constant__ b200_latent_args p, int chunks, int lpr)
+{
+    using El = Elem<WT>;
+    using T = typename El::T;
+    constexpr int E = El::E;
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    const int R = p.kv_rank, R8 = up8(R), rot8 = up8(p.rot_dim), CS = R8 + rot8, dq = p.dim + p.rot_dim;
+    if ((int)blockIdx.x == p.heads * chunks) {
+        pdl_wait();
+        const int pos = *p.d_pos;
+        if (pos < 0 || pos >= p.max_seq) return;
+        write_cache_row<T>(p, p.d_dkv, pos, red);
+        const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
+        for (int i = threadIdx.x; i < p.heads * rot8; i += blockDim.x) {
+            const int h = i / rot8, e = i % rot8;
+            p.d_qlat[(size_t)h * CS + R8 + e] =
+                e < p.rot_dim ? p.scale * rotated(p.d_q + (size_t)h * dq + p.dim, e, p.rot_dims, rope) : 0.0f;
+        }
+        return;
+    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.x / chunks, chunk = blockIdx.x % chunks;
+    const int dim8 = up8(p.dim), rpw = 32 / lpr, sl = lane % lpr;
+    const int row0 = (chunk * ABSORB_PASSES * 8 + warp) * rpw + lane / lpr;      // pass k adds k * 8 * rpw
+    const T *w0 = static_cast<const T *>(p.d_w_uk_t) + (size_t)h * R * dim8;
+    uint4 w[ABSORB_PASSES];
+#pragma unroll
+    for (int k = 0; k < ABSORB_PASSES; ++k) {
+        const int row = row0 + k * 8 * rpw;
+        w[k] = row < R && sl * E < dim8 ? *reinterpret_cast<const uint4 *>(w0 + (size_t)row * dim8 + sl * E) : make_uint4(0, 0, 0, 0);
+    }
+    pdl_wait();
+    const float *q = p.d_q + (size_t)h * dq;
+    float x[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) x[e] = sl * E + e < p.dim ? q[sl * E + e] : 0.0f;
+#pragma unroll
+    for (int k = 0; k < ABSORB_PASSES; ++k) {
+        const int row = row0 + k * 8 * rpw;
+        float acc = El::dot(w[k], x);
+        if (row < R)
+            for (int d = (sl + lpr) * E; d < dim8; d += lpr * E) {               // heads wider than a warp's slices
+                float y[E];
+#pragma unroll
+                for (int e = 0; e < E; ++e) y[e] = d + e < p.dim ? q[d + e] : 0.0f;
+                acc += El::dot(*reinterpret_cast<const uint4 *>(w0 + (size_t)row * dim8 + d), y);
+            }
+        for (int o = 1; o < lpr; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (sl == 0 && row < R) p.d_qlat[(size_t)h * CS + row] = p.scale * acc;
+    }
+    // padding columns of the latent part
+    if (chunk == 0 && threadIdx.x < R8 - R) p.d_qlat[(size_t)h * CS + R + threadIdx.x] = 0.0f;
+}
+
+template <int WT, int NCH>
+__global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constant__ b200_latent_args p, int row16)
+{
+    using El = Elem<WT>;
+    using T = typename El::T;
+    constexpr int E = El::E;
+    extern __shared__ __align__(16) unsigned char smem[];
+    pdl_launch_dependents();
+    const int R8 = up8(p.kv_rank), rot8 = up8(p.rot_dim), CS = R8 + rot8, PS = R8 + 8;
+    const int S = CS / E;                                    // 16-byte slices of a cache row
+    unsigned char *keys = smem;                              // [KT] rows, row16 slices apart (odd: no bank conflicts)
+    float *qs = reinterpret_cast<float *>(smem + (size_t)KT * row16 * 16);       // [HB][CS]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h0 = blockIdx.y * HB, h = h0 + warp, split = blockIdx.x;
+    const int pos = *p.d_pos;                                // changes only between tokens, not between their kernels
+    const bool valid = pos >= 0 && pos < p.max_seq;
+    const int lo = valid && p.window > 0 && pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
+    const int nk = valid ? pos - lo + 1 : 0;
+    const int tiles = (nk + KT - 1) / KT, per = (tiles + p.n_split - 1) / p.n_split;
+    const int t0 = split * per, t1 = min(t0 + per, tiles);
+    const T *cache = static_cast<const T *>(p.d_cache);
+
+    // every row but the new token's was written by an earlier token: the first tile is fetched before the wait
+    auto stage = [&](int tile, bool newest_only) {
+        const int k0 = tile * KT, n = min(KT, nk - k0);
+        for (int i = threadIdx.x; i < n * S; i += 256) {
+            const int r = i / S, c = i % S, kp = lo + k0 + r;
+            if ((kp == pos) != newest_only) continue;
+            *reinterpret_cast<uint4 *>(keys + ((size_t)r * row16 + c) * 16) =
+                *reinterpret_cast<const uint4 *>(cache + (size_t)kp * CS + (size_t)c * E);
+        }
+    };
+    if (t0 < t1) stage(t0, false);
+    pdl_wait();
+    for (int i = threadIdx.x; i < HB * CS; i += 256) qs[i] = h0 + i / CS < p.heads ? p.d_qlat[(size_t)h0 * CS + i] : 0.0f;
+
+    float m = -INFINITY, l = 0.0f, acc[NCH][E];
+#pragma unroll
+    for (int c = 0; c < NCH; ++c)
+#pragma unroll
+        for (int e = 0; e < E; ++e) acc[c][e] = 0.0f;
+    for (int tile = t0; tile < t1; ++tile) {
+        if (tile > t0) { __syncthreads(); stage(tile, false); }
+        if (tile == tiles - 1) stage(tile, true);
+        __syncthreads();
+        const int n = min(KT, nk - tile * KT);
+        float s = -INFINITY;
+        if (lane < n) {
+            const uint4 *kr = reinterpret_cast<const uint4 *>(keys + (size_t)lane * row16 * 16);
+            const float *q = qs + (size_t)warp * CS;
+            float a = 0.0f, b = 0.0f;
+            int c = 0;
+            for (; c + 1 < S; c += 2) { a += El::dot(kr[c], q + c * E); b += El::dot(kr[c + 1], q + (c + 1) * E); }
+            if (c < S) a += El::dot(kr[c], q + c * E);
+            s = a + b;
+        }
+        const float mt = fmaxf(m, warp_max(s));
+        const float w = lane < n ? expf(s - mt) : 0.0f;
+        const float corr = m == -INFINITY ? 0.0f : expf(m - mt);
+        l = l * corr + warp_sum(w);
+        m = mt;
+#pragma unroll
+        for (int c = 0; c < NCH; ++c)
+#pragma unroll
+            for (int e = 0; e < E; ++e) acc[c][e] *= corr;
+        for (int j = 0; j < n; ++j) {
+            const float wj = __shfl_sync(0xffffffffu, w, j);
+#pragma unroll
+            for (int c = 0; c < NCH; ++c) {
+                const int col = (c * 32 + lane) * E;
+                if (col < R8) {
+                    float v[E];
+                    El::unpack(*reinterpret_cast<const uint4 *>(keys + ((size_t)j * row16 + c * 32 + lane) * 16), v);
+#pragma unroll
+                    for (int e = 0; e < E; ++e) acc[c][e] = fmaf(wj, v[e], acc[c][e]);
+                }
+            }
+        }
+    }
+    if (h >= p.heads) return;
+    float *part = p.d_part + ((size_t)h * p.n_split + split) * PS;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+        const int col = (c * 32 + lane) * E;
+        if (col < R8)
+#pragma unroll
+            for (int e = 0; e < E; e += 4)
+                *reinterpret_cast<float4 *>(part + col + e) = make_float4(acc[c][e], acc[c][e + 1], acc[c][e + 2], acc[c][e + 3]);
+    }
+    if (lane == 0) { part[R8] = m; part[R8 + 1] = l; }
+}
+
+template <int WT>
+__global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant__ b200_latent_args p, int chunks)
+{
+    using El = Elem<WT>;
+    using T = typename El::T;
+    constexpr int E = El::E, RPW = VALUE_ROWS / 8, NS = 2;
+    extern __shared__ __align__(16) unsigned char smem[];
+    float *olat = reinterpret_cast<float *>(smem);           // [up8(kv_rank)]
+    __shared__ float sw[MAX_SPLITS];
+    pdl_launch_dependents();
+    const int R8 = up8(p.kv_rank), PS = R8 + 8, S = R8 / E;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.x / chunks, v0 = (blockIdx.x % chunks) * VALUE_ROWS + warp * RPW;
+    const int dim8 = up8(p.dim), per_head = dim8 + up8(p.vdim);
+    const T *w0 = static_cast<const T *>(p.d_w_kv) + ((size_t)h * per_head + dim8) * R8;
+    uint4 w[RPW][NS];
+#pragma unroll
+    for (int k = 0; k < RPW; ++k)
+#pragma unroll
+        for (int s = 0; s < NS; ++s)
+            w[k][s] = v0 + k < p.vdim && s * 32 + lane < S ? *reinterpret_cast<const uint4 *>(w0 + (size_t)(v0 + k) * R8 + (s * 32 + lane) * E)
+                                                           : make_uint4(0, 0, 0, 0);
+    pdl_wait();
+    const float *part = p.d_part + (size_t)h * p.n_split * PS;
+    if (warp == 0) {
+        float m = -INFINITY, l = 0.0f;
+        for (int s = lane; s < p.n_split; s += 32) m = fmaxf(m, part[(size_t)s * PS + R8]);
+        m = warp_max(m);
+        for (int s = lane; s < p.n_split; s += 32) {
+            const float ls = part[(size_t)s * PS + R8 + 1];
+            const float e = ls > 0.0f ? expf(part[(size_t)s * PS + R8] - m) : 0.0f;
+            sw[s] = e;
+            l = fmaf(e, ls, l);
+        }
+        l = warp_sum(l);
+        const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+        for (int s = lane; s < p.n_split; s += 32) sw[s] *= inv;
+    }
+    __syncthreads();
+    for (int r = threadIdx.x; r < R8; r += 256) {
+        float a = 0.0f;
+#pragma unroll 8
+        for (int s = 0; s < p.n_split; ++s) a = fmaf(sw[s], part[(size_t)s * PS + r], a);
+        olat[r] = a;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < RPW; ++k) {
+        if (v0 + k >= p.vdim) break;                         // uniform across the warp
+        float a = 0.0f;
+#pragma unroll
+        for (int s = 0; s < NS; ++s)
+            if (s * 32 + lane < S) a += El::dot(w[k][s], olat + (s * 32 + lane) * E);
+        for (int c = NS * 32 + lane; c < S; c += 32)
+            a += El::dot(*reinterpret_cast<const uint4 *>(w0 + (size_t)(v0 + k) * R8 + (size_t)c * E), olat + c * E);
+        a = warp_sum(a);
+        if (lane == 0) {
+            const int o = h * p.vdim + v0 + k;
+            p.d_out[o] = a * sigmoid_f32(p.d_gate[o]);
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ rows
+
+template <int WT>
+__global__ void __launch_bounds__(256) latent_prep_kernel(const __grid_constant__ b200_latent_args p)
+{
+    using T = typename Elem<WT>::T;
+    __shared__ float red[33];
+    const int m = blockIdx.x, pos = p.pos0 + m;
+    write_cache_row<T>(p, p.d_dkv + (size_t)m * p.proj_ld, pos, red);
+    const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), dq = p.dim + p.rot_dim, QS = dim8 + rot8;
+    const float *q = p.d_q + (size_t)m * p.proj_ld;
+    const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
+    T *out = static_cast<T *>(p.d_q_rows) + (size_t)m * p.heads * QS;
+    for (int i = threadIdx.x; i < p.heads * QS; i += blockDim.x) {
+        const int h = i / QS, e = i % QS;
+        const float *qh = q + (size_t)h * dq;
+        float v = 0.0f;
+        if (e < p.dim) v = qh[e];
+        else if (e >= dim8 && e - dim8 < p.rot_dim) v = rotated(qh + p.dim, e - dim8, p.rot_dims, rope);
+        out[i] = (T)v;
+    }
+}
+
+// fp32: one warp per (row, head), a lane per key, value columns over the lanes (256 per blockIdx.z).
+__global__ void __launch_bounds__(128) latent_attend_f32_kernel(const __grid_constant__ b200_latent_args p)
+{
+    extern __shared__ __align__(16) float qsh[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.y * 4 + warp, m = blockIdx.x, c0 = blockIdx.z * 256;
+    if (h >= p.heads) return;                                // warps are independent of one another
+    const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), QS = dim8 + rot8, vd8 = up8(p.vdim), R8 = up8(p.kv_rank), CS = R8 + rot8;
+    float *q = qsh + (size_t)warp * QS;
+    const float *qg = static_cast<const float *>(p.d_q_rows) + ((size_t)m * p.heads + h) * QS;
+    for (int i = lane; i < QS; i += 32) q[i] = qg[i];
+    __syncwarp();
+    const int pos = p.pos0 + m;
+    const int lo = p.window > 0 && pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
+    const float *kv = static_cast<const float *>(p.d_kv) + (size_t)h * (dim8 + vd8);
+    const float *cache = static_cast<const float *>(p.d_cache);
+    float mx = -INFINITY, l = 0.0f, acc[8];
+#pragma unroll
+    for (int c = 0; c < 8; ++c) acc[c] = 0.0f;
+    for (int k0 = lo; k0 <= pos; k0 += 32) {
+        const int n = min(32, pos - k0 + 1), kp = k0 + lane;
+        float s = -INFINITY;
+        if (lane < n) {
+            const float *kn = kv + (size_t)(kp - p.kv_row0) * p.kv_ld, *kr = cache + (size_t)kp * CS + R8;
+            float a = 0.0f, b = 0.0f;
+            for (int d = 0; d < p.dim; ++d) a = fmaf(q[d], kn[d], a);
+            for (int d = 0; d < p.rot_dim; ++d) b = fmaf(q[dim8 + d], kr[d], b);
+            s = p.scale * (a + b);
+        }
+        const float mt = fmaxf(mx, warp_max(s));
+        const float w = lane < n ? expf(s - mt) : 0.0f;
+        const float corr = mx == -INFINITY ? 0.0f : expf(mx - mt);
+        l = l * corr + warp_sum(w);
+        mx = mt;
+#pragma unroll
+        for (int c = 0; c < 8; ++c) acc[c] *= corr;
+        for (int j = 0; j < n; ++j) {
+            const float wj = __shfl_sync(0xffffffffu, w, j);
+            const float *v = kv + (size_t)(k0 + j - p.kv_row0) * p.kv_ld + dim8;
+#pragma unroll
+            for (int c = 0; c < 8; ++c) {
+                const int col = c0 + c * 32 + lane;
+                if (col < p.vdim) acc[c] = fmaf(wj, v[col], acc[c]);
+            }
+        }
+    }
+    const float inv = 1.0f / l;
+    float *o = static_cast<float *>(p.d_out_rows) + (size_t)m * p.out_ld + (size_t)h * p.vdim;
+    const float *gate = p.d_gate + (size_t)m * p.proj_ld + (size_t)h * p.vdim;
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+        const int col = c0 + c * 32 + lane;
+        if (col < p.vdim) o[col] = acc[c] * inv * sigmoid_f32(gate[col]);
+    }
+}
+
+// bfloat16 on the tensor cores. A block: 64 query rows of one head, four warps of 16 rows; keys 64 at a time, the
+// next tile's copies in flight under the current one. DV value columns per blockIdx.z.
+constexpr int BQ = 64, BKEY = 64;
+
+__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool on)
+{
+    const int n = on ? 16 : 0;                               // 0: the 16 bytes are zero-filled
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t a, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t a, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
+{
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi)
+{
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t *>(&h);
+}
+
+template <int DV>
+__global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_constant__ b200_latent_args p, int dqs, int stages)
+{
+    // dqs: elements of a query / key row in shared memory; its first dqs - 8 are multiples of 16 and hold
+    // [unrotated | rotated | zeros]. Rows are 16 bytes off a multiple of 32: ldmatrix is conflict-free.
+    constexpr int VS = DV + 8;
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), QS = dim8 + rot8, vd8 = up8(p.vdim), R8 = up8(p.kv_rank), CS = R8 + rot8;
+    const int dqk = dqs - 8;
+    __nv_bfloat16 *qsm = reinterpret_cast<__nv_bfloat16 *>(smem);
+    __nv_bfloat16 *ksm = qsm + (size_t)BQ * dqs;             // [stages][BKEY][dqs]
+    __nv_bfloat16 *vsm = ksm + (size_t)stages * BKEY * dqs;  // [stages][BKEY][VS]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int h = blockIdx.y, m0 = blockIdx.x * BQ, c0 = blockIdx.z * DV;
+    const int rows = min(BQ, p.n_rows - m0);
+    const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(p.d_cache);
+    const __nv_bfloat16 *kv = static_cast<const __nv_bfloat16 *>(p.d_kv) + (size_t)h * (dim8 + vd8);
+    const __nv_bfloat16 *qg = static_cast<const __nv_bfloat16 *>(p.d_q_rows) + ((size_t)m0 * p.heads + h) * QS;
+
+    const int first = p.pos0 + m0, last = first + rows - 1;  // absolute positions of this block's queries
+    const int lo = p.window > 0 && first - p.window + 1 > 0 ? first - p.window + 1 : 0;
+    const int tiles = (last - lo) / BKEY + 1;
+    const int sq = dqk / 8, sv = DV / 8;
+
+    for (int i = tid; i < BQ * sq; i += 128) {
+        const int r = i / sq, c = i % sq;
+        const bool on = r < rows && c * 8 < QS;
+        cp16(smem_u32(qsm + (size_t)r * dqs + c * 8), on ? qg + (size_t)r * p.heads * QS + c * 8 : qg, on);
+    }
+    auto stage = [&](int tile, int slot) {
+        __nv_bfloat16 *kd = ksm + (size_t)slot * BKEY * dqs, *vd = vsm + (size_t)slot * BKEY * VS;
+        const int k0 = lo + tile * BKEY;
+        for (int i = tid; i < BKEY * sq; i += 128) {
+            const int r = i / sq, c = i % sq, kp = k0 + r;
+            const bool on = kp <= last && c * 8 < QS;
+            const __nv_bfloat16 *src = !on ? kv : c * 8 < dim8 ? kv + (size_t)(kp - p.kv_row0) * p.kv_ld + c * 8
+                                                               : cache + (size_t)kp * CS + R8 + (c * 8 - dim8);
+            cp16(smem_u32(kd + (size_t)r * dqs + c * 8), src, on);
+        }
+        for (int i = tid; i < BKEY * sv; i += 128) {
+            const int r = i / sv, c = i % sv, kp = k0 + r;
+            const bool on = kp <= last && c0 + c * 8 < vd8;
+            cp16(smem_u32(vd + (size_t)r * VS + c * 8), on ? kv + (size_t)(kp - p.kv_row0) * p.kv_ld + dim8 + c0 + c * 8 : kv, on);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(0, 0);
+
+    float o[DV / 8][4];
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) o[i][k] = 0.0f;
+    float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+    // this thread's rows: r0 and r0 + 8 of the warp's 16
+    const int r0 = warp * 16 + (lane >> 2);
+    const int qpos[2] = {first + r0, first + r0 + 8};
+    const uint32_t qaddr = smem_u32(qsm + (size_t)(warp * 16 + (lane & 15)) * dqs + (lane >> 4) * 8);
+    const float LOG2E = 1.4426950408889634f;
+    const float sc = p.scale * LOG2E;
+
+    for (int tile = 0; tile < tiles; ++tile) {
+        const int slot = stages == 2 ? tile & 1 : 0;
+        if (stages == 2 && tile + 1 < tiles) {
+            stage(tile + 1, slot ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const __nv_bfloat16 *kd = ksm + (size_t)slot * BKEY * dqs, *vd = vsm + (size_t)slot * BKEY * VS;
+        float s[BKEY / 8][4];
+#pragma unroll
+        for (int i = 0; i < BKEY / 8; ++i)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) s[i][k] = 0.0f;
+        // key rows as the B operand: matrices (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
+        const uint32_t kaddr = smem_u32(kd + (size_t)((lane & 7) + ((lane >> 4) << 3)) * dqs + ((lane >> 3) & 1) * 8);
+        for (int kk = 0; kk < dqk; kk += 16) {
+            uint32_t a[4];
+            ldsm4(qaddr + kk * 2, a);
+#pragma unroll
+            for (int n = 0; n < BKEY / 16; ++n) {
+                uint32_t b[4];
+                ldsm4(kaddr + (uint32_t)(n * 16 * dqs + kk) * 2, b);
+                mma_bf16(s[2 * n], a, b[0], b[1]);
+                mma_bf16(s[2 * n + 1], a, b[2], b[3]);
+            }
+        }
+        const int k0 = lo + tile * BKEY;
+        float mt[2] = {mx[0], mx[1]};
+#pragma unroll
+        for (int n = 0; n < BKEY / 8; ++n)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int kp = k0 + n * 8 + (lane & 3) * 2 + (k & 1), d = qpos[k >> 1] - kp;
+                s[n][k] = d >= 0 && (p.window <= 0 || d < p.window) ? s[n][k] * sc : -INFINITY;
+                mt[k >> 1] = fmaxf(mt[k >> 1], s[n][k]);
+            }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 1));
+            mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 2));
+        }
+        // a row with nothing visible so far keeps its maximum at -inf: its weights and its correction are zero
+        const float base[2] = {mt[0] == -INFINITY ? 0.0f : mt[0], mt[1] == -INFINITY ? 0.0f : mt[1]};
+        const float corr[2] = {exp2f(mx[0] - base[0]), exp2f(mx[1] - base[1])};
+        mx[0] = mt[0]; mx[1] = mt[1];
+        float ls[2] = {0.0f, 0.0f};
+#pragma unroll
+        for (int n = 0; n < BKEY / 8; ++n)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                s[n][k] = exp2f(s[n][k] - base[k >> 1]);
+                ls[k >> 1] += s[n][k];
+            }
+        l[0] = l[0] * corr[0] + ls[0];
+        l[1] = l[1] * corr[1] + ls[1];
+#pragma unroll
+        for (int i = 0; i < DV / 8; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+        // value rows as the B operand, transposed on load: (k 0-7, cols 0-7), (k 8-15, cols 0-7), (k 0-7, cols 8-15), ...
+        const uint32_t vaddr = smem_u32(vd + (size_t)(lane & 15) * VS + (lane >> 4) * 8);
+#pragma unroll
+        for (int kk = 0; kk < BKEY / 16; ++kk) {
+            const uint32_t a[4] = {pack_bf16(s[2 * kk][0], s[2 * kk][1]), pack_bf16(s[2 * kk][2], s[2 * kk][3]),
+                                   pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+#pragma unroll
+            for (int n = 0; n < DV / 16; ++n) {
+                uint32_t b[4];
+                ldsm4_t(vaddr + (uint32_t)(kk * 16 * VS + n * 16) * 2, b);
+                mma_bf16(o[2 * n], a, b[0], b[1]);
+                mma_bf16(o[2 * n + 1], a, b[2], b[3]);
+            }
+        }
+        __syncthreads();                                     // the slot is overwritten by the next round's copies
+        if (stages == 1 && tile + 1 < tiles) stage(tile + 1, 0);
+    }
+
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+        if (r0 + 8 * r >= rows) continue;
+        const float inv = 1.0f / l[r];
+        const size_t m = (size_t)(m0 + r0 + 8 * r);
+        __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(p.d_out_rows) + m * p.out_ld + (size_t)h * p.vdim;
+        const float *gate = p.d_gate + m * p.proj_ld + (size_t)h * p.vdim;
+#pragma unroll
+        for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int col = c0 + i * 8 + (lane & 3) * 2 + k;
+                if (col < p.vdim) out[col] = __float2bfloat16_rn(o[i][2 * r + k] * inv * sigmoid_f32(gate[col]));
+            }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ host side
+
+bool shape_ok(const b200_latent_args *a)
+{
+    return a && (a->wtype == B200_WT_BF16 || a->wtype == B200_WT_F32) && a->heads > 0 && a->dim > 0 && a->rot_dim > 0 && a->vdim > 0 &&
+           a->kv_rank > 0 && a->max_seq > 0 && a->rot_dims >= 0 && a->rot_dims <= a->rot_dim && a->rot_dims % 2 == 0 &&
+           a->d_q && a->d_dkv && a->d_dkv_gamma && a->d_rope && a->d_cache;
+}
+
+template <typename K>
+int launch_pdl(K kern, int gx, int gy, int threads, size_t smem, int pdl, cudaStream_t st, const b200_latent_args &a, int i0)
+{
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(gx, gy);
+    cfg.blockDim = dim3(threads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl ? 1 : 0;
+    ++g_b200_launches;
+    return (int)cudaLaunchKernelEx(&cfg, kern, a, i0);
+}
+
+template <typename K>
+int allow_smem(K kern, size_t smem)
+{
+    if (smem > 227 * 1024) return B200_E_TOOLARGE;
+    return smem > 48 * 1024 ? (int)cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : 0;
+}
+
+template <int WT>
+int decode(const b200_latent_args &a, cudaStream_t st)
+{
+    constexpr int E = Elem<WT>::E;
+    const int dim8 = up8(a.dim), R8 = up8(a.kv_rank), CS = R8 + up8(a.rot_dim);
+    int lpr = 1;
+    while (lpr < 32 && lpr * E < dim8) lpr <<= 1;
+    const int rows_per_block = ABSORB_PASSES * 8 * (32 / lpr);
+    const int chunks = (a.kv_rank + rows_per_block - 1) / rows_per_block;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.heads * chunks + 1);
+    cfg.blockDim = dim3(256);
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = a.use_pdl ? 1 : 0;
+    ++g_b200_launches;
+    int rc = (int)cudaLaunchKernelEx(&cfg, latent_absorb_kernel<WT>, a, chunks, lpr);
+    if (rc) return rc;
+
+    const int row16 = (CS / E) | 1;
+    const size_t smem = (size_t)KT * row16 * 16 + (size_t)HB * CS * 4;
+    const int hb = (a.heads + HB - 1) / HB, nch = (R8 + 32 * E - 1) / (32 * E);
+#define SCORES(N)                                                                             \
+    do {                                                                                      \
+        if ((rc = allow_smem(latent_scores_kernel<WT, N>, smem)) != 0) return rc;              \
+        rc = launch_pdl(latent_scores_kernel<WT, N>, a.n_split, hb, 256, smem, a.use_pdl, st, a, row16); \
+    } while (0)
+    if (nch <= 1) SCORES(1);
+    else if (nch <= 2) SCORES(2);
+    else if (nch <= 4) SCORES(4);
+    else if (nch <= 8) SCORES(8);
+    else return B200_E_TOOLARGE;
+#undef SCORES
+    if (rc) return rc;
+    const int vchunks = (a.vdim + VALUE_ROWS - 1) / VALUE_ROWS;
+    return launch_pdl(latent_value_kernel<WT>, a.heads * vchunks, 1, 256, (size_t)R8 * 4, a.use_pdl, st, a, vchunks);
+}
+
+template <int DV>
+int attend_bf16(const b200_latent_args &a, cudaStream_t st)
+{
+    const int dqk = (up8(a.dim) + up8(a.rot_dim) + 15) / 16 * 16, dqs = dqk + 8;
+    int stages = 2;
+    auto bytes = [&](int s) { return ((size_t)(BQ + s * BKEY) * dqs + (size_t)s * BKEY * (DV + 8)) * 2; };
+    if (bytes(2) > 227 * 1024) stages = 1;
+    int rc = allow_smem(latent_attend_bf16_kernel<DV>, bytes(stages));
+    if (rc) return rc;
+    const dim3 grid((a.n_rows + BQ - 1) / BQ, a.heads, (a.vdim + DV - 1) / DV);
+    latent_attend_bf16_kernel<DV><<<grid, 128, bytes(stages), st>>>(a, dqs, stages);
+    ++g_b200_launches;
+    return (int)cudaGetLastError();
+}
+
+}  // namespace
+
+extern "C" int b200_latent_splits(int heads, int window, int max_seq)
+{
+    if (heads <= 0 || max_seq <= 0) return 1;
+    const int span = window > 0 && window < max_seq ? window : max_seq;
+    const int tiles = (span + KT - 1) / KT, groups = (heads + HB - 1) / HB;
+    int n = 2 * 148 / groups;
+    if (n > tiles) n = tiles;
+    if (n > MAX_SPLITS) n = MAX_SPLITS;
+    return n < 1 ? 1 : n;
+}
+
+extern "C" int b200_latent_decode(const b200_latent_args *a, void *stream)
+{
+    if (!shape_ok(a) || !a->d_gate || !a->d_w_uk_t || !a->d_w_kv || !a->d_qlat || !a->d_part || !a->d_out || !a->d_pos ||
+        a->n_split < 1 || a->n_split > MAX_SPLITS)
+        return B200_E_BADARG;
+    return a->wtype == B200_WT_BF16 ? decode<B200_WT_BF16>(*a, (cudaStream_t)stream) : decode<B200_WT_F32>(*a, (cudaStream_t)stream);
+}
+
+static bool rows_ok(const b200_latent_args *a)
+{
+    return shape_ok(a) && a->n_rows > 0 && a->pos0 >= 0 && a->pos0 + a->n_rows <= a->max_seq && a->proj_ld > 0 && a->d_q_rows;
+}
+
+extern "C" int b200_latent_rows_prep(const b200_latent_args *a, void *stream)
+{
+    if (!rows_ok(a)) return B200_E_BADARG;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (a->wtype == B200_WT_BF16) latent_prep_kernel<B200_WT_BF16><<<a->n_rows, 256, 0, st>>>(*a);
+    else latent_prep_kernel<B200_WT_F32><<<a->n_rows, 256, 0, st>>>(*a);
+    ++g_b200_launches;
+    return (int)cudaGetLastError();
+}
+
+extern "C" int b200_latent_rows_attend(const b200_latent_args *a, void *stream)
+{
+    const int oldest = a && a->window > 0 && a->pos0 - a->window + 1 > 0 ? a->pos0 - a->window + 1 : 0;
+    if (!rows_ok(a) || !a->d_gate || !a->d_kv || !a->d_out_rows || a->kv_row0 < 0 || a->kv_row0 > oldest ||
+        a->kv_ld < (long long)a->heads * (up8(a->dim) + up8(a->vdim)) || a->out_ld < (long long)a->heads * a->vdim)
+        return B200_E_BADARG;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (a->wtype == B200_WT_BF16) {
+        if ((a->kv_ld & 7) || ((uintptr_t)a->d_kv & 15) || ((uintptr_t)a->d_q_rows & 15)) return B200_E_BADARG;
+        if (a->vdim <= 32) return attend_bf16<32>(*a, st);
+        if (a->vdim <= 64) return attend_bf16<64>(*a, st);
+        return attend_bf16<128>(*a, st);
+    }
+    const size_t smem = (size_t)4 * (up8(a->dim) + up8(a->rot_dim)) * 4;
+    int rc = allow_smem(latent_attend_f32_kernel, smem);
+    if (rc) return rc;
+    latent_attend_f32_kernel<<<dim3(a->n_rows, (a->heads + 3) / 4, (a->vdim + 255) / 256), 128, smem, st>>>(*a);
+    ++g_b200_launches;
+    return (int)cudaGetLastError();
+}

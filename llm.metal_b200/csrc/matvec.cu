@@ -19,7 +19,7 @@
 // The math is the reference's q8_matvec / f16_matvec
 // (shaders/q8_kernels.metal:10-42, 97-127): fp32 activations, integer quants
 // converted to fp32, fp32 multiply-accumulate, partial block sums scaled by
-// the binary16 block scale. Input assembly and the epilogues fold in rms_norm
+// the binary16 block scale. BF16 and F32 weights have no counterpart there. Input assembly and the epilogues fold in rms_norm
 // (:133-157), residual_add (:369-375), silu_mul / gelu_mul (:337-363), the
 // embedding copy (src/nn/fast_inference.c:386-392) and argmax (:469-476).
 #include "stream_core.cuh"
@@ -49,11 +49,37 @@ struct Geometry {
 };
 
 // blockDim.x = NG*T consumers + 32 producer threads.
+// RMS norm of the vector a group of T threads holds, `groups` equal consecutive parts of its first `dim` elements
+// each by its own mean square. In place; one part after the other, so the sums are in a fixed order.
+template <int SPT, int E>
+__device__ __forceinline__ void norm_parts(float (&x)[SPT][E], const int (&col)[SPT], const float (&gamma)[SPT][E], int dim,
+                                           int groups, float eps, float *gred, int bar_id, int T, int t)
+{
+    const int len = dim / groups;
+    for (int k = 0; k < groups; ++k) {
+        const int lo = k * len, hi = lo + len;
+        float ss = 0.0f;
+#pragma unroll
+        for (int s = 0; s < SPT; ++s)
+#pragma unroll
+            for (int e = 0; e < E; ++e)
+                if (col[s] + e >= lo && col[s] + e < hi) ss = fmaf(x[s][e], x[s][e], ss);
+        ss = group_sum(ss, gred, bar_id, T, t);
+        const float inv = 1.0f / sqrtf(ss / (float)len + eps);
+#pragma unroll
+        for (int s = 0; s < SPT; ++s)
+#pragma unroll
+            for (int e = 0; e < E; ++e)
+                if (col[s] + e >= lo && col[s] + e < hi) x[s][e] = gamma[s][e] * (x[s][e] * inv);
+    }
+}
+
 template <int WT, int SPT, int RB, int MAXT>
 __global__ void __launch_bounds__(MAXT)
 matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
 {
-    constexpr int E = (WT == B200_WT_Q8) ? 16 : 8;       // elements per 16-byte slice
+    constexpr int E = (WT == B200_WT_Q8) ? 16 : (WT == B200_WT_F32) ? 4 : 8;       // elements per 16-byte slice
+    constexpr bool EXT = WT == B200_WT_BF16 || WT == B200_WT_F32;   // post-norm inputs, gated outputs, depth sums
     extern __shared__ __align__(128) unsigned char smem_raw[];
     const int T = geo.T, NG = geo.NG, nstage = geo.nstage, nwg = T >> 5, nC = NG * T;
     unsigned char *ring = smem_raw;
@@ -99,6 +125,17 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                 mbar_expect_tx(&full[slot], bytes);
                 bulk_load(ring + (size_t)slot * geo.slot_bytes, wbase + (long long)row0 * p.row_stride, bytes, &full[slot]);
             }
+        } else if constexpr (EXT) {
+            // the producer warp's other lanes form the depth sums of this block's rows
+            if (p.hist_n > 0) {
+                pdl_wait();
+                for (int row = r0 + (tid - nC - 1); row < r1; row += 31) {
+                    float a = 0.0f;
+#pragma unroll 8
+                    for (int j = 0; j < p.hist_n; ++j) a = fmaf(p.d_hist_coef[j], p.d_hist[(long long)j * p.hist_stride + row], a);
+                    p.d_hist_out[row] = a;
+                }
+            }
         }
         return;
     }
@@ -125,6 +162,19 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
             }
     }
 
+    float gp[EXT ? SPT : 1][E];                  // the same for the norm of a post-norm input
+    if constexpr (EXT) {
+        if (p.in_mode == B200_IN_POSTNORM && (!geo.share_x || g == 0)) {
+#pragma unroll
+            for (int s = 0; s < SPT; ++s)
+#pragma unroll
+                for (int e = 0; e < E; e += 4) {
+                    const float4 v4 = on[s] ? *reinterpret_cast<const float4 *>(p.d_slot_norm_gamma + col[s] + e) : make_float4(0, 0, 0, 0);
+                    gp[s][e] = v4.x; gp[s][e + 1] = v4.y; gp[s][e + 2] = v4.z; gp[s][e + 3] = v4.w;
+                }
+        }
+    }
+
     pdl_wait();
 
     // Tensor parallel: every rank's partial vector must have landed in `slots`
@@ -144,7 +194,7 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
     // SMs at once, and every extra reader of the same L2 lines queues behind the others.
     float x[SPT][E];
     if (!geo.share_x || g == 0) {
-    if (p.in_mode == B200_IN_VEC) {
+    if (p.in_mode == B200_IN_VEC || (EXT && p.in_mode == B200_IN_POSTNORM)) {
 #pragma unroll
         for (int s = 0; s < SPT; ++s)
 #pragma unroll
@@ -152,6 +202,35 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                 float4 v4 = on[s] ? *reinterpret_cast<const float4 *>(p.d_in_vec + col[s] + e) : make_float4(0, 0, 0, 0);
                 x[s][e] = v4.x; x[s][e + 1] = v4.y; x[s][e + 2] = v4.z; x[s][e + 3] = v4.w;
             }
+        if constexpr (EXT) {
+            if (p.in_mode == B200_IN_POSTNORM) {
+                float mix[SPT][E];                       // fetched before the norm's reductions
+#pragma unroll
+                for (int s = 0; s < SPT; ++s)
+#pragma unroll
+                    for (int e = 0; e < E; e += 4) {
+                        const float4 v4 = on[s] && p.d_mix_in ? *reinterpret_cast<const float4 *>(p.d_mix_in + col[s] + e) : make_float4(0, 0, 0, 0);
+                        mix[s][e] = v4.x; mix[s][e + 1] = v4.y; mix[s][e + 2] = v4.z; mix[s][e + 3] = v4.w;
+                    }
+                const float coef = p.d_mix_in ? *p.d_mix_coef : 1.0f;
+                norm_parts<SPT, E>(x, col, gp, p.norm_dim > 0 ? p.norm_dim : p.cols, p.norm_groups > 1 ? p.norm_groups : 1, p.eps,
+                                   gred, 2 + g, T, t);
+                const bool store = blockIdx.x == 0 && g == 0;
+#pragma unroll
+                for (int s = 0; s < SPT; ++s)
+#pragma unroll
+                    for (int e = 0; e < E; e += 4) {
+                        if (store && on[s] && p.d_post_copy)
+                            *reinterpret_cast<float4 *>(p.d_post_copy + col[s] + e) = make_float4(x[s][e], x[s][e + 1], x[s][e + 2], x[s][e + 3]);
+                        if (p.d_mix_in) {
+#pragma unroll
+                            for (int k = 0; k < 4; ++k) x[s][e + k] = fmaf(coef, x[s][e + k], mix[s][e + k]);
+                        }
+                        if (store && on[s] && p.d_resid_out)
+                            *reinterpret_cast<float4 *>(p.d_resid_out + col[s] + e) = make_float4(x[s][e], x[s][e + 1], x[s][e + 2], x[s][e + 3]);
+                    }
+            }
+        }
     } else {
         if (p.in_mode == B200_IN_EMBED) {
             long long tok = p.d_tokens[*p.d_pos];
@@ -217,7 +296,10 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                             make_float4(x[s][e], x[s][e + 1], x[s][e + 2], x[s][e + 3]);
         }
     }
-    if (p.d_norm_gamma) {
+    if (EXT && p.d_norm_gamma) {
+        if constexpr (EXT)
+            norm_parts<SPT, E>(x, col, gm, p.norm_dim > 0 ? p.norm_dim : p.cols, p.norm_groups > 1 ? p.norm_groups : 1, p.eps, gred, 2 + g, T, t);
+    } else if (p.d_norm_gamma) {
         float ss = 0.0f;
 #pragma unroll
         for (int s = 0; s < SPT; ++s)
@@ -268,16 +350,23 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
 #pragma unroll
     for (int s = 0; s < SPT; ++s) {
         const int c = on[s] ? col[s] : 0;
-        qoff[s] = (uint32_t)(WT == B200_WT_Q8 ? c : 2 * c);
+        qoff[s] = (uint32_t)(WT == B200_WT_Q8 ? c : WT == B200_WT_F32 ? 4 * c : 2 * c);
         soff[s] = (uint32_t)p.cols + (uint32_t)(c >> 5) * 2u;   // Q8: scales follow the quants of a row
     }
     const uint32_t ring_s = smem_u32(ring), stride = (uint32_t)p.row_stride;
     for (int i = g, it = 0; i < nst; i += NG, ++it) {
         const int slot = i % nstage;
-        if (!mbar_wait(&full[slot], (i / nstage) & 1) && p.d_err) *p.d_err = 3;
-        const uint32_t sb = ring_s + (uint32_t)slot * geo.slot_bytes;
         const int row0 = r0 + i * RB;
         const int nr = min(RB, r1 - row0);
+        float o_resid = 0.0f, o_gate = 0.0f;            // what the gated output adds to and scales by
+        if constexpr (EXT) {
+            if (p.out_mode == B200_OUT_GATED && wg == 0 && lane < nr) {
+                o_resid = p.d_out_resid[row0 + lane];
+                o_gate = p.d_out_gate[row0 + lane] + p.d_out_gate_bias[row0 + lane];
+            }
+        }
+        if (!mbar_wait(&full[slot], (i / nstage) & 1) && p.d_err) *p.d_err = 3;
+        const uint32_t sb = ring_s + (uint32_t)slot * geo.slot_bytes;
         // Rows past nr hold stale bytes; they are computed like the others (no predicates in the
         // hot loop), stay in their own reduction lane and are never emitted.
         uint4 wq[RB][SPT];
@@ -297,6 +386,8 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
             for (int s = 0; s < SPT; ++s) {
                 float d;
                 if (WT == B200_WT_Q8) d = __half2float(__ushort_as_half((unsigned short)ws[j][s])) * dot16_q8(wq[j][s], x[s]);
+                else if (WT == B200_WT_BF16) d = dot8_bf16(wq[j][s], x[s]);
+                else if (WT == B200_WT_F32) d = dot4_f32(wq[j][s], x[s]);
                 else d = dot8_f16(wq[j][s], x[s]);
                 acc += d;                      // threads past the end of the row hold a zero input slice
             }
@@ -315,11 +406,16 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
             const int row = row0 + lane;
             if (p.out_mode == B200_OUT_GLU) {
                 const float u = __shfl_down_sync(0xffffffffu, y, 1);
-                if (lane < nr && !(lane & 1)) {
+                if (EXT && p.glu_rows > 0 && row >= p.glu_rows) {
+                    if (lane < nr) p.d_out2[row - p.glu_rows] = y;
+                } else if (lane < nr && !(lane & 1)) {
                     const float a = p.act == 0 ? act_silu(y) : act_gelu_tanh(y);
                     p.d_out[0][p.out_offset + (row >> 1)] = a * u;
                 }
+            } else if (EXT && p.out_mode == B200_OUT_GATED) {
+                if (lane < nr) p.d_out[0][p.out_offset + row] = fmaf(p.resid_alpha, o_resid, sigmoid_f32(o_gate) * y);
             } else if (lane < nr) {
+                if (EXT && p.softcap > 0.0f) y = p.softcap * tanhf(y / p.softcap);
                 for (int q = 0; q < p.n_out; ++q) p.d_out[q][p.out_offset + row] = y;
                 if (better(y, row, best_v, best_i)) { best_v = y; best_i = row; }
             }
@@ -415,7 +511,7 @@ int launch(const b200_matvec_args &a, const Geometry &geo, int grid, cudaStream_
     const int nwg = geo.T / 32;
     const size_t smem = (size_t)geo.nstage * geo.slot_bytes + (size_t)geo.nstage * 16 +
                         ((size_t)geo.NG * 2 * nwg * RB + (size_t)geo.NG * 32 + (size_t)geo.NG * RB * 2) * sizeof(float) +
-                        (geo.share_x ? (size_t)SPT * geo.T * (WT == B200_WT_Q8 ? 16 : 8) * sizeof(float) : 0);
+                        (geo.share_x ? (size_t)SPT * geo.T * (WT == B200_WT_Q8 ? 16 : WT == B200_WT_F32 ? 4 : 8) * sizeof(float) : 0);
     auto kern = matvec_kernel<WT, SPT, RB, MAXT>;
     if (smem > 220 * 1024) return B200_E_TOOLARGE;
     if (smem > 48 * 1024) {
@@ -462,14 +558,24 @@ extern "C" int b200_matvec(const b200_matvec_args *ap, void *stream)
     if (!ap) return B200_E_BADARG;
     const b200_matvec_args &a = *ap;
     if (!a.d_w || a.rows <= 0 || a.cols <= 0 || (a.row_stride % 16) || ((uintptr_t)a.d_w % 16)) return B200_E_BADARG;
-    if (a.wtype != B200_WT_Q8 && a.wtype != B200_WT_F16) return B200_E_BADARG;
+    if (a.wtype < B200_WT_Q8 || a.wtype > B200_WT_F32) return B200_E_BADARG;
+    const bool ext = a.wtype == B200_WT_BF16 || a.wtype == B200_WT_F32;
     if (a.wtype == B200_WT_Q8 ? (a.cols % 32) : (a.cols % 8)) return B200_E_BADARG;
     if (a.row_stride < (long long)b200_packed_row_stride(a.wtype, a.cols)) return B200_E_BADARG;
     if (a.in_mode == B200_IN_VEC ? !a.d_in_vec
         : a.in_mode == B200_IN_RESID ? (!a.d_resid_in || a.n_slots < 0 || (a.n_slots > 0 && !a.d_slots))
+        : a.in_mode == B200_IN_POSTNORM ? (!ext || !a.d_in_vec || !a.d_slot_norm_gamma || (a.d_mix_in && !a.d_mix_coef))
         : a.in_mode == B200_IN_EMBED ? (!a.d_emb || !a.d_tokens || !a.d_pos || a.emb_rows <= 0) : true)
         return B200_E_BADARG;
-    if (a.out_mode == B200_OUT_GLU ? (a.rows % 2 || !a.d_out[0]) : (a.out_mode != B200_OUT_STORE || a.n_out < 1 || a.n_out > B200_MAX_PEERS))
+    if (!ext && (a.out_mode == B200_OUT_GATED || a.norm_dim || a.norm_groups || a.hist_n || a.glu_rows || a.softcap != 0.0f)) return B200_E_BADARG;
+    if (ext && (a.norm_dim < 0 || a.norm_dim > a.cols || a.norm_groups < 0 ||
+                (a.norm_groups > 1 && (a.norm_dim > 0 ? a.norm_dim : a.cols) % a.norm_groups) ||
+                a.hist_n < 0 || (a.hist_n > 0 && (!a.d_hist || !a.d_hist_coef || !a.d_hist_out)) ||
+                (a.glu_rows && (a.out_mode != B200_OUT_GLU || a.glu_rows < 0 || a.glu_rows % 2 || a.glu_rows > a.rows || !a.d_out2)) ||
+                (a.in_mode == B200_IN_RESID && a.d_slot_norm_gamma)))
+        return B200_E_BADARG;
+    if (a.out_mode == B200_OUT_GATED ? (!a.d_out[0] || !a.d_out_resid || !a.d_out_gate || !a.d_out_gate_bias)
+        : a.out_mode == B200_OUT_GLU ? (a.rows % 2 || !a.d_out[0]) : (a.out_mode != B200_OUT_STORE || a.n_out < 1 || a.n_out > B200_MAX_PEERS))
         return B200_E_BADARG;
     if (a.n_wait < 0 || a.n_wait > B200_MAX_PEERS || a.n_signal < 0 || a.n_signal > B200_MAX_PEERS ||
         a.n_argmax_out < 0 || a.n_argmax_out > B200_MAX_PEERS)
@@ -482,12 +588,12 @@ extern "C" int b200_matvec(const b200_matvec_args *ap, void *stream)
     if (a.advance_epoch && (!a.d_epoch || !a.d_epoch_rw)) return B200_E_BADARG;
     if (a.d_argmax_scratch && a.out_mode != B200_OUT_STORE) return B200_E_BADARG;
 
-    const int E = a.wtype == B200_WT_Q8 ? 16 : 8;
+    const int E = a.wtype == B200_WT_Q8 ? 16 : a.wtype == B200_WT_F32 ? 4 : 8;
     const int nsl = (a.cols + E - 1) / E;
     // Up to two slices per thread: keeps a group at <= 320 threads for rows of up to 640 slices, so that
     // two blocks (this kernel's and the next one's) fit on an SM; 960 consumers + the producer warp at most.
     // Measured on the 2560 x 9728 down projection: two slices per thread 12.3 us, one slice 16.3 us.
-    const int spt = nsl <= 320 ? 1 : 2;
+    const int spt = nsl <= 320 ? 1 : a.wtype == B200_WT_F32 && nsl > 1920 ? 4 : 2;
     if ((nsl + spt - 1) / spt > 960) return B200_E_TOOLARGE;
     Geometry geo;
     geo.T = (((nsl + spt - 1) / spt) + 31) / 32 * 32;
@@ -519,5 +625,10 @@ extern "C" int b200_matvec(const b200_matvec_args *ap, void *stream)
     cudaStream_t st = (cudaStream_t)stream;
     if (a.wtype == B200_WT_Q8)
         return spt == 1 ? launch_by_rows<B200_WT_Q8, 1>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_Q8, 2>(a, geo, rb, grid, st);
+    if (a.wtype == B200_WT_BF16)
+        return spt == 1 ? launch_by_rows<B200_WT_BF16, 1>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_BF16, 2>(a, geo, rb, grid, st);
+    if (a.wtype == B200_WT_F32)
+        return spt == 1 ? launch_by_rows<B200_WT_F32, 1>(a, geo, rb, grid, st) : spt == 2 ? launch_by_rows<B200_WT_F32, 2>(a, geo, rb, grid, st)
+                                                                                         : launch_by_rows<B200_WT_F32, 4>(a, geo, rb, grid, st);
     return spt == 1 ? launch_by_rows<B200_WT_F16, 1>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_F16, 2>(a, geo, rb, grid, st);
 }

@@ -11,6 +11,8 @@
 #include "common.cuh"
 #include "../../include/llmb200_kernels.h"
 
+#include <cuda_bf16.h>
+
 extern unsigned long long g_b200_launches;
 
 __global__ void __launch_bounds__(256)
@@ -79,6 +81,22 @@ f16_pack_kernel(const float *__restrict__ src, long long ld, int rows, int cols,
     }
 }
 
+// One thread per destination element, padding columns included.
+template <typename T>
+__global__ void __launch_bounds__(256)
+cast_pack_kernel(const float *__restrict__ src, long long ld, int rows, int cols,
+                 uint8_t *__restrict__ dst, long long dst_stride, int dst_row0, int dst_row_step)
+{
+    const int padded = (int)(dst_stride / (long long)sizeof(T));
+    const long long total = (long long)rows * padded;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total;
+         i += (long long)gridDim.x * blockDim.x) {
+        const int r = (int)(i / padded), c = (int)(i % padded);
+        T *row = reinterpret_cast<T *>(dst + (long long)(dst_row0 + (long long)r * dst_row_step) * dst_stride);
+        row[c] = (T)(c < cols ? src[(long long)r * ld + c] : 0.0f);
+    }
+}
+
 // One thread per block: 34 bytes out, written bytewise (the canonical stream is
 // only 2-byte aligned).
 __global__ void __launch_bounds__(256)
@@ -108,7 +126,7 @@ static int grid_for(long long total) {
 
 extern "C" size_t b200_packed_row_stride(int wtype, int cols)
 {
-    size_t raw = wtype == B200_WT_Q8 ? (size_t)(cols / 32) * 34 : (size_t)cols * 2;
+    size_t raw = wtype == B200_WT_Q8 ? (size_t)(cols / 32) * 34 : (size_t)cols * (wtype == B200_WT_F32 ? 4 : 2);
     return (raw + 15) & ~(size_t)15;
 }
 
@@ -140,6 +158,24 @@ extern "C" int b200_f16_pack(const float *d_src, long long ld, int rows, int col
     const long long total = (long long)rows * (cols / 4);
     f16_pack_kernel<<<grid_for(total), 256, 0, (cudaStream_t)stream>>>(
         d_src, ld, rows, cols, (uint8_t *)d_dst, dst_row_stride, dst_row0, dst_row_step);
+    ++g_b200_launches;
+    return (int)cudaGetLastError();
+}
+
+extern "C" int b200_cast_pack(int wtype, const float *d_src, long long ld, int rows, int cols,
+                              void *d_dst, long long dst_row_stride, int dst_row0, int dst_row_step, void *stream)
+{
+    if (!d_src || !d_dst || rows < 0 || cols <= 0 || ld < cols || (wtype != B200_WT_BF16 && wtype != B200_WT_F32) ||
+        dst_row_stride < (long long)b200_packed_row_stride(wtype, cols) || (dst_row_stride % 16) || ((uintptr_t)d_dst % 16))
+        return B200_E_BADARG;
+    if (rows == 0) return 0;
+    const int g = grid_for((long long)rows * (dst_row_stride / (wtype == B200_WT_F32 ? 4 : 2)));
+    if (wtype == B200_WT_BF16)
+        cast_pack_kernel<__nv_bfloat16><<<g, 256, 0, (cudaStream_t)stream>>>(d_src, ld, rows, cols, (uint8_t *)d_dst, dst_row_stride,
+                                                                            dst_row0, dst_row_step);
+    else
+        cast_pack_kernel<float><<<g, 256, 0, (cudaStream_t)stream>>>(d_src, ld, rows, cols, (uint8_t *)d_dst, dst_row_stride,
+                                                                     dst_row0, dst_row_step);
     ++g_b200_launches;
     return (int)cudaGetLastError();
 }

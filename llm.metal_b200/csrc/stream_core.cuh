@@ -103,6 +103,31 @@ __device__ __forceinline__ float dot8_f16(const uint4 &w, const float *x)
     return a.x + a.y;
 }
 
+// bfloat16 is the upper half of an fp32: the low element of a word moves up, the high one is masked.
+__device__ __forceinline__ float2 bf16_pair(uint32_t w)
+{
+    return make_float2(__uint_as_float(w << 16), __uint_as_float(w & 0xffff0000u));
+}
+
+__device__ __forceinline__ float dot8_bf16(const uint4 &w, const float *x)
+{
+    const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+    float2 a = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) a = __ffma2_rn(bf16_pair(u[i]), make_float2(x[2 * i], x[2 * i + 1]), a);
+    return a.x + a.y;
+}
+
+__device__ __forceinline__ float dot4_f32(const uint4 &w, const float *x)
+{
+    float2 a = make_float2(__uint_as_float(w.x) * x[0], __uint_as_float(w.y) * x[1]);
+    a = __ffma2_rn(make_float2(__uint_as_float(w.z), __uint_as_float(w.w)), make_float2(x[2], x[3]), a);
+    return a.x + a.y;
+}
+
+// The logistic function with the accurate exponential (gates whose values are kept in 32-bit).
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+
 // exp through ex2.approx (2 ulp), what the shader's fast-math exp is (q8_kernels.metal:336)
 __device__ __forceinline__ float act_silu(float g) { return g / (1.0f + __expf(-g)); }
 __device__ __forceinline__ float act_gelu_tanh(float g)

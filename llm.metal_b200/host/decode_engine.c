@@ -27,9 +27,7 @@
  * rank order -- the all-reduce is the epilogue of one kernel and the prologue
  * of the next.
  */
-#include "internal.h"
-#include "../../include/llmb200_inference.h"
-#include "../../include/llmb200_sft.h"
+#include "engine.h"
 
 #include <math.h>
 #include <pthread.h>
@@ -38,86 +36,9 @@
 #include <sys/stat.h>
 #include <time.h>
 
-typedef struct { void *w; long long stride; int rows, cols; } PackedMat;
-
-typedef struct {
-    PackedMat qkv, o, gateup, down;
-    float *g_input, *g_post_attn, *g_pre_ff, *g_post_ff, *g_qn, *g_kn;
-    float *inv_freq;
-    float rope_theta;
-    const float *rope;       /* this layer's table in InferenceState.rope_tab (whole-token kernel) */
-    void *k_cache, *v_cache;
-    int loaded;
-} Layer;
-
-enum { K_QKV = 0, K_ATTN, K_O, K_GATEUP, K_DOWN, K_LM, K_KINDS };
-
-struct InferenceState {
-    int D, Hq, Hkv, hd, IS, V, L, max_seq, use_fp16, wtype;
-    ModelType mt;
-    int tp_rank, tp_size, Hq_l, Hkv_l, IS_l, V_l;
-    float emb_scale;
-    int eos[4], n_eos;
-
-    Layer *layers;
-    PackedMat lm;
-    float *g_final, *emb;
-    int finished;
-    unsigned long long weight_bytes;
-
-    /* activations and scratch (device) */
-    float *resid[2], *qkv, *attn_out, *act, *attn_scratch, *am_scratch;
-    unsigned *attn_tickets, *mv_ticket;
-    int n_split;
-
-    /* control words (device): pos, prompt_len, err, epoch, tokens[max_seq+2] */
-    int *d_pos, *d_prompt_len, *d_err, *d_tokens;
-    unsigned *d_epoch;
-
-    /* all-reduce region, shared with the peers */
-    char *comm;
-    size_t comm_bytes, off_slots_o, off_slots_dn, off_flags, off_am_val, off_am_idx, off_logits;
-    char *peer[B200_MAX_PEERS];
-    int connected, loopback;
-    /* single-process tensor parallelism (LLMB200_TP=k): the handle a caller holds is rank 0's state */
-    int group_n, group_dev[B200_MAX_PEERS], local_peers;
-    struct InferenceState *group[B200_MAX_PEERS];
-
-    /* host side */
-    float *h_logits;
-    int *h_tok;              /* pinned ring for generated ids */
-    int *h_ctl;              /* pinned staging for control writes */
-    cudaEvent_t tok_ev[4];
-    cudaEvent_t ev_a, ev_b;
-    cudaGraphExec_t g_full, g_nolm;
-    int kernels_full, kernels_nolm;   /* kernel nodes per graph */
-    int use_pdl;
-    /* LoRA adapter attached with inference_state_set_lora: device pointers into the SFT state's vectors */
-    struct { const float *A_q, *B_q, *A_v, *B_v; } *lora;
-    int lora_rank;
-    float lora_scaling;
-    SFTState *sft_src;                    /* the SFT state whose matrices this state copied, or NULL */
-    unsigned long long sft_version;       /* its weights_version at the time of the copy */
-    float *xnorm;            /* [D]: the normalised layer input, kept by the q/k/v matvec for the LoRA kernel */
-    int cur_len;
-    double last_decode_ms, last_prefill_ms;
-    int last_n_decoded;
-
-    /* instrumentation */
-    cudaEvent_t *prof_ev;
-    int prof_n, prof_cap, prof_on;
-    /* whole-token kernel: layer table on the device, flagged hand-over vectors, launch arguments */
-    b200_token_layer *d_tk_layers;
-    float *rope_tab[8];      /* rotation tables, one per distinct RoPE base */
-    int n_rope_tab;
-    b200_flagged *fl_qkv, *fl_part, *fl_attn, *fl_act, *fl_am;
-    size_t off_fl_slots_o, off_fl_slots_dn, off_fl_am, off_counters;
-    b200_token_args tk;              /* planned arguments; with_lm is set per launch */
-    int fused, tk_planned, n_sm;
-    unsigned long long *d_step_ns;   /* stage trace of the whole-token kernel (LLMB200_TRACE=1) */
-    int only_kind;           /* >= 0: enqueue_token launches only this kind of kernel (timing loops) */
-    int *prof_kind;
-};
+static int enqueue_token(InferenceState *s, int with_lm, int pdl);
+/* Qwen3 and Gemma3: one token at a time, prompts included (as the reference's engine) */
+static const ModelOps per_token_ops = { .enqueue_token = enqueue_token, .whole_token = 1 };
 
 /* per host thread: the ranks of a single-process group are threads */
 static __thread int g_tp_rank = -1, g_tp_size = -1;
@@ -129,7 +50,7 @@ int llmb200_set_tp(int rank, int world)
     return 0;
 }
 
-static void tp_from_env(int *rank, int *world)
+void llmb200_engine_tp(int *rank, int *world)
 {
     *rank = 0; *world = 1;
     if (g_tp_size > 0) { *rank = g_tp_rank; *world = g_tp_size; return; }
@@ -158,7 +79,7 @@ static int alloc_mat(PackedMat *m, int wtype, int rows, int cols)
     return 0;
 }
 
-static float *dev_zero(size_t bytes)
+float *llmb200_dev_zero(size_t bytes)
 {
     void *p = NULL;
     CU_TRY(cudaMalloc(&p, bytes ? bytes : 4), return NULL);
@@ -186,13 +107,14 @@ InferenceState *llmb200_state_begin(const llmb200_config *c)
     if (!s) { fast_metal_shutdown(); return NULL; }
     s->D = c->d_model; s->Hq = c->n_q_heads; s->Hkv = c->n_kv_heads; s->hd = c->head_dim;
     s->IS = c->intermediate_size; s->V = c->vocab_size; s->L = c->n_layers; s->max_seq = max_seq;
+    s->ops = &per_token_ops;
     s->use_fp16 = c->use_fp16 ? 1 : 0;
     s->wtype = s->use_fp16 ? B200_WT_F16 : B200_WT_Q8;
     s->mt = c->model_type == MODEL_GEMMA3 ? MODEL_GEMMA3 : MODEL_QWEN3;
     s->emb_scale = s->mt == MODEL_GEMMA3 ? sqrtf((float)s->D) : 1.0f;
     if (s->mt == MODEL_GEMMA3) { s->eos[0] = 1; s->eos[1] = 106; s->n_eos = 2; }
     else { s->eos[0] = 151645; s->eos[1] = 151643; s->n_eos = 2; }
-    tp_from_env(&s->tp_rank, &s->tp_size);
+    llmb200_engine_tp(&s->tp_rank, &s->tp_size);
     const int k = s->tp_size;
     const int align = s->wtype == B200_WT_Q8 ? 32 : 8;
     if (s->Hkv % k || s->Hq % k || s->IS % k || s->V % k || (s->IS / k) % align || (s->Hq / k * s->hd) % align ||
@@ -214,8 +136,8 @@ InferenceState *llmb200_state_begin(const llmb200_config *c)
         if (alloc_mat(&ly->qkv, s->wtype, qkv_rows, s->D) || alloc_mat(&ly->o, s->wtype, s->D, s->Hq_l * s->hd) ||
             alloc_mat(&ly->gateup, s->wtype, 2 * s->IS_l, s->D) || alloc_mat(&ly->down, s->wtype, s->D, s->IS_l))
             goto fail;
-        ly->k_cache = dev_zero(cache_bytes);
-        ly->v_cache = dev_zero(cache_bytes);
+        ly->k_cache = llmb200_dev_zero(cache_bytes);
+        ly->v_cache = llmb200_dev_zero(cache_bytes);
         if (!ly->k_cache || !ly->v_cache) goto fail;
         s->weight_bytes += (unsigned long long)ly->qkv.stride * ly->qkv.rows + (unsigned long long)ly->o.stride * ly->o.rows +
                            (unsigned long long)ly->gateup.stride * ly->gateup.rows + (unsigned long long)ly->down.stride * ly->down.rows;
@@ -238,19 +160,28 @@ InferenceState *llmb200_state_begin(const llmb200_config *c)
     if (s->n_split > (max_seq + 31) / 32) s->n_split = (max_seq + 31) / 32;    /* at least 32 cache rows per split */
     if (s->n_split < 1) s->n_split = 1;
 
-    s->resid[0] = dev_zero((size_t)s->D * 4);
-    s->resid[1] = dev_zero((size_t)s->D * 4);
-    s->qkv = dev_zero((size_t)qkv_rows * 4);
-    s->attn_out = dev_zero((size_t)s->Hq_l * s->hd * 4);
-    s->act = dev_zero((size_t)s->IS_l * 4);
-    s->attn_scratch = dev_zero(b200_attn_scratch_floats(s->Hq_l, s->hd, s->n_split) * 4);
-    s->am_scratch = dev_zero((size_t)2 * s->n_sm * 32 * 4);
-    s->attn_tickets = (unsigned *)dev_zero((size_t)s->Hkv_l * 4);
-    s->mv_ticket = (unsigned *)dev_zero(4);
-    int *ctl = (int *)dev_zero((size_t)(8 + max_seq + 2) * 4);
-    if (!s->resid[0] || !s->resid[1] || !s->qkv || !s->attn_out || !s->act || !s->attn_scratch || !s->am_scratch ||
-        !s->attn_tickets || !s->mv_ticket || !ctl)
-        goto fail;
+    s->resid[0] = llmb200_dev_zero((size_t)s->D * 4);
+    s->resid[1] = llmb200_dev_zero((size_t)s->D * 4);
+    s->qkv = llmb200_dev_zero((size_t)qkv_rows * 4);
+    s->attn_out = llmb200_dev_zero((size_t)s->Hq_l * s->hd * 4);
+    s->act = llmb200_dev_zero((size_t)s->IS_l * 4);
+    s->attn_scratch = llmb200_dev_zero(b200_attn_scratch_floats(s->Hq_l, s->hd, s->n_split) * 4);
+    s->attn_tickets = (unsigned *)llmb200_dev_zero((size_t)s->Hkv_l * 4);
+    if (!s->resid[0] || !s->resid[1] || !s->qkv || !s->attn_out || !s->act || !s->attn_scratch || !s->attn_tickets) goto fail;
+    if (llmb200_engine_common(s) != 0) goto fail;
+    return s;
+fail:
+    inference_state_free(s);
+    return NULL;
+}
+
+int llmb200_engine_common(InferenceState *s)
+{
+    const int max_seq = s->max_seq;
+    s->am_scratch = llmb200_dev_zero((size_t)2 * s->n_sm * 32 * 4);
+    s->mv_ticket = (unsigned *)llmb200_dev_zero(4);
+    int *ctl = (int *)llmb200_dev_zero((size_t)(8 + max_seq + 2) * 4);
+    if (!s->am_scratch || !s->mv_ticket || !ctl) { cudaFree(ctl); return -1; }
     s->d_pos = ctl; s->d_prompt_len = ctl + 1; s->d_err = ctl + 2; s->d_epoch = (unsigned *)(ctl + 3);
     s->d_tokens = ctl + 8;
 
@@ -268,23 +199,20 @@ InferenceState *llmb200_state_begin(const llmb200_config *c)
     s->off_fl_am = off;       off += 256;
     s->off_counters = off;    off += (size_t)72 * B200_CNT_STRIDE * 4;   /* arrival counters, one 128-byte line each */
     s->comm_bytes = off;
-    s->comm = (char *)dev_zero(off);
-    if (!s->comm) goto fail;
+    s->comm = (char *)llmb200_dev_zero(off);
+    if (!s->comm) return -1;
     s->peer[s->tp_rank] = s->comm;
-    s->connected = (k == 1);
+    s->connected = (s->tp_size == 1);
 
-    CU_TRY(cudaMallocHost((void **)&s->h_logits, (size_t)s->V * 4), goto fail);
-    CU_TRY(cudaMallocHost((void **)&s->h_tok, 256), goto fail);    /* [0]: the first id; [8 ..]: four groups of ids read back */
-    CU_TRY(cudaMallocHost((void **)&s->h_ctl, (size_t)(8 + max_seq + 2) * 4), goto fail);
-    for (int i = 0; i < 4; ++i) CU_TRY(cudaEventCreateWithFlags(&s->tok_ev[i], cudaEventDisableTiming), goto fail);
-    CU_TRY(cudaEventCreate(&s->ev_a), goto fail);
-    CU_TRY(cudaEventCreate(&s->ev_b), goto fail);
+    CU_TRY(cudaMallocHost((void **)&s->h_logits, (size_t)s->V * 4), return -1);
+    CU_TRY(cudaMallocHost((void **)&s->h_tok, 256), return -1);    /* [0]: the first id; [8 ..]: four groups of ids read back */
+    CU_TRY(cudaMallocHost((void **)&s->h_ctl, (size_t)(8 + max_seq + 2) * 4), return -1);
+    for (int i = 0; i < 4; ++i) CU_TRY(cudaEventCreateWithFlags(&s->tok_ev[i], cudaEventDisableTiming), return -1);
+    CU_TRY(cudaEventCreate(&s->ev_a), return -1);
+    CU_TRY(cudaEventCreate(&s->ev_b), return -1);
     s->use_pdl = getenv("LLMB200_NO_PDL") ? 0 : 1;
     s->only_kind = -1;
-    return s;
-fail:
-    inference_state_free(s);
-    return NULL;
+    return 0;
 }
 
 /* ------------------------------------------------------------ weights */
@@ -369,7 +297,7 @@ int llmb200_state_finish(InferenceState *s, const float *lm_head, const float *f
 
 /* ------------------------------------------------------------ one token */
 
-static void prof_mark(InferenceState *s, int kind)
+void llmb200_prof_mark(InferenceState *s, int kind)
 {
     if (!s->prof_on || s->prof_n >= s->prof_cap) return;
     if (kind >= 0) {
@@ -385,11 +313,11 @@ static unsigned *flags_of(InferenceState *s, int peer, int which) /* which: 0 o,
     return (unsigned *)(s->peer[peer] + s->off_flags) + which * B200_MAX_PEERS;
 }
 
-static void base_args(InferenceState *s, b200_matvec_args *a, const PackedMat *m, int pdl)
+void llmb200_matvec_base(InferenceState *s, b200_matvec_args *a, const PackedMat *m, float eps, int pdl)
 {
     memset(a, 0, sizeof(*a));
     a->d_w = m->w; a->row_stride = m->stride; a->rows = m->rows; a->cols = m->cols; a->wtype = s->wtype;
-    a->eps = 1e-6f;                               /* hard-wired in the reference: src/nn/fast_inference.c:383 */
+    a->eps = eps;
     a->d_pos = s->d_pos; a->d_pos_rw = s->d_pos;
     a->d_epoch = s->d_epoch; a->d_epoch_rw = s->d_epoch; a->d_err = s->d_err;
     a->epoch_mul = s->L + 1;
@@ -397,7 +325,7 @@ static void base_args(InferenceState *s, b200_matvec_args *a, const PackedMat *m
 }
 
 /* Timing loops launch one kind of kernel only; such launches must not touch the token state. */
-static int want(InferenceState *s, int kind, b200_matvec_args *a)
+int llmb200_want_kind(InferenceState *s, int kind, b200_matvec_args *a)
 {
     if (s->only_kind < 0) return 1;
     if (s->only_kind != kind) return 0;
@@ -407,6 +335,8 @@ static int want(InferenceState *s, int kind, b200_matvec_args *a)
     }
     return 1;
 }
+
+#define RMS_EPS 1e-6f                             /* hard-wired in the reference: src/nn/fast_inference.c:383 */
 
 /* Enqueue every kernel of one token on the library stream. */
 static int enqueue_token(InferenceState *s, int with_lm, int pdl)
@@ -419,7 +349,7 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
     for (int l = 0; l < L; ++l) {
         Layer *ly = &s->layers[l];
         /* --- qkv --- */
-        base_args(s, &a, &ly->qkv, pdl);
+        llmb200_matvec_base(s, &a, &ly->qkv, RMS_EPS, pdl);
         if (l == 0) {
             a.in_mode = B200_IN_EMBED; a.d_emb = s->emb; a.d_tokens = s->d_tokens; a.emb_scale = s->emb_scale;
             a.emb_rows = s->V;
@@ -435,13 +365,13 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
         a.d_norm_gamma = ly->g_input;
         a.out_mode = B200_OUT_STORE; a.d_out[0] = s->qkv; a.n_out = 1;
         if (s->lora) a.d_in_copy = s->xnorm;
-        prof_mark(s, K_QKV);
-        if (want(s, K_QKV, &a)) K_TRY(b200_matvec(&a, st), return -1);
+        llmb200_prof_mark(s, K_QKV);
+        if (llmb200_want_kind(s, K_QKV, &a)) K_TRY(b200_matvec(&a, st), return -1);
         /* q += s B_q (A_q ln), v += s B_v (A_v ln)  (src/nn/fast_inference.c:406-421) */
         if (s->lora && (s->only_kind < 0 || s->only_kind == K_QKV))
             K_TRY(b200_lora_decode(s->xnorm, s->lora[l].A_q, s->lora[l].B_q, s->lora[l].A_v, s->lora[l].B_v, s->qkv, D,
                                    s->Hq_l * s->hd, s->Hkv_l * s->hd, s->lora_rank, s->lora_scaling, st), return -1);
-        prof_mark(s, -1);
+        llmb200_prof_mark(s, -1);
         /* --- attention --- */
         b200_attn_args at;
         memset(&at, 0, sizeof(at));
@@ -450,11 +380,11 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
         at.d_out = s->attn_out; at.d_scratch = s->attn_scratch; at.d_tickets = s->attn_tickets; at.d_pos = s->d_pos;
         at.n_q = s->Hq_l; at.n_kv = s->Hkv_l; at.hd = s->hd; at.max_seq = s->max_seq; at.n_split = s->n_split;
         at.eps = 1e-6f; at.use_pdl = pdl;
-        prof_mark(s, K_ATTN);
-        if (want(s, K_ATTN, NULL)) K_TRY(b200_attn_decode(&at, st), return -1);
-        prof_mark(s, -1);
+        llmb200_prof_mark(s, K_ATTN);
+        if (llmb200_want_kind(s, K_ATTN, NULL)) K_TRY(b200_attn_decode(&at, st), return -1);
+        llmb200_prof_mark(s, -1);
         /* --- o: partial sums into slot `me` of every rank --- */
-        base_args(s, &a, &ly->o, pdl);
+        llmb200_matvec_base(s, &a, &ly->o, RMS_EPS, pdl);
         a.in_mode = B200_IN_VEC; a.d_in_vec = s->attn_out;
         a.out_mode = B200_OUT_STORE; a.n_out = k;
         for (int p = 0; p < k; ++p) a.d_out[p] = (float *)(s->peer[p] + s->off_slots_o) + (size_t)me * D;
@@ -462,22 +392,22 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
             a.d_ticket = s->mv_ticket; a.n_signal = k; a.signal_index = me; a.epoch_add = l + 1;
             for (int p = 0; p < k; ++p) a.d_signal_flags[p] = flags_of(s, p, 0);
         }
-        prof_mark(s, K_O);
-        if (want(s, K_O, &a)) K_TRY(b200_matvec(&a, st), return -1);
-        prof_mark(s, -1);
+        llmb200_prof_mark(s, K_O);
+        if (llmb200_want_kind(s, K_O, &a)) K_TRY(b200_matvec(&a, st), return -1);
+        llmb200_prof_mark(s, -1);
         /* --- gate/up --- */
-        base_args(s, &a, &ly->gateup, pdl);
+        llmb200_matvec_base(s, &a, &ly->gateup, RMS_EPS, pdl);
         a.in_mode = B200_IN_RESID; a.d_resid_in = s->resid[1]; a.d_resid_out = s->resid[0];
         a.d_slots = slots_o; a.n_slots = k; a.slot_stride = D;
         a.d_slot_norm_gamma = gemma ? ly->g_post_attn : NULL;
         a.d_norm_gamma = gemma ? ly->g_pre_ff : ly->g_post_attn;
         if (k > 1) { a.d_wait_flags = flags_of(s, me, 0); a.n_wait = k; a.epoch_add = l + 1; }
         a.out_mode = B200_OUT_GLU; a.act = gemma ? 1 : 0; a.d_out[0] = s->act; a.n_out = 1;
-        prof_mark(s, K_GATEUP);
-        if (want(s, K_GATEUP, &a)) K_TRY(b200_matvec(&a, st), return -1);
-        prof_mark(s, -1);
+        llmb200_prof_mark(s, K_GATEUP);
+        if (llmb200_want_kind(s, K_GATEUP, &a)) K_TRY(b200_matvec(&a, st), return -1);
+        llmb200_prof_mark(s, -1);
         /* --- down --- */
-        base_args(s, &a, &ly->down, pdl);
+        llmb200_matvec_base(s, &a, &ly->down, RMS_EPS, pdl);
         a.in_mode = B200_IN_VEC; a.d_in_vec = s->act;
         a.out_mode = B200_OUT_STORE; a.n_out = k;
         for (int p = 0; p < k; ++p) a.d_out[p] = (float *)(s->peer[p] + s->off_slots_dn) + (size_t)me * D;
@@ -486,13 +416,13 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
             for (int p = 0; p < k; ++p) a.d_signal_flags[p] = flags_of(s, p, 1);
         }
         if (!with_lm && l == L - 1) { a.d_ticket = s->mv_ticket; a.advance_pos = 1; a.advance_epoch = 1; }
-        prof_mark(s, K_DOWN);
-        if (want(s, K_DOWN, &a)) K_TRY(b200_matvec(&a, st), return -1);
-        prof_mark(s, -1);
+        llmb200_prof_mark(s, K_DOWN);
+        if (llmb200_want_kind(s, K_DOWN, &a)) K_TRY(b200_matvec(&a, st), return -1);
+        llmb200_prof_mark(s, -1);
     }
     if (!with_lm) return 0;
     /* --- final norm + LM head + greedy pick --- */
-    base_args(s, &a, &s->lm, pdl);
+    llmb200_matvec_base(s, &a, &s->lm, RMS_EPS, pdl);
     a.in_mode = B200_IN_RESID; a.d_resid_in = s->resid[0];
     a.d_slots = slots_dn; a.n_slots = k; a.slot_stride = D;
     a.d_slot_norm_gamma = gemma ? s->layers[L - 1].g_post_ff : NULL;
@@ -519,9 +449,9 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
          * same value L; the finalize kernel waits for that value. */
         a.epoch_add = L;
     }
-    prof_mark(s, K_LM);
-    if (want(s, K_LM, &a)) K_TRY(b200_matvec(&a, st), return -1);
-    prof_mark(s, -1);
+    llmb200_prof_mark(s, K_LM);
+    if (llmb200_want_kind(s, K_LM, &a)) K_TRY(b200_matvec(&a, st), return -1);
+    llmb200_prof_mark(s, -1);
     if (k > 1 && s->only_kind < 0) {
         K_TRY(b200_tp_argmax_finalize((const float *)(s->comm + s->off_am_val), (const int *)(s->comm + s->off_am_idx), k,
                                       flags_of(s, me, 2), s->d_epoch, L + 1, L, s->d_tokens, s->d_pos, s->d_prompt_len,
@@ -608,14 +538,14 @@ static int build_plan(InferenceState *s)
     CU_TRY(cudaMemcpy(s->d_tk_layers, tl, (size_t)L * sizeof(*tl), cudaMemcpyHostToDevice), { free(tl); return -1; });
     free(tl);
     const int qkv_rows = (s->Hq_l + 2 * s->Hkv_l) * s->hd;
-    if (!s->fl_qkv) s->fl_qkv = (b200_flagged *)dev_zero((size_t)qkv_rows * 8);
-    if (!s->fl_part) s->fl_part = (b200_flagged *)dev_zero((size_t)s->Hq_l * a->n_split * (s->hd + 2) * 8);
-    if (!s->fl_attn) s->fl_attn = (b200_flagged *)dev_zero((size_t)s->Hq_l * s->hd * 8);
-    if (!s->fl_act) s->fl_act = (b200_flagged *)dev_zero((size_t)s->IS_l * 8);
-    if (!s->fl_am) s->fl_am = (b200_flagged *)dev_zero((size_t)2 * s->n_sm * 8);
+    if (!s->fl_qkv) s->fl_qkv = (b200_flagged *)llmb200_dev_zero((size_t)qkv_rows * 8);
+    if (!s->fl_part) s->fl_part = (b200_flagged *)llmb200_dev_zero((size_t)s->Hq_l * a->n_split * (s->hd + 2) * 8);
+    if (!s->fl_attn) s->fl_attn = (b200_flagged *)llmb200_dev_zero((size_t)s->Hq_l * s->hd * 8);
+    if (!s->fl_act) s->fl_act = (b200_flagged *)llmb200_dev_zero((size_t)s->IS_l * 8);
+    if (!s->fl_am) s->fl_am = (b200_flagged *)llmb200_dev_zero((size_t)2 * s->n_sm * 8);
     if (!s->fl_qkv || !s->fl_part || !s->fl_attn || !s->fl_act || !s->fl_am) return -1;
     if (getenv("LLMB200_TRACE") && !s->d_step_ns)
-        s->d_step_ns = (unsigned long long *)dev_zero((size_t)s->n_sm * (6 * L + 1) * 16 * 8);
+        s->d_step_ns = (unsigned long long *)llmb200_dev_zero((size_t)s->n_sm * (6 * L + 1) * 16 * 8);
     CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1);
 
     a->d_layers = s->d_tk_layers;
@@ -666,7 +596,7 @@ static int capture(InferenceState *s, int with_lm, int pdl, cudaGraphExec_t *out
     cudaGraph_t g = NULL;
     CU_TRY(cudaStreamBeginCapture(g_rt.stream, cudaStreamCaptureModeThreadLocal), return -1);
     const unsigned long long before = b200_launch_count(0);
-    int rc = s->fused ? enqueue_token_fused(s, with_lm) : enqueue_token(s, with_lm, pdl);
+    int rc = s->fused ? enqueue_token_fused(s, with_lm) : s->ops->enqueue_token(s, with_lm, pdl);
     if (with_lm) s->kernels_full = (int)(b200_launch_count(0) - before);
     else s->kernels_nolm = (int)(b200_launch_count(0) - before);
     cudaError_t e = cudaStreamEndCapture(g_rt.stream, &g);
@@ -692,7 +622,7 @@ static int ensure_graphs(InferenceState *s)
      * kernel's limits or a LoRA adapter is attached (it has no LoRA side path). */
     s->fused = 0;
     const char *tk = getenv("LLMB200_TOKEN_KERNEL");
-    if (!(tk && tk[0] == '0') && !s->lora) {
+    if (s->ops->whole_token && !(tk && tk[0] == '0') && !s->lora) {
         int pr = build_plan(s);
         if (pr < 0) return -1;
         if (pr == 0) {
@@ -954,6 +884,7 @@ void inference_state_set_lora(InferenceState *s, SFTState *sft)
     if (!s || !sft) return;
     const int R = sft_get_lora_rank(sft);
     if (R == 0) return;
+    if (!s->layers) { fprintf(stderr, "[FastGen] inference_state_set_lora: not available for this model type\n"); return; }
     if (s->tp_size != 1) {
         fprintf(stderr, "[FastGen] inference_state_set_lora: not available with tensor parallelism\n");
         return;
@@ -983,6 +914,7 @@ static void free_one(InferenceState *s)
     if (!s) return;
     if (g_rt.refs > 0) cudaStreamSynchronize(g_rt.stream);
     free_graphs(s);
+    if (s->ops && s->ops->free_model) s->ops->free_model(s);
     if (s->layers) {
         for (int i = 0; i < s->L; ++i) {
             Layer *ly = &s->layers[i];
@@ -1078,7 +1010,7 @@ int llmb200_state_connect_loopback(InferenceState *s)
 }
 
 /* Writes pos / prompt_len (and, when n_tok > 0, token ids starting at tok_at) into the control block. */
-static int set_control(InferenceState *s, int pos, int prompt_len, const uint32_t *tok, int tok_at, int n_tok)
+int llmb200_set_control(InferenceState *s, int pos, int prompt_len, const uint32_t *tok, int tok_at, int n_tok)
 {
     CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1);   /* h_ctl may still be in flight */
     s->h_ctl[0] = pos; s->h_ctl[1] = prompt_len;
@@ -1099,7 +1031,7 @@ static const float *forward_token_one(InferenceState *s, int token)
     if (token < 0 || token >= s->V) { fprintf(stderr, "[FastGen] token id %d out of range\n", token); return NULL; }
     uint32_t t = (uint32_t)token;
     /* prompt_len beyond pos+1 keeps the graph from overwriting caller-supplied ids */
-    if (set_control(s, s->cur_len, s->max_seq + 2, &t, s->cur_len, 1) != 0) return NULL;
+    if (llmb200_set_control(s, s->cur_len, s->max_seq + 2, &t, s->cur_len, 1) != 0) return NULL;
     CU_TRY(cudaGraphLaunch(s->g_full, g_rt.stream), return NULL);
     if (s->fused && s->tp_size > 1) {
         /* the whole-token kernel leaves every rank's logits shard on that rank: fetch each from its owner
@@ -1114,6 +1046,54 @@ static const float *forward_token_one(InferenceState *s, int token)
     CU_TRY(cudaStreamSynchronize(g_rt.stream), return NULL);
     s->cur_len++;
     return s->h_logits;
+}
+
+/* One token through the per-token graph; logits == NULL: none are asked for. */
+static int step_one(InferenceState *s, uint32_t token, float *logits)
+{
+    if (llmb200_set_control(s, s->cur_len, s->max_seq + 2, &token, s->cur_len, 1) != 0) return -1;
+    CU_TRY(cudaGraphLaunch(logits ? s->g_full : s->g_nolm, g_rt.stream), return -1);
+    if (logits) CU_TRY(cudaMemcpyAsync(s->h_logits, s->comm + s->off_logits, (size_t)s->V * 4, cudaMemcpyDeviceToHost, g_rt.stream), return -1);
+    CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1);
+    if (logits) memcpy(logits, s->h_logits, (size_t)s->V * 4);
+    s->cur_len++;
+    return 0;
+}
+
+int inference_forward_tokens(InferenceState *s, const uint32_t *tokens, int n, const int *want, int n_want, float *logits)
+{
+    if (!s || !tokens || n <= 0 || n_want < 0 || (n_want > 0 && (!want || !logits))) return B200_E_BADARG;
+    if (s->cur_len + n > s->max_seq) {
+        fprintf(stderr, "[FastGen] %d tokens at position %d exceed the KV cache (%d)\n", n, s->cur_len, s->max_seq);
+        return B200_E_TOOLARGE;
+    }
+    for (int i = 0; i < n; ++i)
+        if (tokens[i] >= (uint32_t)s->V) { fprintf(stderr, "[FastGen] token id %u out of range\n", tokens[i]); return B200_E_BADARG; }
+    for (int i = 0; i < n_want; ++i)
+        if (want[i] < (i ? want[i - 1] + 1 : 0) || want[i] >= n) return B200_E_BADARG;
+    int rc = 0, w = 0;
+    if (s->group_n > 1 || s->tp_size > 1) {      /* tensor parallel: token by token, the logits gathered from the ranks */
+        for (int i = 0; i < n; ++i) {
+            const float *lg = inference_forward_token(s, (int)tokens[i]);
+            if (!lg) return -1;
+            if (w < n_want && want[w] == i) memcpy(logits + (size_t)w++ * s->V, lg, (size_t)s->V * 4);
+        }
+        return llmb200_state_error(s) ? -1 : 0;
+    }
+    follow_sft(s);
+    if (ensure_graphs(s) != 0) return -1;
+    if (s->ops->forward_rows && n > 1) {
+        rc = s->ops->forward_rows(s, tokens, n, want, n_want, logits);
+        if (rc == 0) s->cur_len += n;
+    } else {
+        for (int i = 0; i < n && rc == 0; ++i) {
+            const int wanted = w < n_want && want[w] == i;
+            rc = step_one(s, tokens[i], wanted ? logits + (size_t)w * s->V : NULL);
+            w += wanted;
+        }
+    }
+    if (rc == 0 && llmb200_state_error(s)) { fprintf(stderr, "[FastGen] a device-side wait timed out; results are invalid\n"); rc = -1; }
+    return rc;
 }
 
 static int is_eos(const InferenceState *s, int tok)
@@ -1135,11 +1115,16 @@ static int generate_one(InferenceState *s, const uint32_t *prompt, int prompt_le
         if (prompt[i] >= (uint32_t)s->V) { fprintf(stderr, "[FastGen] prompt token %u out of range\n", prompt[i]); return 0; }
     s->cur_len = 0;
     const int P = prompt_len;
-    if (set_control(s, 0, P, prompt, 0, P) != 0) return 0;
+    if (llmb200_set_control(s, 0, P, prompt, 0, P) != 0) return 0;
 
     fprintf(stderr, "[FastGen] Prefilling %d tokens...\n", P);
     double t0 = now_ms();
-    for (int i = 0; i < P - 1; ++i) CU_TRY(cudaGraphLaunch(s->g_nolm, g_rt.stream), return 0);
+    if (s->ops->forward_rows && P > 2) {         /* all but the last prompt token in one pass; the last one yields the first id */
+        if (s->ops->forward_rows(s, prompt, P - 1, NULL, 0, NULL) != 0) return 0;
+        if (llmb200_set_control(s, P - 1, P, prompt, 0, P) != 0) return 0;
+    } else {
+        for (int i = 0; i < P - 1; ++i) CU_TRY(cudaGraphLaunch(s->g_nolm, g_rt.stream), return 0);
+    }
     CU_TRY(cudaGraphLaunch(s->g_full, g_rt.stream), return 0);
     CU_TRY(cudaMemcpyAsync(&s->h_tok[0], s->d_tokens + P, 4, cudaMemcpyDeviceToHost, g_rt.stream), return 0);
     CU_TRY(cudaStreamSynchronize(g_rt.stream), return 0);
@@ -1418,7 +1403,7 @@ int qwen3_generate_fast(llmb200_qwen3_model *model, const uint32_t *prompt, int 
 }
 
 /* Reads the whole file into a NUL-terminated heap buffer (NULL when it cannot be read). */
-static char *slurp(const char *path)
+char *llmb200_slurp(const char *path)
 {
     FILE *fp = fopen(path, "rb");
     if (!fp) return NULL;
@@ -1449,7 +1434,7 @@ static int parse_eos(const char *model_path, int *eos, int max_eos)
     }
     memcpy(cfg, model_path, dir);
     strcpy(cfg + dir, dir > 0 || model_path[0] == '/' ? "/config.json" : "config.json");
-    char *text = slurp(cfg);
+    char *text = llmb200_slurp(cfg);
     free(cfg);
     if (!text) return 0;
     int n = 0;
@@ -1483,7 +1468,7 @@ void inference_state_load_eos(InferenceState *s, const char *model_path)
     if (s->n_eos == 0) {
         if (s->mt == MODEL_GEMMA3) { s->eos[0] = 1; s->eos[1] = 106; }
         else { s->eos[0] = 151645; s->eos[1] = 151643; }
-        s->n_eos = 2;
+        s->n_eos = s->mt == MODEL_MORILORN ? 0 : 2;            /* that design names none */
     }
     fprintf(stderr, "[FastGen] EOS tokens (%d):", s->n_eos);
     for (int i = 0; i < s->n_eos; ++i) fprintf(stderr, " %d", s->eos[i]);
@@ -1497,7 +1482,7 @@ float llmb200_state_run_device_steps(InferenceState *s, int n_steps)
 {
     if (!s || n_steps <= 0 || ensure_graphs(s) != 0) return -1.0f;
     if (s->cur_len + n_steps > s->max_seq) return -1.0f;
-    if (set_control(s, s->cur_len, 0, NULL, 0, 0) != 0) return -1.0f;
+    if (llmb200_set_control(s, s->cur_len, 0, NULL, 0, 0) != 0) return -1.0f;
     CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1.0f);
     CU_TRY(cudaEventRecord(s->ev_a, g_rt.stream), return -1.0f);
     for (int i = 0; i < n_steps; ++i) CU_TRY(cudaGraphLaunch(s->g_full, g_rt.stream), return -1.0f);
@@ -1513,12 +1498,12 @@ float llmb200_state_time_kind(InferenceState *s, int kind, int reps, int *launch
 {
     if (!s || kind < 0 || kind >= K_KINDS || reps <= 0 || ensure_graphs(s) != 0) return -1.0f;
     if (s->cur_len >= s->max_seq) return -1.0f;
-    if (set_control(s, s->cur_len, 0, NULL, 0, 0) != 0) return -1.0f;
+    if (llmb200_set_control(s, s->cur_len, 0, NULL, 0, 0) != 0) return -1.0f;
     s->only_kind = kind;
-    int rc = enqueue_token(s, kind == K_LM, 0);                 /* warm-up pass, untimed */
+    int rc = s->ops->enqueue_token(s, kind == K_LM, 0);                 /* warm-up pass, untimed */
     const unsigned long long before = b200_launch_count(0);
     if (rc == 0) rc = (int)cudaEventRecord(s->ev_a, g_rt.stream);
-    for (int i = 0; i < reps && rc == 0; ++i) rc = enqueue_token(s, kind == K_LM, 0);
+    for (int i = 0; i < reps && rc == 0; ++i) rc = s->ops->enqueue_token(s, kind == K_LM, 0);
     if (rc == 0) rc = (int)cudaEventRecord(s->ev_b, g_rt.stream);
     s->only_kind = -1;
     if (launches) *launches = (int)(b200_launch_count(0) - before);
@@ -1541,11 +1526,11 @@ int llmb200_state_profile_token(InferenceState *s, float *ms, int *launches)
         for (int i = 0; i < need; ++i) CU_TRY(cudaEventCreate(&s->prof_ev[i]), return -1);
         s->prof_cap = need;
     }
-    if (set_control(s, s->cur_len, 0, NULL, 0, 0) != 0) return -1;
+    if (llmb200_set_control(s, s->cur_len, 0, NULL, 0, 0) != 0) return -1;
     s->prof_n = 0;
     cudaEvent_t *ev = s->prof_ev;
     s->prof_on = 1;
-    int rc = enqueue_token(s, 1, 0);
+    int rc = s->ops->enqueue_token(s, 1, 0);
     s->prof_on = 0;
     const int n = s->prof_n;
     CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1);
@@ -1566,11 +1551,11 @@ size_t llmb200_state_export_weight(InferenceState *s, int layer, int which, void
     if (!s) return 0;
     const PackedMat *m = NULL;
     if (which == 4) m = &s->lm;
-    else if (layer >= 0 && layer < s->L) {
+    else if (s->layers && layer >= 0 && layer < s->L) {
         Layer *ly = &s->layers[layer];
         m = which == 0 ? &ly->qkv : which == 1 ? &ly->o : which == 2 ? &ly->gateup : which == 3 ? &ly->down : NULL;
     }
-    if (!m) return 0;
+    if (!m || !m->w) return 0;
     const size_t bytes = s->wtype == B200_WT_Q8 ? (size_t)m->rows * (m->cols / 32) * 34 : (size_t)m->rows * m->cols * 2;
     if (!buf) return bytes;
     if (cap < bytes) return 0;

@@ -198,7 +198,10 @@ int llmb200_upload_packed(int wtype, const float *src, long long ld, int rows, i
         }
         CU_TRY(cudaMemcpyAsync(g_rt.d_stage[sb], g_rt.h_stage[sb], (size_t)nr * row_floats * sizeof(float),
                                cudaMemcpyHostToDevice, g_rt.stream), return -101);
-        int rc = wtype == B200_WT_Q8
+        int rc = wtype == B200_WT_BF16 || wtype == B200_WT_F32
+            ? b200_cast_pack(wtype, g_rt.d_stage[sb], cols, nr, cols, d_dst, dst_row_stride,
+                             dst_row0 + (int)r * dst_row_step, dst_row_step, g_rt.stream)
+            : wtype == B200_WT_Q8
             ? b200_q8_pack(g_rt.d_stage[sb], cols, nr, cols, d_dst, dst_row_stride,
                            dst_row0 + (int)r * dst_row_step, dst_row_step, g_rt.stream)
             : b200_f16_pack(g_rt.d_stage[sb], cols, nr, cols, d_dst, dst_row_stride,
