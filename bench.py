@@ -438,6 +438,282 @@ def batch_main(args, rank, local_rank, world):
     return 0
 
 
+LATENT_WORKLOADS = {
+    # name: sizes of (width, layers, heads, dim, rot_dim, vdim, kv_rank, ff, vocab, window), each beside a Qwen3 model of the same
+    # width, layers, heads x 128, feed-forward and vocabulary; prompt portion, generated tokens
+    "morilorn": ([dict(width=2048, layers=16, heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, ff=6144, vocab=32768, window=1024),
+                  dict(width=2560, layers=12, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, ff=9728, vocab=65536, window=1024),
+                  dict(width=4096, layers=6, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, ff=12288, vocab=65536, window=4096)], 2048, 256),
+    "tiny-morilorn": ([dict(width=256, layers=3, heads=4, dim=48, rot_dim=16, vdim=64, kv_rank=64, ff=512, vocab=1024, window=64)], 128, 32),
+}
+
+
+def write_latent_model(folder, z, seed):
+    """A Morilorn model folder of the sizes z: matrices N(0, 0.02) cut from one random block, norm weights one."""
+    layer = {"type": "latent_attention",
+             "mixer": {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+                       "mask": {"size": z["window"]}, "rot": {"base": 10000.0, "dims": z["rot_dim"]}, "scale": (z["dim"] + z["rot_dim"]) ** -0.5},
+             "mlp": {"kind": "dense", "ff": z["ff"]}}
+    D, V, F, H, R, nl = z["width"], z["vocab"], z["ff"], z["heads"], z["kv_rank"], z["layers"]
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump({"architecture": "Morilorn", "vocab": V, "width": D, "embedding": {"scale": 12.0}, "norm": {"eps": 1e-5, "groups": 2},
+                   "postln_alpha": 2.0, "logit_softcap": 15.0, "layers": [layer] * nl}, f)
+    shapes = {"embed": (V, D), "head": (V, D), "final.norm": (D,)}
+    for i in range(nl):
+        shapes.update({f"l{i}.{k}": v for k, v in {
+            "norm1": (D,), "norm2": (D,), "mix.q": (H * (z["dim"] + z["rot_dim"]), D), "mix.dkv": (R + z["rot_dim"], D), "mix.dkv.norm": (R,),
+            "mix.uk": (H * z["dim"], R), "mix.uv": (H * z["vdim"], R), "mix.g": (H * z["vdim"], D), "mix.o": (D, H * z["vdim"]),
+            "mlp.gate": (F, D), "mlp.up": (F, D), "mlp.down": (D, F), "rg1": (D, D), "rg1.b": (D,), "rg2": (D, D), "rg2.b": (D,),
+            "dwa": (i + 2,)}.items()})
+    header, at = {}, 0
+    for k, v in shapes.items():
+        n = 2 * int(np.prod(v))
+        header[k] = {"dtype": "BF16", "shape": list(v), "data_offsets": [at, at + n]}
+        at += n
+    text = json.dumps(header).encode()
+    rng = np.random.default_rng(seed)
+    block = ((rng.standard_normal(1 << 22).astype(np.float32) * 0.02).view(np.uint32) >> 16).astype("<u2")
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(len(text).to_bytes(8, "little") + text)
+        for k, v in shapes.items():
+            n = int(np.prod(v))
+            if k.endswith("dwa"):
+                w = np.full(n, 0.1, dtype=np.float32)
+                w[-1] = 1.0
+            elif "norm" in k:
+                w = np.ones(n, dtype=np.float32)
+            else:
+                w = None
+            if w is not None:
+                f.write((w.view(np.uint32) >> 16).astype("<u2").tobytes())
+                continue
+            o = int(rng.integers(0, block.size))
+            while n > 0:
+                m = min(n, block.size - o)
+                f.write(block[o:o + m].tobytes())
+                n, o = n - m, 0
+    return folder
+
+
+def latent_kernel_timings(pkg, L, torch, z, M, peaks):
+    """Prompt-portion kernels alone at these sizes, beside the like kernel of the Qwen3 path: the gate/up product on bfloat16
+    against binary16 operands, and the attention of one layer for M tokens."""
+    up8 = lambda n: (n + 7) // 8 * 8
+    D, F, H = z["width"], z["ff"], z["heads"]
+    hbm, tc = peaks
+    out = {}
+
+    def timed(fn, reps=10):
+        for _ in range(3):
+            fn()
+        flush = torch.empty(1 << 28, dtype=torch.uint8, device="cuda")
+        ms = []
+        for _ in range(reps):
+            flush.zero_()                                        # larger than L2
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            e1.synchronize()
+            ms.append(e0.elapsed_time(e1))
+        return statistics.median(ms)
+
+    st = torch.cuda.current_stream().cuda_stream
+    for name, fn, dt in (("gateup_product_bf16", L.b200_gemm_bf16, torch.bfloat16), ("gateup_product_f16_closest_model", L.b200_gemm_f16, torch.float16)):
+        a, b = torch.randn(M, D, device="cuda").to(dt), (torch.randn(2 * F, D, device="cuda") * 0.02).to(dt)
+        c = torch.empty(M, 2 * F, device="cuda")
+        g = pkg.GemmArgs()
+        g.A, g.a_row, g.a_col, g.B, g.b_row, g.b_col = a.data_ptr(), D, 1, b.data_ptr(), 1, D
+        g.C, g.ldc, g.M, g.N, g.K, g.alpha = c.data_ptr(), 2 * F, M, 2 * F, D, 1.0
+
+        def run():
+            if fn(C.byref(g), st) != 0:
+                raise RuntimeError(name)
+        ms = timed(run)
+        tf = 2.0 * M * 2 * F * D / ms / 1e9
+        out[name] = {"us": 1e3 * ms, "tflops": tf, "frac_of_tensor_peak": tf / tc}
+    d8, r8, v8, R8, n = up8(z["dim"]), up8(z["rot_dim"]), up8(z["vdim"]), up8(z["kv_rank"]), M
+    W = min(z["window"], n)
+    a = pkg.LatentArgs()
+    a.wtype, a.heads, a.dim, a.rot_dim, a.rot_dims, a.vdim, a.kv_rank = 2, H, z["dim"], z["rot_dim"], z["rot_dim"], z["vdim"], z["kv_rank"]
+    a.window, a.max_seq, a.scale, a.eps, a.n_rows, a.pos0, a.kv_row0 = z["window"], n, 0.07, 1e-5, n, 0, 0
+    ld = H * (z["dim"] + z["rot_dim"]) + z["kv_rank"] + z["rot_dim"] + H * z["vdim"]
+    proj = torch.randn(n, ld, device="cuda")
+    gam, rope = torch.ones(R8, device="cuda"), torch.randn(n, z["rot_dim"], device="cuda")
+    cache, q = (torch.randn(n, s, device="cuda").bfloat16() for s in (R8 + r8, H * (d8 + r8)))
+    kv, o = (torch.randn(n, s, device="cuda").bfloat16() for s in (H * (d8 + v8), H * z["vdim"]))
+    a.d_q = proj.data_ptr()
+    a.d_dkv = a.d_q + 4 * H * (z["dim"] + z["rot_dim"])
+    a.d_gate, a.proj_ld = a.d_dkv + 4 * (z["kv_rank"] + z["rot_dim"]), ld
+    a.d_dkv_gamma, a.d_rope, a.d_cache, a.d_q_rows = gam.data_ptr(), rope.data_ptr(), cache.data_ptr(), q.data_ptr()
+    a.d_kv, a.kv_ld, a.d_out_rows, a.out_ld = kv.data_ptr(), kv.shape[1], o.data_ptr(), o.shape[1]
+    seen = sum(min(i + 1, W) for i in range(n))
+    flops = 2.0 * seen * H * (z["dim"] + z["rot_dim"] + z["vdim"])
+    for name, fn in (("attention_rows", L.b200_latent_rows_attend), ("attention_rows_prep", L.b200_latent_rows_prep)):
+        def run():
+            if fn(C.byref(a), st) != 0:
+                raise RuntimeError(name)
+        ms = timed(run)
+        out[name] = {"us": 1e3 * ms}
+        if name == "attention_rows":
+            out[name].update(tflops=flops / ms / 1e9, frac_of_tensor_peak=flops / ms / 1e9 / tc)
+        else:
+            nb = n * (4.0 * (ld - H * z["vdim"]) + 2.0 * (R8 + r8 + H * (d8 + r8)))
+            out[name].update(gbs=nb / ms / 1e6, frac_of_hbm=nb / ms / 1e6 / hbm)
+    # the closest model's attention over rows (its SFT forward), same heads and sequence, head dimension 128, causal without a window
+    ns = min(n, 512)
+    qt, kt, vt, at, pr = (torch.randn(ns, H * 128, device="cuda") for _ in range(5))
+    probs = torch.empty(H * ns * ns, device="cuda")
+
+    def run():
+        rc = L.b200_attn_train_fwd(qt.data_ptr(), kt.data_ptr(), vt.data_ptr(), H * 128, 1, ns, H, H, 128, C.c_float(0.09), probs.data_ptr(),
+                                   at.data_ptr(), st)
+        if rc != 0:
+            raise RuntimeError("attn_train_fwd: %d" % rc)
+    ms = timed(run, 3)
+    fl = 2.0 * (ns * (ns + 1) / 2) * H * 256
+    out["attention_rows_closest_model"] = {"us": 1e3 * ms, "tokens": ns, "tflops": fl / ms / 1e9, "frac_of_tensor_peak": fl / ms / 1e9 / tc}
+    return out
+
+
+def latent_main(args, rank, local_rank, world):
+    """Morilorn: prompt portions and decode at several sizes, each beside a Qwen3 (binary16) model of equal width, depth, heads,
+    feed-forward and vocabulary on this library. The line's value is the first size's decode rate."""
+    if args.impl == "reference" or world > 1:
+        if rank == 0:
+            emit(json.dumps({"impl": args.impl, "unavailable": "the reference has no such model; the workload runs on one GPU"}))
+        return 0
+    import shutil
+    import tempfile
+    import torch
+    torch.cuda.set_device(local_rank)
+    sizes, P, G = LATENT_WORKLOADS[args.workload]
+    P, G = args.prompt_len or P, args.gen_len or G
+    pkg = entry.load_package()
+    L, S = pkg.lib(), pkg.synth()
+    peak, peak_kind = measured_peaks()
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tc = float(json.load(f)["bf16_tflops"])
+    except Exception:
+        tc = 1590.0
+    threads = max(1, min(32, os.cpu_count() or 8))
+    kinds = ["in", "attention", "o", "gateup", "down", "lm_head"]
+    rows, launches = [], 0
+    sampler = ClockSampler(local_rank)
+    for zi, z in enumerate(sizes):
+        z = dict(z, layers=args.layers or z["layers"])
+        folder = tempfile.mkdtemp(prefix="morilorn-")
+        try:
+            write_latent_model(folder, z, 7 + zi)
+            m = pkg.DirModel(folder, P + G + 8, "bfloat16")
+        finally:
+            shutil.rmtree(folder)
+        D, nl, H, V = z["width"], z["layers"], z["heads"], z["vocab"]
+        prompt = np.zeros(P, dtype=np.uint32)
+        S.llmb200_synth_tokens(prompt.ctypes.data, P, 4321, V)
+        pp = prompt.ctypes.data_as(pkg.c_u32_p)
+        L.llmb200_state_set_eos(m.state, None, 0)
+        out = np.zeros(G, dtype=np.uint32)
+        op = out.ctypes.data_as(pkg.c_u32_p)
+        if zi == 0:
+            sampler.start()
+        prefill, decode, e2e = [], [], []
+        graph = L.llmb200_state_graph_kernels(m.state, 1)
+        for it in range(args.warmup + args.steps):
+            m.reset()
+            L.metal_flush()
+            t0 = time.perf_counter()
+            if L.inference_forward_tokens(m.state, pp, P, None, 0, None) != 0:
+                raise RuntimeError("prompt portion failed")
+            t1 = time.perf_counter()
+            ms = L.llmb200_state_run_device_steps(m.state, G - 1)
+            if ms <= 0:
+                raise RuntimeError("device steps failed")
+            n = L.inference_generate(m.state, pp, P, op, G)
+            nd = C.c_int(0)
+            dms = L.llmb200_last_decode_ms(m.state, C.byref(nd))
+            if n != G:
+                raise RuntimeError("generate failed")
+            if it >= args.warmup:
+                prefill.append((t1 - t0) * 1e3); decode.append(ms); e2e.append(dms)
+                launches += graph * (G - 1)
+        per_kind = {}
+        m.reset()
+        m.feed(prompt.tolist())
+        for k, name in enumerate(kinds):
+            cnt = C.c_int(0)
+            ms = L.llmb200_state_time_kind(m.state, k, 8 if k < 5 else 24, C.byref(cnt))
+            per_layer = 3 if name == "attention" else 1
+            per_kind[name] = {"us": 1e3 * ms / cnt.value * per_layer}
+        up8 = lambda v: (v + 7) // 8 * 8
+        in_rows = H * (z["dim"] + z["rot_dim"]) + z["kv_rank"] + z["rot_dim"] + H * z["vdim"] + D
+        cs, W = z["kv_rank"] + z["rot_dim"], min(z["window"], P)
+        kbytes = {"in": 2 * in_rows * D, "attention": 2 * (H * z["kv_rank"] * (z["dim"] + z["vdim"]) + W * cs), "o": 2 * D * H * z["vdim"],
+                  "gateup": 2 * (2 * z["ff"] + D) * D, "down": 2 * D * z["ff"], "lm_head": 2 * V * D}
+        for name, b in kbytes.items():
+            per_kind[name].update(bytes=b, gbs=b / per_kind[name]["us"] / 1e3, frac_of_hbm=b / per_kind[name]["us"] / 1e3 / peak)
+        token_bytes = sum(b * (nl if k != "lm_head" else 1) for k, b in kbytes.items())
+        us = 1e3 * statistics.median(decode) / (G - 1)
+        pf = statistics.median(prefill)
+        row_flops = 2.0 * P * nl * (in_rows * D + H * z["kv_rank"] * (z["dim"] + z["vdim"]) + D * H * z["vdim"] + (3 * z["ff"] + D) * D)
+        res = {"sizes": z, "decode": {"tokens_per_s": 1e6 / us, "us_per_token": us, "bytes_per_token": token_bytes,
+                                      "frac_of_hbm": token_bytes / us / 1e3 / peak, "kernels": per_kind, "launches_per_token": graph},
+               "decode_e2e_tokens_per_s": (G - 1) / statistics.median(e2e) * 1e3,
+               "prefill": {"tokens": P, "ms": pf, "tokens_per_s": P / pf * 1e3, "product_tflops": row_flops / pf / 1e9,
+                           "frac_of_tensor_peak": row_flops / pf / 1e9 / tc}}
+        if L.llmb200_state_error(m.state):
+            raise RuntimeError("a device-side wait timed out")
+        m.close()
+        res["kernels_alone"] = latent_kernel_timings(pkg, L, torch, z, P, (peak, tc))
+        # the closest model at equal size
+        sp = pkg.spec("qwen3-4b", n_layers=nl, d_model=D, n_q_heads=H, n_kv_heads=max(1, H // 4), head_dim=128, intermediate_size=z["ff"], vocab_size=V)
+        near = {}
+        for label, env in (("whole_token_kernel", "1"), ("one_kernel_per_stage", "0")):
+            os.environ["LLMB200_TOKEN_KERNEL"] = env
+            st = build_state_streaming(pkg, L, S, sp, min(4096, P + G + 8), 1, threads)
+            L.llmb200_state_set_eos(st, None, 0)
+            Pq = min(P, 4096 - G - 8)
+            ms, pfq = [], []
+            for it in range(1 + args.steps):
+                if L.inference_generate(st, pp, Pq, op, 1) != 1:
+                    raise RuntimeError("prefill failed")
+                pfq.append(L.llmb200_last_prefill_ms(st))
+                ms.append(L.llmb200_state_run_device_steps(st, G - 1))
+            qb = float(np.mean([algorithmic_bytes_per_token(sp, k, 1, 1) for k in (Pq, Pq + G)]))
+            uq = 1e3 * statistics.median(ms[1:]) / (G - 1)
+            near[label] = {"us_per_token": uq, "tokens_per_s": 1e6 / uq, "bytes_per_token": qb, "frac_of_hbm": qb / uq / 1e3 / peak,
+                           "prefill_tokens_per_s": Pq / statistics.median(pfq[1:]) * 1e3}
+            if env == "0":
+                ks, hd = {}, 128
+                qkb = {"in": 2 * (H + 2 * max(1, H // 4)) * hd * D, "attention": 2 * 2 * max(1, H // 4) * hd * (Pq + G), "o": 2 * D * H * hd,
+                       "gateup": 2 * 2 * z["ff"] * D, "down": 2 * D * z["ff"], "lm_head": 2 * V * D}
+                for k, name in enumerate(kinds):
+                    cnt = C.c_int(0)
+                    t = L.llmb200_state_time_kind(st, k, 8 if k < 5 else 24, C.byref(cnt))
+                    ks[name] = {"us": 1e3 * t / cnt.value, "gbs": qkb[name] / (1e3 * t / cnt.value) / 1e3,
+                                "frac_of_hbm": qkb[name] / (1e3 * t / cnt.value) / 1e3 / peak}
+                near[label]["kernels"] = ks
+            L.inference_state_free(st)
+        os.environ.pop("LLMB200_TOKEN_KERNEL")
+        res["closest_model"] = dict(near, what="Qwen3 blocks, binary16 weights, same width / layers / heads x 128 / feed-forward / vocabulary")
+        rows.append(res)
+    clocks = sampler.stop()
+    r0 = rows[0]
+    emit(json.dumps({
+        "metric": "decode_tokens_per_s", "value": r0["decode"]["tokens_per_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": r0["decode"]["us_per_token"] * (G - 1) / 1e3, "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+        "dtype": "bf16 matrices and products, f32 accumulate, norms, scores and residuals", "data": "synthetic",
+        "config": {"workload": f"Morilorn latent-attention decoder: prompt portion of {P} tokens in one pass, {G - 1} decode steps, sizes in 'sizes'",
+                   "prompt_len": P, "gen_len": G, "parallelism": "tp1", "l2": "inputs larger than L2 (all weights streamed per token); kernels alone: L2 flushed"},
+        "e2e": {"value": r0["decode_e2e_tokens_per_s"], "unit": "tok/s", "h2d_bytes_per_step": int(P * 4 + 8), "d2h_bytes_per_step": int(G * 4)},
+        "gpu_launches": int(launches),
+        "roofline": {"bound": "hbm", "kernel": "one token, all kernels", "achieved": r0["decode"]["bytes_per_token"] / r0["decode"]["us_per_token"] / 1e3,
+                     "peak": peak, "unit": "GB/s", "frac": r0["decode"]["frac_of_hbm"], "peak_source": peak_kind, "traffic": None},
+        "clocks": clocks, "sizes": rows}))
+    return 0
+
+
 def sft_main(args, rank, local_rank, world):
     arch, seq, n_seq, lrank, alpha = SFT_WORKLOADS[args.workload]
     pkg = entry.load_package()
@@ -763,7 +1039,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="qwen3-4b-q8",
-                    choices=sorted(WORKLOADS) + sorted(SFT_WORKLOADS) + sorted(BATCH_WORKLOADS) + ["matvec-sweep"])
+                    choices=sorted(WORKLOADS) + sorted(SFT_WORKLOADS) + sorted(BATCH_WORKLOADS) + sorted(LATENT_WORKLOADS) + ["matvec-sweep"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-secondary", action="store_true", help="skip the secondary configurations and the parity stamp")
     ap.add_argument("--prompt-len", type=int, default=0, help="override the workload's prompt length (profiling runs)")
@@ -778,6 +1054,8 @@ def main():
         return sft_main(args, rank, local_rank, world)
     if args.workload in BATCH_WORKLOADS:
         return batch_main(args, rank, local_rank, world)
+    if args.workload in LATENT_WORKLOADS:
+        return latent_main(args, rank, local_rank, world)
     if args.workload == "matvec-sweep":
         if args.impl == "reference" or world > 1:
             if rank == 0:

@@ -363,6 +363,7 @@ static void take_layer_result(const Latent *m, int l, const float *z, b200_matve
 static void gated(const Latent *m, int l, int last, const float *resid, const float *gate, const float *bias, float *z, b200_matvec_args *a)
 {
     a->in_mode = B200_IN_VEC;
+    a->norm_dim = a->norm_groups = 0;                        /* this product's input is not of the model's width */
     a->out_mode = B200_OUT_GATED;
     a->d_out_resid = resid; a->d_out_gate = gate; a->d_out_gate_bias = bias; a->resid_alpha = m->alpha;
     a->d_out[0] = z;
