@@ -4,8 +4,8 @@
 //   latent_absorb  per head q_lat = scale * W_uk^T q (the weight slice of a block is in registers before the
 //                  previous kernel has finished); one extra block normalises the new token's latent, rotates its
 //                  key part and the queries, and writes the cache row
-//   latent_scores  split-sequence attention in the latent space: a block takes 32 cache rows at a time for eight
-//                  heads (one warp each), rows staged once in shared memory and used for the scores and for the
+//   latent_scores  split-sequence attention in the latent space: a block takes 32 cache rows at a time for four
+//                  heads (two warps each), rows staged once in shared memory and used for the scores and for the
 //                  weighted sum; partial (sum, maximum, total) records per split
 //   latent_value   merges the splits of a head, applies W_uv and the output gate
 //
@@ -23,9 +23,9 @@ extern unsigned long long g_b200_launches;
 namespace {
 
 constexpr int KT = 32;             // cache rows per tile of the decode scores = lanes of a warp
-constexpr int HB = 8;              // heads per block of the decode scores = warps
+constexpr int HB = 4;              // heads per block of the decode scores, two warps each
 constexpr int ABSORB_PASSES = 4;   // row passes whose weights a warp of latent_absorb holds in registers
-constexpr int VALUE_ROWS = 32;     // value rows per block of latent_value, four per warp
+constexpr int VALUE_ROWS = 16;     // value rows per block of latent_value, two per warp
 constexpr int MAX_SPLITS = 256;
 
 __host__ __device__ __forceinline__ int up8(int n) { return (n + 7) & ~7; }
@@ -61,23 +61,53 @@ __device__ __forceinline__ float rotated(const float *v, int i, int dims, const 
     return (i & 1) ? b * c + a * s : a * c - b * s;
 }
 
-// The cache row of one token, by all threads of a block. `red` holds >= 33 floats.
-template <typename T>
-__device__ __forceinline__ void write_cache_row(const b200_latent_args &p, const float *dkv, int pos, float *red)
+__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool on)
 {
-    const int R = p.kv_rank, R8 = up8(R), rot8 = up8(p.rot_dim);
+    const int n = on ? 16 : 0;                               // 0: the 16 bytes are zero-filled
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// The cache row of one token, by all 256 threads of a block. `wait` runs before anything an earlier kernel of the
+// same token wrote is read; norm weights and angles are fetched ahead of it. `red` holds >= 33 floats.
+template <typename T, typename Wait>
+__device__ __forceinline__ void write_cache_row(const b200_latent_args &p, const float *dkv, int pos, float *red, Wait wait)
+{
+    constexpr int HELD = 4;                                  // elements a thread keeps in registers: 1024 a block
+    const int R = p.kv_rank, R8 = up8(R), rot8 = up8(p.rot_dim), tid = threadIdx.x;
     T *row = static_cast<T *>(p.d_cache) + (size_t)pos * (R8 + rot8);
     const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
+    float g[HELD], v[HELD];
+#pragma unroll
+    for (int k = 0; k < HELD; ++k) g[k] = tid + k * 256 < R ? p.d_dkv_gamma[tid + k * 256] : 0.0f;
+    float c = 1.0f, s = 0.0f;
+    if (tid < p.rot_dims) { c = rope[tid & ~1]; s = rope[(tid & ~1) + 1]; }
+    wait();
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < R; i += blockDim.x) ss = fmaf(dkv[i], dkv[i], ss);
+#pragma unroll
+    for (int k = 0; k < HELD; ++k) { v[k] = tid + k * 256 < R ? dkv[tid + k * 256] : 0.0f; ss = fmaf(v[k], v[k], ss); }
+    for (int i = tid + HELD * 256; i < R; i += 256) ss = fmaf(dkv[i], dkv[i], ss);
+    if (tid < rot8) {
+        float r = 0.0f;
+        if (tid < p.rot_dims) {
+            const float x = dkv[R + (tid & ~1)], y = dkv[R + (tid & ~1) + 1];
+            r = (tid & 1) ? y * c + x * s : x * c - y * s;
+        } else if (tid < p.rot_dim) r = dkv[R + tid];
+        row[R8 + tid] = (T)r;
+    }
+    for (int i = tid + 256; i < rot8; i += 256) row[R8 + i] = (T)(i < p.rot_dim ? rotated(dkv + R, i, p.rot_dims, rope) : 0.0f);
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)R + p.eps);
-    for (int i = threadIdx.x; i < R8; i += blockDim.x) row[i] = (T)(i < R ? p.d_dkv_gamma[i] * (dkv[i] * inv) : 0.0f);
-    for (int i = threadIdx.x; i < rot8; i += blockDim.x)
-        row[R8 + i] = (T)(i < p.rot_dim ? rotated(dkv + R, i, p.rot_dims, rope) : 0.0f);
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+        if (tid + k * 256 < R8) row[tid + k * 256] = (T)(g[k] * (v[k] * inv));
+    for (int i = tid + HELD * 256; i < R8; i += 256) row[i] = (T)(i < R ? p.d_dkv_gamma[i] * (dkv[i] * inv) : 0.0f);
 }
 
 // ------------------------------------------------------------------------------------------------ decode
+// The position changes between tokens only, never between the kernels of one token, so each kernel may read it (and
+// everything that depends on it alone: angles, cache rows of earlier tokens) before it waits for its predecessor.
 
 template <int WT>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constant__ b200_latent_args p, int chunks, int lpr)
@@ -88,17 +118,11 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
     __shared__ float red[33];
     pdl_launch_dependents();
     const int R = p.kv_rank, R8 = up8(R), rot8 = up8(p.rot_dim), CS = R8 + rot8, dq = p.dim + p.rot_dim;
+    const int pos = *p.d_pos;
+    const bool valid = pos >= 0 && pos < p.max_seq;
     if ((int)blockIdx.x == p.heads * chunks) {
-        pdl_wait();
-        const int pos = *p.d_pos;
-        if (pos < 0 || pos >= p.max_seq) return;
-        write_cache_row<T>(p, p.d_dkv, pos, red);
-        const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
-        for (int i = threadIdx.x; i < p.heads * rot8; i += blockDim.x) {
-            const int h = i / rot8, e = i % rot8;
-            p.d_qlat[(size_t)h * CS + R8 + e] =
-                e < p.rot_dim ? p.scale * rotated(p.d_q + (size_t)h * dq + p.dim, e, p.rot_dims, rope) : 0.0f;
-        }
+        if (valid) write_cache_row<T>(p, p.d_dkv, pos, red, [] { pdl_wait(); });
+        else pdl_wait();
         return;
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -117,6 +141,13 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
     float x[E];
 #pragma unroll
     for (int e = 0; e < E; ++e) x[e] = sl * E + e < p.dim ? q[sl * E + e] : 0.0f;
+    // the head's first block also rotates its query and clears the padding columns of the latent part
+    if (chunk == 0 && valid) {
+        float *ql = p.d_qlat + (size_t)h * CS;
+        const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
+        for (int i = threadIdx.x; i < rot8; i += 256) ql[R8 + i] = i < p.rot_dim ? p.scale * rotated(q + p.dim, i, p.rot_dims, rope) : 0.0f;
+        if ((int)threadIdx.x < R8 - R) ql[R + threadIdx.x] = 0.0f;
+    }
 #pragma unroll
     for (int k = 0; k < ABSORB_PASSES; ++k) {
         const int row = row0 + k * 8 * rpw;
@@ -131,10 +162,10 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
         for (int o = 1; o < lpr; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
         if (sl == 0 && row < R) p.d_qlat[(size_t)h * CS + row] = p.scale * acc;
     }
-    // padding columns of the latent part
-    if (chunk == 0 && threadIdx.x < R8 - R) p.d_qlat[(size_t)h * CS + R + threadIdx.x] = 0.0f;
 }
 
+// Two warps per head: warp 2i + f of head i scores the tile's keys 16 f .. 16 f + 15 (two lanes per key, every
+// other slice each) and sums the columns of half f (slices f, f + 2, ... of 32) of the weighted rows.
 template <int WT, int NCH>
 __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constant__ b200_latent_args p, int row16)
 {
@@ -142,14 +173,15 @@ __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constan
     using T = typename El::T;
     constexpr int E = El::E;
     extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float ssh[HB][KT];
     pdl_launch_dependents();
     const int R8 = up8(p.kv_rank), rot8 = up8(p.rot_dim), CS = R8 + rot8, PS = R8 + 8;
     const int S = CS / E;                                    // 16-byte slices of a cache row
-    unsigned char *keys = smem;                              // [KT] rows, row16 slices apart (odd: no bank conflicts)
+    unsigned char *keys = smem;                              // [KT] rows, row16 slices apart (2 mod 4: no bank conflicts)
     float *qs = reinterpret_cast<float *>(smem + (size_t)KT * row16 * 16);       // [HB][CS]
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int h0 = blockIdx.y * HB, h = h0 + warp, split = blockIdx.x;
-    const int pos = *p.d_pos;                                // changes only between tokens, not between their kernels
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hi = warp >> 1, half = warp & 1;
+    const int h0 = blockIdx.y * HB, h = h0 + hi, split = blockIdx.x;
+    const int pos = *p.d_pos;
     const bool valid = pos >= 0 && pos < p.max_seq;
     const int lo = valid && p.window > 0 && pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
     const int nk = valid ? pos - lo + 1 : 0;
@@ -157,40 +189,60 @@ __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constan
     const int t0 = split * per, t1 = min(t0 + per, tiles);
     const T *cache = static_cast<const T *>(p.d_cache);
 
-    // every row but the new token's was written by an earlier token: the first tile is fetched before the wait
-    auto stage = [&](int tile, bool newest_only) {
+    // rows of a tile except the new token's, which this token's previous kernel has written
+    auto stage_row = [&](int r, int kp) {
+        for (int c = lane; c < S; c += 32) cp16(smem_u32(keys + ((size_t)r * row16 + c) * 16), cache + (size_t)kp * CS + (size_t)c * E, true);
+    };
+    auto stage = [&](int tile) {
         const int k0 = tile * KT, n = min(KT, nk - k0);
-        for (int i = threadIdx.x; i < n * S; i += 256) {
-            const int r = i / S, c = i % S, kp = lo + k0 + r;
-            if ((kp == pos) != newest_only) continue;
-            *reinterpret_cast<uint4 *>(keys + ((size_t)r * row16 + c) * 16) =
-                *reinterpret_cast<const uint4 *>(cache + (size_t)kp * CS + (size_t)c * E);
+#pragma unroll
+        for (int i = 0; i < KT / 8; ++i) {
+            const int r = warp + 8 * i;
+            if (r < n && lo + k0 + r != pos) stage_row(r, lo + k0 + r);
         }
     };
-    if (t0 < t1) stage(t0, false);
+    if (t0 < t1) stage(t0);
     pdl_wait();
-    for (int i = threadIdx.x; i < HB * CS; i += 256) qs[i] = h0 + i / CS < p.heads ? p.d_qlat[(size_t)h0 * CS + i] : 0.0f;
-
+    {
+        const int n = min(HB, p.heads - h0) * CS / 4;        // queries: contiguous fp32 rows
+        for (int i = threadIdx.x; i < n; i += 256) cp16(smem_u32(qs + 4 * i), p.d_qlat + (size_t)h0 * CS + 4 * i, true);
+        if (t0 < t1 && t1 == tiles && warp == 0) {           // the newest key is the last row of the last tile
+            const int r = nk - 1 - (tiles - 1) * KT;
+            if (tiles - 1 == t0) stage_row(r, pos);
+        }
+    }
     float m = -INFINITY, l = 0.0f, acc[NCH][E];
 #pragma unroll
     for (int c = 0; c < NCH; ++c)
 #pragma unroll
         for (int e = 0; e < E; ++e) acc[c][e] = 0.0f;
     for (int tile = t0; tile < t1; ++tile) {
-        if (tile > t0) { __syncthreads(); stage(tile, false); }
-        if (tile == tiles - 1) stage(tile, true);
+        if (tile > t0) {
+            __syncthreads();
+            stage(tile);
+            if (tile == tiles - 1 && warp == 0) stage_row(nk - 1 - tile * KT, pos);
+        }
+        cp_commit();
+        cp_wait<0>();
         __syncthreads();
         const int n = min(KT, nk - tile * KT);
-        float s = -INFINITY;
-        if (lane < n) {
-            const uint4 *kr = reinterpret_cast<const uint4 *>(keys + (size_t)lane * row16 * 16);
-            const float *q = qs + (size_t)warp * CS;
+        {
+            const int k = half * 16 + (lane >> 1), par = lane & 1;
             float a = 0.0f, b = 0.0f;
-            int c = 0;
-            for (; c + 1 < S; c += 2) { a += El::dot(kr[c], q + c * E); b += El::dot(kr[c + 1], q + (c + 1) * E); }
-            if (c < S) a += El::dot(kr[c], q + c * E);
-            s = a + b;
+            if (k < n && h < p.heads) {
+                const uint4 *kr = reinterpret_cast<const uint4 *>(keys + (size_t)k * row16 * 16);
+                const float *q = qs + (size_t)hi * CS;
+                int c = par;
+#pragma unroll 2
+                for (; c + 2 < S; c += 4) { a += El::dot(kr[c], q + c * E); b += El::dot(kr[c + 2], q + (c + 2) * E); }
+                if (c < S) a += El::dot(kr[c], q + c * E);
+            }
+            a += b;
+            a += __shfl_xor_sync(0xffffffffu, a, 1);
+            if (par == 0) ssh[hi][k] = k < n ? a : -INFINITY;
         }
+        __syncthreads();
+        const float s = ssh[hi][lane];
         const float mt = fmaxf(m, warp_max(s));
         const float w = lane < n ? expf(s - mt) : 0.0f;
         const float corr = m == -INFINITY ? 0.0f : expf(m - mt);
@@ -200,14 +252,15 @@ __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constan
         for (int c = 0; c < NCH; ++c)
 #pragma unroll
             for (int e = 0; e < E; ++e) acc[c][e] *= corr;
+#pragma unroll 4
         for (int j = 0; j < n; ++j) {
             const float wj = __shfl_sync(0xffffffffu, w, j);
 #pragma unroll
             for (int c = 0; c < NCH; ++c) {
-                const int col = (c * 32 + lane) * E;
-                if (col < R8) {
+                const int sl = (2 * c + half) * 32 + lane;
+                if (sl * E < R8) {
                     float v[E];
-                    El::unpack(*reinterpret_cast<const uint4 *>(keys + ((size_t)j * row16 + c * 32 + lane) * 16), v);
+                    El::unpack(*reinterpret_cast<const uint4 *>(keys + ((size_t)j * row16 + sl) * 16), v);
 #pragma unroll
                     for (int e = 0; e < E; ++e) acc[c][e] = fmaf(wj, v[e], acc[c][e]);
                 }
@@ -218,23 +271,23 @@ __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constan
     float *part = p.d_part + ((size_t)h * p.n_split + split) * PS;
 #pragma unroll
     for (int c = 0; c < NCH; ++c) {
-        const int col = (c * 32 + lane) * E;
+        const int col = ((2 * c + half) * 32 + lane) * E;
         if (col < R8)
 #pragma unroll
             for (int e = 0; e < E; e += 4)
                 *reinterpret_cast<float4 *>(part + col + e) = make_float4(acc[c][e], acc[c][e + 1], acc[c][e + 2], acc[c][e + 3]);
     }
-    if (lane == 0) { part[R8] = m; part[R8 + 1] = l; }
+    if (half == 0 && lane == 0) { part[R8] = m; part[R8 + 1] = l; }
 }
 
 template <int WT>
-__global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant__ b200_latent_args p, int chunks)
+__global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant__ b200_latent_args p, int chunks, int sgroups)
 {
     using El = Elem<WT>;
     using T = typename El::T;
-    constexpr int E = El::E, RPW = VALUE_ROWS / 8, NS = 2;
+    constexpr int E = El::E, RPW = VALUE_ROWS / 8, NS = 2, BATCH = 16;
     extern __shared__ __align__(16) unsigned char smem[];
-    float *olat = reinterpret_cast<float *>(smem);           // [up8(kv_rank)]
+    float *olat = reinterpret_cast<float *>(smem);           // [sgroups][up8(kv_rank)]
     __shared__ float sw[MAX_SPLITS];
     pdl_launch_dependents();
     const int R8 = up8(p.kv_rank), PS = R8 + 8, S = R8 / E;
@@ -251,43 +304,90 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant
                                                            : make_uint4(0, 0, 0, 0);
     pdl_wait();
     const float *part = p.d_part + (size_t)h * p.n_split * PS;
+    const float gate = lane < RPW && v0 + lane < p.vdim ? p.d_gate[h * p.vdim + v0 + lane] : 0.0f;
+    // A thread sums four columns over every sgroups-th split. Its first loads are in flight while warp 0 turns the
+    // splits' maxima and totals into weights.
+    const int cg = R8 / 4, col4 = (int)threadIdx.x % cg, sg = (int)threadIdx.x / cg;
+    float4 held[BATCH];
+    if (sg < sgroups)
+#pragma unroll
+        for (int i = 0; i < BATCH; ++i) {
+            const int s = sg + i * sgroups;
+            held[i] = s < p.n_split ? *reinterpret_cast<const float4 *>(part + (size_t)s * PS + 4 * col4) : make_float4(0, 0, 0, 0);
+        }
     if (warp == 0) {
-        float m = -INFINITY, l = 0.0f;
-        for (int s = lane; s < p.n_split; s += 32) m = fmaxf(m, part[(size_t)s * PS + R8]);
+        float m = -INFINITY, l = 0.0f, ms[MAX_SPLITS / 32], ls[MAX_SPLITS / 32];
+#pragma unroll
+        for (int i = 0; i < MAX_SPLITS / 32; ++i) {
+            const int s = lane + 32 * i;
+            ms[i] = s < p.n_split ? part[(size_t)s * PS + R8] : -INFINITY;
+            ls[i] = s < p.n_split ? part[(size_t)s * PS + R8 + 1] : 0.0f;
+            m = fmaxf(m, ms[i]);
+        }
         m = warp_max(m);
-        for (int s = lane; s < p.n_split; s += 32) {
-            const float ls = part[(size_t)s * PS + R8 + 1];
-            const float e = ls > 0.0f ? expf(part[(size_t)s * PS + R8] - m) : 0.0f;
-            sw[s] = e;
-            l = fmaf(e, ls, l);
+#pragma unroll
+        for (int i = 0; i < MAX_SPLITS / 32; ++i) {
+            ms[i] = ls[i] > 0.0f ? expf(ms[i] - m) : 0.0f;
+            l = fmaf(ms[i], ls[i], l);
         }
         l = warp_sum(l);
         const float inv = l > 0.0f ? 1.0f / l : 0.0f;
-        for (int s = lane; s < p.n_split; s += 32) sw[s] *= inv;
+#pragma unroll
+        for (int i = 0; i < MAX_SPLITS / 32; ++i)
+            if (lane + 32 * i < p.n_split) sw[lane + 32 * i] = ms[i] * inv;
     }
     __syncthreads();
-    for (int r = threadIdx.x; r < R8; r += 256) {
-        float a = 0.0f;
+    if (sg < sgroups)
+        for (int c4 = col4; c4 < cg; c4 += 256) {            // a second trip only where a row is wider than 1024
+            float4 a = make_float4(0, 0, 0, 0);
+            int s = sg;
+            if (c4 == col4) {
+#pragma unroll
+                for (int i = 0; i < BATCH; ++i, s += sgroups) {
+                    const float f = s < p.n_split ? sw[s] : 0.0f;
+                    a.x = fmaf(f, held[i].x, a.x); a.y = fmaf(f, held[i].y, a.y); a.z = fmaf(f, held[i].z, a.z); a.w = fmaf(f, held[i].w, a.w);
+                }
+            }
 #pragma unroll 8
-        for (int s = 0; s < p.n_split; ++s) a = fmaf(sw[s], part[(size_t)s * PS + r], a);
-        olat[r] = a;
-    }
+            for (; s < p.n_split; s += sgroups) {
+                const float f = sw[s];
+                const float4 v = *reinterpret_cast<const float4 *>(part + (size_t)s * PS + 4 * c4);
+                a.x = fmaf(f, v.x, a.x); a.y = fmaf(f, v.y, a.y); a.z = fmaf(f, v.z, a.z); a.w = fmaf(f, v.w, a.w);
+            }
+            *reinterpret_cast<float4 *>(olat + (size_t)sg * R8 + 4 * c4) = a;
+        }
     __syncthreads();
+    if (sgroups > 1) {
+        for (int r = threadIdx.x; r < R8; r += 256) {
+            float a = olat[r];
+            for (int g = 1; g < sgroups; ++g) a += olat[(size_t)g * R8 + r];
+            olat[r] = a;                                     // this thread alone reads and writes column r
+        }
+        __syncthreads();
+    }
+    float y[RPW];
+#pragma unroll
+    for (int k = 0; k < RPW; ++k) y[k] = 0.0f;
+#pragma unroll
+    for (int s = 0; s < NS; ++s)
+        if (s * 32 + lane < S) {
+            float x[E];
+#pragma unroll
+            for (int e = 0; e < E; e += 4) *reinterpret_cast<float4 *>(x + e) = *reinterpret_cast<const float4 *>(olat + (s * 32 + lane) * E + e);
+#pragma unroll
+            for (int k = 0; k < RPW; ++k) y[k] += El::dot(w[k][s], x);
+        }
+    for (int c = NS * 32 + lane; c < S; c += 32)
+#pragma unroll
+        for (int k = 0; k < RPW; ++k)
+            if (v0 + k < p.vdim) y[k] += El::dot(*reinterpret_cast<const uint4 *>(w0 + (size_t)(v0 + k) * R8 + (size_t)c * E), olat + c * E);
+    float mine = 0.0f;
 #pragma unroll
     for (int k = 0; k < RPW; ++k) {
-        if (v0 + k >= p.vdim) break;                         // uniform across the warp
-        float a = 0.0f;
-#pragma unroll
-        for (int s = 0; s < NS; ++s)
-            if (s * 32 + lane < S) a += El::dot(w[k][s], olat + (s * 32 + lane) * E);
-        for (int c = NS * 32 + lane; c < S; c += 32)
-            a += El::dot(*reinterpret_cast<const uint4 *>(w0 + (size_t)(v0 + k) * R8 + (size_t)c * E), olat + c * E);
-        a = warp_sum(a);
-        if (lane == 0) {
-            const int o = h * p.vdim + v0 + k;
-            p.d_out[o] = a * sigmoid_f32(p.d_gate[o]);
-        }
+        const float t = warp_sum(y[k]);
+        if (lane == k) mine = t;
     }
+    if (lane < RPW && v0 + lane < p.vdim) p.d_out[h * p.vdim + v0 + lane] = mine * sigmoid_f32(gate);
 }
 
 // ------------------------------------------------------------------------------------------------ rows
@@ -298,7 +398,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const __grid_constant_
     using T = typename Elem<WT>::T;
     __shared__ float red[33];
     const int m = blockIdx.x, pos = p.pos0 + m;
-    write_cache_row<T>(p, p.d_dkv + (size_t)m * p.proj_ld, pos, red);
+    write_cache_row<T>(p, p.d_dkv + (size_t)m * p.proj_ld, pos, red, [] {});
     const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), dq = p.dim + p.rot_dim, QS = dim8 + rot8;
     const float *q = p.d_q + (size_t)m * p.proj_ld;
     const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
@@ -373,11 +473,6 @@ __global__ void __launch_bounds__(128) latent_attend_f32_kernel(const __grid_con
 // next tile's copies in flight under the current one. DV value columns per blockIdx.z.
 constexpr int BQ = 64, BKEY = 64;
 
-__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool on)
-{
-    const int n = on ? 16 : 0;                               // 0: the 16 bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
 __device__ __forceinline__ void ldsm4(uint32_t a, uint32_t (&r)[4])
 {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -441,7 +536,7 @@ __global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_co
             const bool on = kp <= last && c0 + c * 8 < vd8;
             cp16(smem_u32(vd + (size_t)r * VS + c * 8), on ? kv + (size_t)(kp - p.kv_row0) * p.kv_ld + dim8 + c0 + c * 8 : kv, on);
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        cp_commit();
     };
     stage(0, 0);
 
@@ -462,9 +557,9 @@ __global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_co
         const int slot = stages == 2 ? tile & 1 : 0;
         if (stages == 2 && tile + 1 < tiles) {
             stage(tile + 1, slot ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
+            cp_wait<1>();
         } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
+            cp_wait<0>();
         }
         __syncthreads();
         const __nv_bfloat16 *kd = ksm + (size_t)slot * BKEY * dqs, *vd = vsm + (size_t)slot * BKEY * VS;
@@ -563,12 +658,13 @@ bool shape_ok(const b200_latent_args *a)
            a->d_q && a->d_dkv && a->d_dkv_gamma && a->d_rope && a->d_cache;
 }
 
-template <typename K>
-int launch_pdl(K kern, int gx, int gy, int threads, size_t smem, int pdl, cudaStream_t st, const b200_latent_args &a, int i0)
+// 256 threads, chained to the previous launch when pdl is set
+template <typename K, typename... Args>
+int launch_pdl(K kern, int gx, int gy, size_t smem, int pdl, cudaStream_t st, Args... args)
 {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(gx, gy);
-    cfg.blockDim = dim3(threads);
+    cfg.blockDim = dim3(256);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = st;
     cudaLaunchAttribute attr[1];
@@ -577,7 +673,7 @@ int launch_pdl(K kern, int gx, int gy, int threads, size_t smem, int pdl, cudaSt
     cfg.attrs = attr;
     cfg.numAttrs = pdl ? 1 : 0;
     ++g_b200_launches;
-    return (int)cudaLaunchKernelEx(&cfg, kern, a, i0);
+    return (int)cudaLaunchKernelEx(&cfg, kern, args...);
 }
 
 template <typename K>
@@ -596,36 +692,27 @@ int decode(const b200_latent_args &a, cudaStream_t st)
     while (lpr < 32 && lpr * E < dim8) lpr <<= 1;
     const int rows_per_block = ABSORB_PASSES * 8 * (32 / lpr);
     const int chunks = (a.kv_rank + rows_per_block - 1) / rows_per_block;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(a.heads * chunks + 1);
-    cfg.blockDim = dim3(256);
-    cfg.stream = st;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = a.use_pdl ? 1 : 0;
-    ++g_b200_launches;
-    int rc = (int)cudaLaunchKernelEx(&cfg, latent_absorb_kernel<WT>, a, chunks, lpr);
+    int rc = launch_pdl(latent_absorb_kernel<WT>, a.heads * chunks + 1, 1, 0, a.use_pdl, st, a, chunks, lpr);
     if (rc) return rc;
 
-    const int row16 = (CS / E) | 1;
+    int row16 = CS / E;                                      // 2 mod 4: four keys x two slices touch different banks
+    while (row16 % 4 != 2) ++row16;
     const size_t smem = (size_t)KT * row16 * 16 + (size_t)HB * CS * 4;
-    const int hb = (a.heads + HB - 1) / HB, nch = (R8 + 32 * E - 1) / (32 * E);
+    const int hb = (a.heads + HB - 1) / HB, nch = (R8 + 64 * E - 1) / (64 * E);
 #define SCORES(N)                                                                             \
     do {                                                                                      \
         if ((rc = allow_smem(latent_scores_kernel<WT, N>, smem)) != 0) return rc;              \
-        rc = launch_pdl(latent_scores_kernel<WT, N>, a.n_split, hb, 256, smem, a.use_pdl, st, a, row16); \
+        rc = launch_pdl(latent_scores_kernel<WT, N>, a.n_split, hb, smem, a.use_pdl, st, a, row16); \
     } while (0)
     if (nch <= 1) SCORES(1);
     else if (nch <= 2) SCORES(2);
     else if (nch <= 4) SCORES(4);
-    else if (nch <= 8) SCORES(8);
     else return B200_E_TOOLARGE;
 #undef SCORES
     if (rc) return rc;
     const int vchunks = (a.vdim + VALUE_ROWS - 1) / VALUE_ROWS;
-    return launch_pdl(latent_value_kernel<WT>, a.heads * vchunks, 1, 256, (size_t)R8 * 4, a.use_pdl, st, a, vchunks);
+    const int sgroups = R8 / 4 >= 256 ? 1 : 256 / (R8 / 4) < a.n_split ? 256 / (R8 / 4) : a.n_split;
+    return launch_pdl(latent_value_kernel<WT>, a.heads * vchunks, 1, (size_t)sgroups * R8 * 4, a.use_pdl, st, a, vchunks, sgroups);
 }
 
 template <int DV>
