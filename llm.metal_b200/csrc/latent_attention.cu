@@ -469,10 +469,16 @@ __global__ void __launch_bounds__(128) latent_attend_f32_kernel(const __grid_con
     }
 }
 
-// bfloat16 on the tensor cores. A block: 64 query rows of one head, four warps of 16 rows; keys 64 at a time, the
-// next tile's copies in flight under the current one. DV value columns per blockIdx.z.
-constexpr int BQ = 64, BKEY = 64;
+// bfloat16 on the tensor cores. A block: NW warps of 16 query rows of one head; keys 32 at a time, the next tile's
+// copies in flight under the current one. DV value columns per blockIdx.z.
+constexpr int BKEY = 32;
 
+__device__ __forceinline__ float ex2(float x)                // 2^x, 2 ulp, 0 for -inf
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ void ldsm4(uint32_t a, uint32_t (&r)[4])
 {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
@@ -492,12 +498,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi)
     return *reinterpret_cast<const uint32_t *>(&h);
 }
 
-template <int DV>
-__global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_constant__ b200_latent_args p, int dqs, int stages)
+template <int DV, int NW>
+__global__ void __launch_bounds__(NW * 32, 16 / NW) latent_attend_bf16_kernel(const __grid_constant__ b200_latent_args p, int dqs, int stages)
 {
     // dqs: elements of a query / key row in shared memory; its first dqs - 8 are multiples of 16 and hold
     // [unrotated | rotated | zeros]. Rows are 16 bytes off a multiple of 32: ldmatrix is conflict-free.
-    constexpr int VS = DV + 8;
+    constexpr int VS = DV + 8, BQ = NW * 16, NT = NW * 32;
     extern __shared__ __align__(16) unsigned char smem[];
     const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), QS = dim8 + rot8, vd8 = up8(p.vdim), R8 = up8(p.kv_rank), CS = R8 + rot8;
     const int dqk = dqs - 8;
@@ -514,27 +520,35 @@ __global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_co
     const int first = p.pos0 + m0, last = first + rows - 1;  // absolute positions of this block's queries
     const int lo = p.window > 0 && first - p.window + 1 > 0 ? first - p.window + 1 : 0;
     const int tiles = (last - lo) / BKEY + 1;
-    const int sq = dqk / 8, sv = DV / 8;
+    const int sq = dqk / 8;
+    constexpr int SV = DV / 8;
+    // 16-byte chunks of a [rows][sq] tile go round the threads: (row, chunk) of this thread and its step, no divisions
+    const int r_first = tid / sq, c_first = tid % sq, r_step = NT / sq, c_step = NT % sq;
 
-    for (int i = tid; i < BQ * sq; i += 128) {
-        const int r = i / sq, c = i % sq;
+    for (int r = r_first, c = c_first; r < BQ;) {
         const bool on = r < rows && c * 8 < QS;
-        cp16(smem_u32(qsm + (size_t)r * dqs + c * 8), on ? qg + (size_t)r * p.heads * QS + c * 8 : qg, on);
+        cp16(smem_u32(qsm + r * dqs + c * 8), on ? qg + (size_t)r * p.heads * QS + c * 8 : qg, on);
+        r += r_step; c += c_step;
+        if (c >= sq) { c -= sq; ++r; }
     }
     auto stage = [&](int tile, int slot) {
-        __nv_bfloat16 *kd = ksm + (size_t)slot * BKEY * dqs, *vd = vsm + (size_t)slot * BKEY * VS;
-        const int k0 = lo + tile * BKEY;
-        for (int i = tid; i < BKEY * sq; i += 128) {
-            const int r = i / sq, c = i % sq, kp = k0 + r;
-            const bool on = kp <= last && c * 8 < QS;
-            const __nv_bfloat16 *src = !on ? kv : c * 8 < dim8 ? kv + (size_t)(kp - p.kv_row0) * p.kv_ld + c * 8
-                                                               : cache + (size_t)kp * CS + R8 + (c * 8 - dim8);
-            cp16(smem_u32(kd + (size_t)r * dqs + c * 8), src, on);
+        const uint32_t kd = smem_u32(ksm + slot * BKEY * dqs), vd = smem_u32(vsm + slot * BKEY * VS);
+        const int k0 = lo + tile * BKEY, n = last - k0;      // rows past n hold zeros
+        const __nv_bfloat16 *kvt = kv + (long long)(k0 - p.kv_row0) * p.kv_ld, *crt = cache + (long long)k0 * CS + (R8 - dim8);
+        for (int r = r_first, c = c_first; r < BKEY;) {
+            const bool on = r <= n && c * 8 < QS;
+            const __nv_bfloat16 *src = c * 8 < dim8 ? kvt + (long long)r * p.kv_ld : crt + r * CS;
+            cp16(kd + (r * dqs + c * 8) * 2, on ? src + c * 8 : kv, on);
+            r += r_step; c += c_step;
+            if (c >= sq) { c -= sq; ++r; }
         }
-        for (int i = tid; i < BKEY * sv; i += 128) {
-            const int r = i / sv, c = i % sv, kp = k0 + r;
-            const bool on = kp <= last && c0 + c * 8 < vd8;
-            cp16(smem_u32(vd + (size_t)r * VS + c * 8), on ? kv + (size_t)(kp - p.kv_row0) * p.kv_ld + dim8 + c0 + c * 8 : kv, on);
+#pragma unroll
+        for (int i = 0; i < (BKEY * SV + NT - 1) / NT; ++i) {
+            const int e = tid + i * NT, r = e / SV, c = e % SV;
+            if (BKEY * SV % NT == 0 || r < BKEY) {
+                const bool on = r <= n && c0 + c * 8 < vd8;
+                cp16(vd + (r * VS + c * 8) * 2, on ? kvt + (long long)r * p.kv_ld + dim8 + c0 + c * 8 : kv, on);
+            }
         }
         cp_commit();
     };
@@ -545,13 +559,11 @@ __global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_co
     for (int i = 0; i < DV / 8; ++i)
 #pragma unroll
         for (int k = 0; k < 4; ++k) o[i][k] = 0.0f;
-    float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+    float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};      // maxima of the unscaled scores
     // this thread's rows: r0 and r0 + 8 of the warp's 16
     const int r0 = warp * 16 + (lane >> 2);
-    const int qpos[2] = {first + r0, first + r0 + 8};
-    const uint32_t qaddr = smem_u32(qsm + (size_t)(warp * 16 + (lane & 15)) * dqs + (lane >> 4) * 8);
-    const float LOG2E = 1.4426950408889634f;
-    const float sc = p.scale * LOG2E;
+    const uint32_t qaddr = smem_u32(qsm + (warp * 16 + (lane & 15)) * dqs + (lane >> 4) * 8);
+    const float sc = p.scale * 1.4426950408889634f;          // weights as powers of two
 
     for (int tile = 0; tile < tiles; ++tile) {
         const int slot = stages == 2 ? tile & 1 : 0;
@@ -562,68 +574,86 @@ __global__ void __launch_bounds__(128) latent_attend_bf16_kernel(const __grid_co
             cp_wait<0>();
         }
         __syncthreads();
-        const __nv_bfloat16 *kd = ksm + (size_t)slot * BKEY * dqs, *vd = vsm + (size_t)slot * BKEY * VS;
-        float s[BKEY / 8][4];
-#pragma unroll
-        for (int i = 0; i < BKEY / 8; ++i)
-#pragma unroll
-            for (int k = 0; k < 4; ++k) s[i][k] = 0.0f;
-        // key rows as the B operand: matrices (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
-        const uint32_t kaddr = smem_u32(kd + (size_t)((lane & 7) + ((lane >> 4) << 3)) * dqs + ((lane >> 3) & 1) * 8);
-        for (int kk = 0; kk < dqk; kk += 16) {
-            uint32_t a[4];
-            ldsm4(qaddr + kk * 2, a);
-#pragma unroll
-            for (int n = 0; n < BKEY / 16; ++n) {
-                uint32_t b[4];
-                ldsm4(kaddr + (uint32_t)(n * 16 * dqs + kk) * 2, b);
-                mma_bf16(s[2 * n], a, b[0], b[1]);
-                mma_bf16(s[2 * n + 1], a, b[2], b[3]);
-            }
-        }
         const int k0 = lo + tile * BKEY;
-        float mt[2] = {mx[0], mx[1]};
+        // the warp's queries see nothing of this tile: all of it is ahead of them, or has left their windows
+        const int w_first = first + warp * 16, w_last = w_first + 15;
+        const bool idle = k0 > w_last || (p.window > 0 && w_first - (k0 + BKEY - 1) >= p.window);
+        if (!idle) {
+            float s[BKEY / 8][4];
 #pragma unroll
-        for (int n = 0; n < BKEY / 8; ++n)
+            for (int i = 0; i < BKEY / 8; ++i)
 #pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                const int kp = k0 + n * 8 + (lane & 3) * 2 + (k & 1), d = qpos[k >> 1] - kp;
-                s[n][k] = d >= 0 && (p.window <= 0 || d < p.window) ? s[n][k] * sc : -INFINITY;
-                mt[k >> 1] = fmaxf(mt[k >> 1], s[n][k]);
+                for (int k = 0; k < 4; ++k) s[i][k] = 0.0f;
+            // key rows as the B operand: matrices (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
+            const uint32_t kaddr = smem_u32(ksm + slot * BKEY * dqs + ((lane & 7) + ((lane >> 4) << 3)) * dqs + ((lane >> 3) & 1) * 8);
+#pragma unroll 4
+            for (int kk = 0; kk < dqk; kk += 16) {
+                uint32_t a[4];
+                ldsm4(qaddr + kk * 2, a);
+#pragma unroll
+                for (int n = 0; n < BKEY / 16; ++n) {
+                    uint32_t b[4];
+                    ldsm4(kaddr + (uint32_t)(n * 16 * dqs + kk) * 2, b);
+                    mma_bf16(s[2 * n], a, b[0], b[1]);
+                    mma_bf16(s[2 * n + 1], a, b[2], b[3]);
+                }
+            }
+            // only tiles at an edge of the warp's visible range need the mask
+            if (k0 + BKEY - 1 > w_first || (p.window > 0 && w_last - k0 >= p.window)) {
+                const int span = p.window > 0 ? p.window : 0x7fffffff;
+                const int d0 = first + r0 - k0 - (lane & 3) * 2;
+#pragma unroll
+                for (int n = 0; n < BKEY / 8; ++n)
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const int d = d0 + (k >> 1) * 8 - n * 8 - (k & 1);
+                        if (d < 0 || d >= span) s[n][k] = -INFINITY;
+                    }
+            }
+            float mt[2] = {mx[0], mx[1]};
+#pragma unroll
+            for (int n = 0; n < BKEY / 8; ++n) {
+                mt[0] = fmaxf(mt[0], fmaxf(s[n][0], s[n][1]));
+                mt[1] = fmaxf(mt[1], fmaxf(s[n][2], s[n][3]));
             }
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 1));
-            mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 2));
-        }
-        // a row with nothing visible so far keeps its maximum at -inf: its weights and its correction are zero
-        const float base[2] = {mt[0] == -INFINITY ? 0.0f : mt[0], mt[1] == -INFINITY ? 0.0f : mt[1]};
-        const float corr[2] = {exp2f(mx[0] - base[0]), exp2f(mx[1] - base[1])};
-        mx[0] = mt[0]; mx[1] = mt[1];
-        float ls[2] = {0.0f, 0.0f};
-#pragma unroll
-        for (int n = 0; n < BKEY / 8; ++n)
-#pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                s[n][k] = exp2f(s[n][k] - base[k >> 1]);
-                ls[k >> 1] += s[n][k];
+            for (int r = 0; r < 2; ++r) {
+                mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 1));
+                mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 2));
             }
-        l[0] = l[0] * corr[0] + ls[0];
-        l[1] = l[1] * corr[1] + ls[1];
+            // a row with nothing visible so far keeps its maximum at -inf: its weights and its correction are zero
+            // (differences first: the score at the maximum then weighs exactly one, whatever its size)
+            const float base[2] = {mt[0] == -INFINITY ? 0.0f : mt[0], mt[1] == -INFINITY ? 0.0f : mt[1]};
+            const float corr[2] = {ex2((mx[0] - base[0]) * sc), ex2((mx[1] - base[1]) * sc)};
+            const bool moved = mt[0] != mx[0] || mt[1] != mx[1];
+            mx[0] = mt[0]; mx[1] = mt[1];
+            float ls[2] = {0.0f, 0.0f};
 #pragma unroll
-        for (int i = 0; i < DV / 8; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
-        // value rows as the B operand, transposed on load: (k 0-7, cols 0-7), (k 8-15, cols 0-7), (k 0-7, cols 8-15), ...
-        const uint32_t vaddr = smem_u32(vd + (size_t)(lane & 15) * VS + (lane >> 4) * 8);
+            for (int n = 0; n < BKEY / 8; ++n)
 #pragma unroll
-        for (int kk = 0; kk < BKEY / 16; ++kk) {
-            const uint32_t a[4] = {pack_bf16(s[2 * kk][0], s[2 * kk][1]), pack_bf16(s[2 * kk][2], s[2 * kk][3]),
-                                   pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+                for (int k = 0; k < 4; ++k) {
+                    s[n][k] = ex2((s[n][k] - base[k >> 1]) * sc);
+                    ls[k >> 1] += s[n][k];
+                }
+            l[0] = fmaf(l[0], corr[0], ls[0]);
+            l[1] = fmaf(l[1], corr[1], ls[1]);
+            if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
-            for (int n = 0; n < DV / 16; ++n) {
-                uint32_t b[4];
-                ldsm4_t(vaddr + (uint32_t)(kk * 16 * VS + n * 16) * 2, b);
-                mma_bf16(o[2 * n], a, b[0], b[1]);
-                mma_bf16(o[2 * n + 1], a, b[2], b[3]);
+                for (int i = 0; i < DV / 8; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+            }
+            // value rows as the B operand, transposed on load: (k 0-7, cols 0-7), (k 8-15, cols 0-7), (k 0-7, cols 8-15), ...
+            const uint32_t vaddr = smem_u32(vsm + slot * BKEY * VS + (lane & 15) * VS + (lane >> 4) * 8);
+#pragma unroll
+            for (int kk = 0; kk < BKEY / 16; ++kk) {
+                const uint32_t a[4] = {pack_bf16(s[2 * kk][0], s[2 * kk][1]), pack_bf16(s[2 * kk][2], s[2 * kk][3]),
+                                       pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+#pragma unroll
+                for (int n = 0; n < DV / 16; ++n) {
+                    uint32_t b[4];
+                    ldsm4_t(vaddr + (uint32_t)(kk * 16 * VS + n * 16) * 2, b);
+                    mma_bf16(o[2 * n], a, b[0], b[1]);
+                    mma_bf16(o[2 * n + 1], a, b[2], b[3]);
+                }
             }
         }
         __syncthreads();                                     // the slot is overwritten by the next round's copies
@@ -715,19 +745,26 @@ int decode(const b200_latent_args &a, cudaStream_t st)
     return launch_pdl(latent_value_kernel<WT>, a.heads * vchunks, 1, (size_t)sgroups * R8 * 4, a.use_pdl, st, a, vchunks, sgroups);
 }
 
-template <int DV>
+template <int DV, int NW>
 int attend_bf16(const b200_latent_args &a, cudaStream_t st)
 {
     const int dqk = (up8(a.dim) + up8(a.rot_dim) + 15) / 16 * 16, dqs = dqk + 8;
     int stages = 2;
-    auto bytes = [&](int s) { return ((size_t)(BQ + s * BKEY) * dqs + (size_t)s * BKEY * (DV + 8)) * 2; };
+    auto bytes = [&](int s) { return ((size_t)(NW * 16 + s * BKEY) * dqs + (size_t)s * BKEY * (DV + 8)) * 2; };
     if (bytes(2) > 227 * 1024) stages = 1;
-    int rc = allow_smem(latent_attend_bf16_kernel<DV>, bytes(stages));
+    int rc = allow_smem(latent_attend_bf16_kernel<DV, NW>, bytes(stages));
     if (rc) return rc;
-    const dim3 grid((a.n_rows + BQ - 1) / BQ, a.heads, (a.vdim + DV - 1) / DV);
-    latent_attend_bf16_kernel<DV><<<grid, 128, bytes(stages), st>>>(a, dqs, stages);
+    const dim3 grid((a.n_rows + NW * 16 - 1) / (NW * 16), a.heads, (a.vdim + DV - 1) / DV);
+    latent_attend_bf16_kernel<DV, NW><<<grid, NW * 32, bytes(stages), st>>>(a, dqs, stages);
     ++g_b200_launches;
     return (int)cudaGetLastError();
+}
+
+// 128 query rows a block where that still fills the machine (a tile of keys serves twice the rows), 64 otherwise
+template <int DV>
+int attend_bf16(const b200_latent_args &a, cudaStream_t st)
+{
+    return (long long)((a.n_rows + 127) / 128) * a.heads >= 148 ? attend_bf16<DV, 8>(a, st) : attend_bf16<DV, 4>(a, st);
 }
 
 }  // namespace
