@@ -403,13 +403,29 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const __grid_constant_
     const float *q = p.d_q + (size_t)m * p.proj_ld;
     const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
     T *out = static_cast<T *>(p.d_q_rows) + (size_t)m * p.heads * QS;
-    for (int i = threadIdx.x; i < p.heads * QS; i += blockDim.x) {
-        const int h = i / QS, e = i % QS;
+    // a warp per head, two elements (one rotated pair) per lane
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int h = warp; h < p.heads; h += 8) {
         const float *qh = q + (size_t)h * dq;
-        float v = 0.0f;
-        if (e < p.dim) v = qh[e];
-        else if (e >= dim8 && e - dim8 < p.rot_dim) v = rotated(qh + p.dim, e - dim8, p.rot_dims, rope);
-        out[i] = (T)v;
+        for (int e = 2 * lane; e < QS; e += 64) {
+            float v[2];
+            if (e < dim8) {
+                v[0] = e < p.dim ? qh[e] : 0.0f;
+                v[1] = e + 1 < p.dim ? qh[e + 1] : 0.0f;
+            } else {
+                const int r = e - dim8;
+                v[0] = r < p.rot_dim ? qh[p.dim + r] : 0.0f;
+                v[1] = r + 1 < p.rot_dim ? qh[p.dim + r + 1] : 0.0f;
+                if (r < p.rot_dims) {
+                    const float c = rope[r], s = rope[r + 1], x = v[0], y = v[1];
+                    v[0] = x * c - y * s;
+                    v[1] = y * c + x * s;
+                }
+            }
+            T *o = out + (size_t)h * QS + e;
+            if constexpr (WT == B200_WT_BF16) *reinterpret_cast<__nv_bfloat162 *>(o) = __floats2bfloat162_rn(v[0], v[1]);
+            else *reinterpret_cast<float2 *>(o) = make_float2(v[0], v[1]);
+        }
     }
 }
 

@@ -18,6 +18,8 @@ CONFIGS = {
     "narrow": o.model_config(64, 96, [L(1, 16, 8, 24, 24, 1, 48), L(1, 8, 16, 8, 40, 300, 80)], groups=1, alpha=1.0, cap=30.0),
     # more heads than one block of the decode scores holds; latent and value sizes beyond one pass
     "wide": o.model_config(320, 520, [L(18, 40, 24, 72, 300, 150, 256), L(9, 64, 32, 136, 96, 33, 200)], groups=5, alpha=3.5, emb_scale=6.0),
+    # smaller than every tile and than the narrowest tensor-core product
+    "tiny": o.model_config(24, 30, [L(1, 4, 2, 3, 5, 6, 10), L(2, 3, 4, 1, 8, 33, 9, base=30.0)], groups=4, emb_scale=1.0, alpha=2.0, cap=5.0),
     # the last layer has no feed-forward
     "bare-end": o.model_config(80, 136, [L(4, 16, 16, 16, 32, 50, 96, base=1000.0), L(4, 24, 8, 32, 48, 64, None)], groups=2),
 }

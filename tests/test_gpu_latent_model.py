@@ -137,6 +137,21 @@ def test_long_decoding(pkg, family):
         good(m, run(m, family["tokens"], [3]), family["want"])
 
 
+def test_a_prompt_longer_than_one_pass_of_the_row_path(pkg, tmp_path):
+    """2300 tokens: two passes inside one call, windows reaching across the cut; then decoding from there."""
+    config = o.model_config(48, 64, [T.L(2, 12, 4, 8, 16, 90, 40), T.L(1, 8, 8, 16, 24, 2200, None)], groups=2)
+    w = o.random_model(config, 31)
+    t = T.tokens(config, 2300, 6)
+    want, _ = o.forward(config, w, t)
+    folder = o.write_model(str(tmp_path / "m"), config, w)
+    places = [0, 1, 89, 90, 1000, 2046, 2047, 2048, 2049, 2136, 2137, 2138, 2199, 2200, 2280, 2289]
+    for dtype in DTYPES:
+        with pkg.DirModel(folder, 2300, dtype) as m:
+            got = np.array(m.feed(t[:2290], places), dtype=np.float64).reshape(len(places), -1)
+            tail = run(m, t, [], start=2290)
+            assert T.errors(np.concatenate([got, tail]), want[places + list(range(2290, 2300))]).max() <= T.LIMIT[dtype]
+
+
 # ------------------------------------------------------------------ generation
 
 def greedy(family, prompt, n):
