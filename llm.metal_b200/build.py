@@ -23,7 +23,7 @@ OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libllmb200.so")
 LIB_SYNTH = os.path.join(HERE, "libllmb200_synth.so")
 
-CU_SOURCES = ["pack.cu", "matvec.cu", "attention.cu", "decode_token.cu", "lora_decode.cu", "batch_kernels.cu", "gemm_f32.cu", "gemm_tf32.cu", "train_kernels.cu",
+CU_SOURCES = ["pack.cu", "matvec.cu", "matvec_ext.cu", "attention.cu", "decode_token.cu", "lora_decode.cu", "batch_kernels.cu", "gemm_f32.cu", "gemm_tf32.cu", "train_kernels.cu",
               "latent_attention.cu", "row_kernels.cu"]
 C_SOURCES = ["weights.c", "decode_engine.c", "sft_engine.c", "batch_engine.c", "json.c", "tensor_file.c", "model_dir.c", "latent_model.c"]
 
