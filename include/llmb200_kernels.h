@@ -225,7 +225,7 @@ int b200_attn_decode_static(const b200_attn_args *a, void *stream);
  * With up8(n) = n rounded up to a multiple of 8: a cache row is [up8(kv_rank) | up8(rot_dim)] elements of
  * the type `wtype` names (BF16 or F32), padding zero. d_w_uk_t: per head [kv_rank][up8(dim)] (the
  * transposed map). d_w_kv: per head up8(dim) rows of W_uk and up8(vdim) rows of W_uv, up8(kv_rank)
- * columns. All vectors of the decode form are fp32.
+ * columns. The decode form's vectors are fp32 but for d_qlat.
  *
  * Decode (b200_latent_decode, three launches): one new token at *d_pos. The query is moved into the latent
  * space (q_lat = W_uk^T q), the scores and the weighted sum run over cache rows with all heads sharing
@@ -243,7 +243,7 @@ typedef struct b200_latent_args {
     void *d_cache;
     const void *d_w_uk_t, *d_w_kv;
     /* decode */
-    float *d_qlat;                       /* [heads][up8(kv_rank) + up8(rot_dim)] */
+    void *d_qlat;                        /* [heads][up8(kv_rank) + up8(rot_dim)] elements of the type `wtype` names */
     float *d_part;                       /* [heads][n_split][up8(kv_rank) + 8] */
     float *d_out;                        /* [heads * vdim] */
     const int *d_pos;

@@ -4,9 +4,9 @@
 //   latent_absorb  per head q_lat = scale * W_uk^T q (the weight slice of a block is in registers before the
 //                  previous kernel has finished); one extra block normalises the new token's latent, rotates its
 //                  key part and the queries, and writes the cache row
-//   latent_scores  split-sequence attention in the latent space: a block takes 32 cache rows at a time for four
-//                  heads (two warps each), rows staged once in shared memory and used for the scores and for the
-//                  weighted sum; partial (sum, maximum, total) records per split
+//   latent_scores  split-sequence attention in the latent space: a block takes 32 cache rows at a time for sixteen
+//                  heads (bfloat16: tensor cores; fp32: four heads, CUDA cores), rows staged once in shared memory
+//                  and used for the scores and for the weighted sum; partial (sum, maximum, total) records per split
 //   latent_value   merges the splits of a head, applies W_uv and the output gate
 //
 // Prompt portions: latent_prep writes cache rows and rotated queries of all rows; keys and values are expanded
@@ -23,7 +23,8 @@ extern unsigned long long g_b200_launches;
 namespace {
 
 constexpr int KT = 32;             // cache rows per tile of the decode scores = lanes of a warp
-constexpr int HB = 4;              // heads per block of the decode scores, two warps each
+constexpr int HB = 4;              // heads per block of the fp32 decode scores, two warps each
+constexpr int HB_MMA = 16;         // heads per block of the bfloat16 decode scores: the rows of a tensor-core tile
 constexpr int ABSORB_PASSES = 4;   // row passes whose weights a warp of latent_absorb holds in registers
 constexpr int VALUE_ROWS = 16;     // value rows per block of latent_value, two per warp
 constexpr int MAX_SPLITS = 256;
@@ -143,10 +144,10 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
     for (int e = 0; e < E; ++e) x[e] = sl * E + e < p.dim ? q[sl * E + e] : 0.0f;
     // the head's first block also rotates its query and clears the padding columns of the latent part
     if (chunk == 0 && valid) {
-        float *ql = p.d_qlat + (size_t)h * CS;
+        T *ql = static_cast<T *>(p.d_qlat) + (size_t)h * CS;
         const float *rope = p.d_rope + (size_t)pos * p.rot_dims;
-        for (int i = threadIdx.x; i < rot8; i += 256) ql[R8 + i] = i < p.rot_dim ? p.scale * rotated(q + p.dim, i, p.rot_dims, rope) : 0.0f;
-        if ((int)threadIdx.x < R8 - R) ql[R + threadIdx.x] = 0.0f;
+        for (int i = threadIdx.x; i < rot8; i += 256) ql[R8 + i] = (T)(i < p.rot_dim ? p.scale * rotated(q + p.dim, i, p.rot_dims, rope) : 0.0f);
+        if ((int)threadIdx.x < R8 - R) ql[R + threadIdx.x] = (T)0.0f;
     }
 #pragma unroll
     for (int k = 0; k < ABSORB_PASSES; ++k) {
@@ -160,17 +161,17 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const __grid_constan
                 acc += El::dot(*reinterpret_cast<const uint4 *>(w0 + (size_t)row * dim8 + d), y);
             }
         for (int o = 1; o < lpr; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-        if (sl == 0 && row < R) p.d_qlat[(size_t)h * CS + row] = p.scale * acc;
+        if (sl == 0 && row < R) static_cast<T *>(p.d_qlat)[(size_t)h * CS + row] = (T)(p.scale * acc);
     }
 }
 
-// Two warps per head: warp 2i + f of head i scores the tile's keys 16 f .. 16 f + 15 (two lanes per key, every
+// fp32, on the CUDA cores. Two warps per head: warp 2i + f of head i scores the tile's keys 16 f .. 16 f + 15 (two lanes per key, every
 // other slice each) and sums the columns of half f (slices f, f + 2, ... of 32) of the weighted rows.
-template <int WT, int NCH>
-__global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constant__ b200_latent_args p, int row16)
+template <int NCH>
+__global__ void __launch_bounds__(256) latent_scores_f32_kernel(const __grid_constant__ b200_latent_args p, int row16)
 {
-    using El = Elem<WT>;
-    using T = typename El::T;
+    using El = Elem<B200_WT_F32>;
+    using T = float;
     constexpr int E = El::E;
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float ssh[HB][KT];
@@ -205,7 +206,7 @@ __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constan
     pdl_wait();
     {
         const int n = min(HB, p.heads - h0) * CS / 4;        // queries: contiguous fp32 rows
-        for (int i = threadIdx.x; i < n; i += 256) cp16(smem_u32(qs + 4 * i), p.d_qlat + (size_t)h0 * CS + 4 * i, true);
+        for (int i = threadIdx.x; i < n; i += 256) cp16(smem_u32(qs + 4 * i), static_cast<const float *>(p.d_qlat) + (size_t)h0 * CS + 4 * i, true);
         if (t0 < t1 && t1 == tiles && warp == 0) {           // the newest key is the last row of the last tile
             const int r = nk - 1 - (tiles - 1) * KT;
             if (tiles - 1 == t0) stage_row(r, pos);
@@ -278,6 +279,163 @@ __global__ void __launch_bounds__(256) latent_scores_kernel(const __grid_constan
                 *reinterpret_cast<float4 *>(part + col + e) = make_float4(acc[c][e], acc[c][e + 1], acc[c][e + 2], acc[c][e + 3]);
     }
     if (half == 0 && lane == 0) { part[R8] = m; part[R8 + 1] = l; }
+}
+
+__device__ __forceinline__ void ldsm4(uint32_t a, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t a, uint32_t (&r)[4])
+{
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
+{
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi)
+{
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t *>(&h);
+}
+
+// bfloat16, on the tensor cores: sixteen heads are the rows of both products, so a cache row is read from shared
+// memory once per sixteen heads. Warp w scores keys 8 (w & 3) .. + 7 over half w >> 2 of the columns, keeps the
+// softmax state of heads 2 w and 2 w + 1, and sums NTW tiles of eight latent columns of the weighted rows. Two tiles
+// of keys in shared memory, the next one's copies under the current one.
+template <int NTW>
+__global__ void __launch_bounds__(256) latent_scores_bf16_kernel(const __grid_constant__ b200_latent_args p, int row16)
+{
+    constexpr int PST = KT + 8;                              // row of the weights in shared memory: 16 bytes off 64
+    extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ float sc[2][HB_MMA][KT + 1], corr_sh[HB_MMA];
+    __shared__ __align__(16) __nv_bfloat16 wsh[HB_MMA][PST];
+    pdl_launch_dependents();
+    const int R8 = up8(p.kv_rank), rot8 = up8(p.rot_dim), CS = R8 + rot8, PS = R8 + 8;
+    const int S = CS / 8, SP = (S + 3) & ~3;                 // 16-byte slices of a row; padded to steps of 32 columns
+    const uint32_t rowb = row16 * 16;                        // odd in 16-byte units: ldmatrix is conflict-free
+    const uint32_t qs = smem_u32(smem), ks = qs + HB_MMA * rowb;          // [16] query rows, [2][KT] key rows
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h0 = blockIdx.y * HB_MMA, split = blockIdx.x;
+    const int pos = *p.d_pos;
+    const bool valid = pos >= 0 && pos < p.max_seq;
+    const int lo = valid && p.window > 0 && pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
+    const int nk = valid ? pos - lo + 1 : 0;
+    const int tiles = (nk + KT - 1) / KT, per = (tiles + p.n_split - 1) / p.n_split;
+    const int t0 = split * per, t1 = min(t0 + per, tiles);
+    const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(p.d_cache);
+
+    auto copy_row = [&](uint32_t dst, const __nv_bfloat16 *src, bool on) {         // columns past the row hold zeros
+        for (int c = lane; c < SP; c += 32) cp16(dst + c * 16, src + (c < S ? c * 8 : 0), on && c < S);
+    };
+    auto stage = [&](int tile) {                             // all rows but the new token's; rows past the last hold zeros
+        const int k0 = lo + tile * KT;
+#pragma unroll
+        for (int i = 0; i < KT / 8; ++i) {
+            const int r = warp + 8 * i, kp = k0 + r;
+            if (kp != pos) copy_row(ks + ((tile & 1) * KT + r) * rowb, cache + (size_t)(kp < pos ? kp : 0) * CS, kp < pos);
+        }
+    };
+    auto stage_newest = [&](int tile) {
+        if (tile == tiles - 1 && warp == 0) copy_row(ks + ((tile & 1) * KT + nk - 1 - tile * KT) * rowb, cache + (size_t)pos * CS, true);
+    };
+    if (t0 < t1) stage(t0);
+    pdl_wait();
+    if (t0 < t1) {
+        const __nv_bfloat16 *q = static_cast<const __nv_bfloat16 *>(p.d_qlat);
+#pragma unroll
+        for (int i = 0; i < HB_MMA / 8; ++i) {
+            const int r = warp + 8 * i, h = h0 + r;
+            copy_row(qs + r * rowb, q + (size_t)(h < p.heads ? h : 0) * CS, h < p.heads);
+        }
+        stage_newest(t0);
+    }
+    cp_commit();
+
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f}, acc[NTW][4];
+#pragma unroll
+    for (int i = 0; i < NTW; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) acc[i][k] = 0.0f;
+    for (int tile = t0; tile < t1; ++tile) {
+        if (tile + 1 < t1) {
+            stage(tile + 1);
+            stage_newest(tile + 1);
+        }
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();
+        const uint32_t kt = ks + (tile & 1) * KT * rowb;
+        {   // scores: 16 heads x 8 keys per warp, this half of the columns
+            const int steps = SP / 4, mid = (steps + 1) / 2, s0 = warp < 4 ? 0 : mid, s1 = warp < 4 ? mid : steps;
+            const uint32_t qa = qs + (lane & 15) * rowb + (lane >> 4) * 16;
+            const uint32_t ka = kt + ((warp & 3) * 8 + (lane & 7)) * rowb + (lane >> 3) * 16;
+            float d[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+#pragma unroll 3
+            for (int s = s0; s < s1; ++s) {                  // 32 columns
+                uint32_t a[4], a2[4], b[4];
+                ldsm4(qa + s * 64, a);
+                ldsm4(qa + s * 64 + 32, a2);
+                ldsm4(ka + s * 64, b);
+                mma_bf16(d[0], a, b[0], b[1]);
+                mma_bf16(d[1], a2, b[2], b[3]);
+            }
+            const int r = lane >> 2, c = (warp & 3) * 8 + (lane & 3) * 2;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) sc[warp >> 2][r + (k >> 1) * 8][c + (k & 1)] = d[0][k] + d[1][k];
+        }
+        __syncthreads();
+        const int n = nk - tile * KT;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {                        // a lane per key
+            const int r = 2 * warp + i;
+            const float s = lane < n ? sc[0][r][lane] + sc[1][r][lane] : -INFINITY;
+            const float mt = fmaxf(m[i], warp_max(s));
+            const float w = lane < n ? expf(s - mt) : 0.0f;
+            const float corr = m[i] == -INFINITY ? 0.0f : expf(m[i] - mt);
+            l[i] = fmaf(l[i], corr, warp_sum(w));
+            m[i] = mt;
+            wsh[r][lane] = __float2bfloat16_rn(w);
+            if (lane == 0) corr_sh[r] = corr;
+        }
+        __syncthreads();
+        const float c0 = corr_sh[lane >> 2], c1 = corr_sh[(lane >> 2) + 8];
+        uint32_t wa[KT / 16][4];
+#pragma unroll
+        for (int k = 0; k < KT / 16; ++k) ldsm4(smem_u32(&wsh[lane & 15][k * 16 + (lane >> 4) * 8]), wa[k]);
+#pragma unroll
+        for (int i = 0; i < NTW; i += 2) {
+            const int col = (warp * NTW + i) * 8;
+            if (col >= R8) break;                            // uniform across the warp
+#pragma unroll
+            for (int j = 0; j < 2; ++j) { acc[i + j][0] *= c0; acc[i + j][1] *= c0; acc[i + j][2] *= c1; acc[i + j][3] *= c1; }
+            const uint32_t va = kt + (lane & 15) * rowb + (col + (lane >> 4) * 8) * 2;
+#pragma unroll
+            for (int k = 0; k < KT / 16; ++k) {
+                uint32_t b[4];
+                ldsm4_t(va + k * 16 * rowb, b);
+                mma_bf16(acc[i], wa[k], b[0], b[1]);
+                mma_bf16(acc[i + 1], wa[k], b[2], b[3]);
+            }
+        }
+        __syncthreads();                                     // this tile's rows, scores and weights are overwritten next
+    }
+#pragma unroll
+    for (int i = 0; i < NTW; ++i) {
+        const int col = (warp * NTW + i) * 8 + (lane & 3) * 2;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int h = h0 + (lane >> 2) + 8 * r;
+            if (col < R8 && h < p.heads)
+                *reinterpret_cast<float2 *>(p.d_part + ((size_t)h * p.n_split + split) * PS + col) = make_float2(acc[i][2 * r], acc[i][2 * r + 1]);
+        }
+    }
+    if (lane < 2 && h0 + 2 * warp + lane < p.heads) {
+        float *part = p.d_part + ((size_t)(h0 + 2 * warp + lane) * p.n_split + split) * PS;
+        part[R8] = lane ? m[1] : m[0];
+        part[R8 + 1] = lane ? l[1] : l[0];
+    }
 }
 
 template <int WT>
@@ -495,25 +653,6 @@ __device__ __forceinline__ float ex2(float x)                // 2^x, 2 ulp, 0 fo
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
-__device__ __forceinline__ void ldsm4(uint32_t a, uint32_t (&r)[4])
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t a, uint32_t (&r)[4])
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
-{
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi)
-{
-    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t *>(&h);
-}
-
 template <int DV, int NW>
 __global__ void __launch_bounds__(NW * 32, 16 / NW) latent_attend_bf16_kernel(const __grid_constant__ b200_latent_args p, int dqs, int stages)
 {
@@ -741,19 +880,31 @@ int decode(const b200_latent_args &a, cudaStream_t st)
     int rc = launch_pdl(latent_absorb_kernel<WT>, a.heads * chunks + 1, 1, 0, a.use_pdl, st, a, chunks, lpr);
     if (rc) return rc;
 
-    int row16 = CS / E;                                      // 2 mod 4: four keys x two slices touch different banks
-    while (row16 % 4 != 2) ++row16;
-    const size_t smem = (size_t)KT * row16 * 16 + (size_t)HB * CS * 4;
-    const int hb = (a.heads + HB - 1) / HB, nch = (R8 + 64 * E - 1) / (64 * E);
-#define SCORES(N)                                                                             \
+#define SCORES(K, GROUPS)                                                                     \
     do {                                                                                      \
-        if ((rc = allow_smem(latent_scores_kernel<WT, N>, smem)) != 0) return rc;              \
-        rc = launch_pdl(latent_scores_kernel<WT, N>, a.n_split, hb, smem, a.use_pdl, st, a, row16); \
+        if ((rc = allow_smem(K, smem)) != 0) return rc;                                        \
+        rc = launch_pdl(K, a.n_split, GROUPS, smem, a.use_pdl, st, a, row16);                  \
     } while (0)
-    if (nch <= 1) SCORES(1);
-    else if (nch <= 2) SCORES(2);
-    else if (nch <= 4) SCORES(4);
-    else return B200_E_TOOLARGE;
+    if (WT == B200_WT_BF16) {
+        int row16 = (CS / 8 + 3) & ~3;                       // steps of 32 columns, then odd
+        row16 |= 1;
+        const size_t smem = (size_t)(HB_MMA + 2 * KT) * row16 * 16;
+        const int groups = (a.heads + HB_MMA - 1) / HB_MMA;
+        if (R8 <= 128) SCORES(latent_scores_bf16_kernel<2>, groups);
+        else if (R8 <= 256) SCORES(latent_scores_bf16_kernel<4>, groups);
+        else if (R8 <= 512) SCORES(latent_scores_bf16_kernel<8>, groups);
+        else if (R8 <= 1024) SCORES(latent_scores_bf16_kernel<16>, groups);
+        else return B200_E_TOOLARGE;
+    } else {
+        int row16 = CS / E;                                  // 2 mod 4: four keys x two slices touch different banks
+        while (row16 % 4 != 2) ++row16;
+        const size_t smem = (size_t)KT * row16 * 16 + (size_t)HB * CS * 4;
+        const int groups = (a.heads + HB - 1) / HB;
+        if (R8 <= 64 * E) SCORES(latent_scores_f32_kernel<1>, groups);
+        else if (R8 <= 128 * E) SCORES(latent_scores_f32_kernel<2>, groups);
+        else if (R8 <= 256 * E) SCORES(latent_scores_f32_kernel<4>, groups);
+        else return B200_E_TOOLARGE;
+    }
 #undef SCORES
     if (rc) return rc;
     const int vchunks = (a.vdim + VALUE_ROWS - 1) / VALUE_ROWS;
@@ -789,8 +940,8 @@ extern "C" int b200_latent_splits(int heads, int window, int max_seq)
 {
     if (heads <= 0 || max_seq <= 0) return 1;
     const int span = window > 0 && window < max_seq ? window : max_seq;
-    const int tiles = (span + KT - 1) / KT, groups = (heads + HB - 1) / HB;
-    int n = 2 * 148 / groups;
+    const int tiles = (span + KT - 1) / KT, groups = (heads + HB_MMA - 1) / HB_MMA;
+    int n = 148 / groups;
     if (n > tiles) n = tiles;
     if (n > MAX_SPLITS) n = MAX_SPLITS;
     return n < 1 ? 1 : n;

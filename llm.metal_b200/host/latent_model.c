@@ -52,7 +52,8 @@ typedef struct {
     PackedMat head;
     float **rope_tab; int n_rope;
     /* one token */
-    float *proj, *qlat, *part, *attn, *z, *u, *rg2, *act, *hist, *mix, *x;
+    void *qlat;
+    float *proj, *part, *attn, *z, *u, *rg2, *act, *hist, *mix, *x;
     /* rows (allocated at the first portion) */
     int chunk;
     float *r_proj, *r_hist, *r_x, *r_u, *r_y, *r_gu, *r_logits;
