@@ -456,8 +456,8 @@ def write_latent_model(folder, z, seed):
              "mlp": {"kind": "dense", "ff": z["ff"]}}
     D, V, F, H, R, nl = z["width"], z["vocab"], z["ff"], z["heads"], z["kv_rank"], z["layers"]
     with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump({"architecture": "Morilorn", "vocab": V, "width": D, "embedding": {"scale": 12.0}, "norm": {"eps": 1e-5, "groups": 2},
-                   "postln_alpha": 2.0, "logit_softcap": 15.0, "layers": [layer] * nl}, f)
+        json.dump({"architecture": "Morilorn", "vocab": V, "width": D, "embedding": {"scale": 8.0}, "norm": {"eps": 1e-6, "groups": 4},
+                   "postln_alpha": 2.0, "logit_softcap": 30.0, "layers": [layer] * nl}, f)
     shapes = {"embed": (V, D), "head": (V, D), "final.norm": (D,)}
     for i in range(nl):
         shapes.update({f"l{i}.{k}": v for k, v in {
