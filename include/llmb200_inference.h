@@ -166,9 +166,9 @@ int llmb200_state_graph_kernels(InferenceState *state, int with_lm_head);
 size_t llmb200_state_export_weight(InferenceState *state, int layer, int which, void *buf, size_t cap);
 
 /* A state for the model in a folder that holds config.json and model.safetensors; the model type is
- * config.json's "architecture" (Morilorn). wtype: B200_WT_BF16 (bfloat16 matrices and products with fp32
+ * config.json's "architecture" (Morilorn, Zidepel). wtype: B200_WT_BF16 (bfloat16 matrices and products with fp32
  * accumulation; norms, scores, softmax, gates and the residual stream in fp32) or B200_WT_F32 (everything in
- * fp32). max_seq_len positions of cache, not clamped. NULL with a message on stderr on any failure. No
+ * fp32). max_seq_len positions of cache (no more than the table of a model with learned positions holds). NULL with a message on stderr on any failure. No
  * counterpart in the reference, whose loaders fill the structures that inference_state_create takes. */
 InferenceState *inference_state_create_from_dir(const char *dir, int max_seq_len, int wtype);
 /* Feeds n tokens at the current position and advances it by n; logits of the places want[0..n_want), ascending

@@ -79,13 +79,17 @@ int b200_q8_unpack_blocks(const void *d_packed, long long row_stride, int rows, 
  *                  (if slot_norm_gamma: S <- rmsnorm(S) * slot_norm_gamma first);
  *                  block 0 stores h to resid_out; x = h
  *   B200_IN_EMBED  h = emb[tokens[*pos]][0..cols) * emb_scale; stored to
- *                  resid_out by block 0; x = h
+ *                  resid_out by block 0; x = h. BF16 / F32 weights: emb_pos[*pos][0..cols) is added when given
+ *                  (rows past emb_pos_rows read the last one), then slot_norm_gamma / slot_norm_beta
+ *                  make h its layer norm, and x = *mix_coef * h when mix_coef is given
  *   B200_IN_POSTNORM (BF16 / F32 weights) h = norm(in_vec) * slot_norm_gamma; block 0 stores h to
  *                  post_copy (if not NULL); x = mix_in ? mix_in + *mix_coef * h : h, stored to
  *                  resid_out by block 0 (if not NULL)
  * then, if norm_gamma != NULL, x <- x * rsqrt(mean(x^2)+eps) * norm_gamma. With norm_groups > 1 the
  * norms of BF16 / F32 launches treat that many equal consecutive parts of the vector separately;
- * norm_dim (0 = cols) is the length they run over when the columns past it are padding.
+ * norm_dim (0 = cols) is the length they run over when the columns past it are padding. A norm that is
+ * given a bias (norm_beta, slot_norm_beta; BF16 / F32) is a layer norm: (x - mean) / sqrt(variance + eps)
+ * * gamma + beta.
  *
  * Output (out_mode):
  *   B200_OUT_STORE  out[p][out_offset + r] = y[r] for every peer p < n_out
@@ -94,6 +98,14 @@ int b200_q8_unpack_blocks(const void *d_packed, long long row_stride, int rows, 
  *                   it are pairs, row r above goes to out2[r - glu_rows] as it is
  *   B200_OUT_GATED  (BF16 / F32 weights) out[0][r] = resid_alpha * out_resid[r]
  *                   + sigmoid(out_gate[r] + out_gate_bias[r]) * y[r]
+ *   B200_OUT_STREAMS (BF16 / F32 weights) the result joins n_streams residual streams X_s: X'_t[r] =
+ *                   sum over s of mix[s][t] * X_s[r] + spread[t] * y[r], stored at streams_out +
+ *                   t * streams_out_stride, and out[0][r] = sum over t of take[t] * X'_t[r], what the next
+ *                   reader sees. connect = mix (from, to) | spread | take, n_streams * (n_streams + 2) floats.
+ *                   streams_in_stride 0: all old streams are one vector
+ * B200_OUT_STORE with act = B200_ACT_RELU2 (BF16 / F32) stores max(y, 0)^2.
+ * Layer norms, learned positions, streams and the squared relu form one family of kernels, post-norm inputs,
+ * GLU, gated outputs, depth sums, RMS norms and the cap another: a BF16 / F32 launch uses one of the two.
  * BF16 / F32 launches can also cap what they store, y <- softcap * tanh(y / softcap), and form a depth
  * sum for the rows they own, hist_out[r] = sum over j < hist_n of hist_coef[j] * hist[j * hist_stride + r].
  * With d_argmax_scratch != NULL (B200_OUT_STORE only) the launch also leaves
@@ -107,7 +119,9 @@ int b200_q8_unpack_blocks(const void *d_packed, long long row_stride, int rows, 
  * that runs out sets *err = 1 and the kernel carries on without hanging.
  * ---------------------------------------------------------------------- */
 enum { B200_IN_VEC = 0, B200_IN_RESID = 1, B200_IN_EMBED = 2, B200_IN_POSTNORM = 3 };
-enum { B200_OUT_STORE = 0, B200_OUT_GLU = 1, B200_OUT_GATED = 2 };
+enum { B200_OUT_STORE = 0, B200_OUT_GLU = 1, B200_OUT_GATED = 2, B200_OUT_STREAMS = 3 };
+enum { B200_ACT_SILU = 0, B200_ACT_GELU_TANH = 1, B200_ACT_RELU2 = 2 };
+#define B200_MAX_STREAMS 8
 
 typedef struct b200_matvec_args {
     /* weights */
@@ -156,6 +170,11 @@ typedef struct b200_matvec_args {
     const float *d_hist; int hist_n; long long hist_stride; const float *d_hist_coef; float *d_hist_out;
     int glu_rows; float *d_out2;
     float softcap;                 /* 0 = none */
+    const float *d_norm_beta, *d_slot_norm_beta;
+    const float *d_emb_pos; int emb_pos_rows;
+    const float *d_streams_in; long long streams_in_stride;
+    float *d_streams_out; long long streams_out_stride;
+    const float *d_connect; int n_streams;
 } b200_matvec_args;
 
 int b200_matvec(const b200_matvec_args *a, void *stream);
@@ -263,6 +282,83 @@ int b200_latent_rows_prep(const b200_latent_args *a, void *stream);
 int b200_latent_rows_attend(const b200_latent_args *a, void *stream);
 
 /* ------------------------------------------------------------------------
+ * Grouped-query attention with normed queries and keys, no rotation. Per position:
+ *   q = rms_norm(q head) * q_gamma * q_scale[position], k = rms_norm(k head) * k_gamma   (gammas shared by heads)
+ *   score = scale * (q . k), then softcap * tanh(score / softcap) when softcap > 0
+ * softmax over every earlier position and its own; query head h reads key / value head h / (heads / kv_heads).
+ * The caches hold [kv_heads][max_seq] rows of up8(dim) / up8(vdim) elements of the type `wtype` names (BF16 or
+ * F32), padding zero.
+ * Decode (b200_gqa_decode, one launch): the token at *d_pos; writes its cache rows. A position outside
+ * [0, max_seq) is ignored. d_tickets: kv_heads * heads zero-initialised words, zero again afterwards.
+ * Rows: n_rows tokens from position pos0 on. _prep writes their cache rows and d_q_rows, _attend runs the
+ * attention (BF16: tensor cores, F32: CUDA cores).
+ * ---------------------------------------------------------------------- */
+typedef struct b200_gqa_args {
+    int wtype;
+    int heads, kv_heads, dim, vdim, max_seq;
+    float scale, softcap, eps;
+    const float *d_q, *d_k, *d_v;        /* one token, or n_rows rows proj_ld floats apart */
+    const float *d_q_gamma, *d_k_gamma;  /* [dim] */
+    const float *d_q_scale;              /* [max_seq] or NULL */
+    void *d_k_cache, *d_v_cache;
+    /* decode */
+    float *d_part;                       /* [heads][n_split][up8(vdim) + 8] */
+    unsigned *d_tickets;
+    float *d_out;                        /* [heads * vdim] */
+    const int *d_pos;
+    int n_split, use_pdl;
+    /* rows */
+    int n_rows, pos0;
+    long long proj_ld;
+    void *d_q_rows;                      /* [n_rows][heads][up8(dim)] */
+    void *d_out_rows; long long out_ld;  /* [n_rows] rows of heads * vdim, out_ld elements apart */
+} b200_gqa_args;
+
+/* Splits of the sequence worth launching for this shape (1 .. 256). */
+int b200_gqa_splits(int wtype, int heads, int kv_heads, int dim, int vdim, int max_seq);
+int b200_gqa_decode(const b200_gqa_args *a, void *stream);
+int b200_gqa_rows_prep(const b200_gqa_args *a, void *stream);
+int b200_gqa_rows_attend(const b200_gqa_args *a, void *stream);
+
+/* ------------------------------------------------------------------------
+ * Gated linear attention: per head a state S [dim][vdim] in fp32 that decays by a factor per key channel,
+ *   a = logistic(W_a2 f + a2_bias)^(1/tau),  S <- diag(a) S + k v^T,  o = S^T (q * q_scale)
+ * then o is RMS-normed over vdim (norm_gamma, shared by heads) and multiplied by silu(gate).
+ * f (rank numbers) is the low-rank input of the decay; d_a2 is [heads * dim][up4(rank)] fp32, padding zero.
+ * Everything from the projections on is fp32.
+ *
+ * States are kept per position: the state before position p is in slot p mod n_slots of d_state
+ * [n_slots][heads][dim][up8(vdim)] (padding zero) and the one after it goes to the next slot, so running a position again gives the
+ * same result, as with a key cache. Before position 0 the state is zero, whatever the slot holds.
+ * Decode (b200_gla_decode, one launch): the token at *d_pos. Rows (b200_gla_rows): n_rows tokens from position
+ * pos0 on, cut into chunks of 64 that are summed in parallel and joined by a scan over their states.
+ * ---------------------------------------------------------------------- */
+#define B200_GLA_CHUNK 64
+typedef struct b200_gla_args {
+    int wtype;                           /* element type of d_out_rows */
+    int heads, dim, vdim, rank, n_slots;
+    float tau, q_scale, eps;
+    const float *d_q, *d_k, *d_v, *d_gate, *d_f;   /* one token, or n_rows rows proj_ld floats apart */
+    const float *d_a2, *d_a2_bias, *d_norm_gamma;
+    float *d_state;
+    /* decode */
+    float *d_out;                        /* [heads * vdim] */
+    const int *d_pos;
+    int use_pdl;
+    /* rows; n_chunks = (n_rows + 63) / 64 */
+    int n_rows, pos0;
+    long long proj_ld;
+    float *d_qd, *d_kd;                  /* [n_chunks * 64][heads][up8(dim)]: queries and keys times their decays */
+    float *d_decay;                      /* [n_chunks][heads][up8(dim)]: decay over a whole chunk */
+    float *d_scores;                     /* [n_chunks][heads][64][64] */
+    float *d_chunk_state;                /* [n_chunks][heads][dim][up8(vdim)] */
+    float *d_o;                          /* [n_rows][heads * vdim]; vdim > 128 only */
+    void *d_out_rows; long long out_ld;  /* [n_rows] rows of heads * vdim, out_ld elements apart */
+} b200_gla_args;
+int b200_gla_decode(const b200_gla_args *a, void *stream);
+int b200_gla_rows(const b200_gla_args *a, void *stream);
+
+/* ------------------------------------------------------------------------
  * Row-wise steps of a prompt portion. Rows are ld floats apart; columns dim .. ld-1 are padding and are
  * written as zeros. out_h (BF16 copies for the tensor-core products) may be NULL.
  * ---------------------------------------------------------------------- */
@@ -283,6 +379,33 @@ typedef struct b200_rows_postnorm_args {
     float *out; void *out_h;
 } b200_rows_postnorm_args;
 int b200_rows_postnorm(const b200_rows_postnorm_args *a, void *stream);
+/* Residual streams, one sublayer's result y joined in: X'_t[m] = sum over s of mix[s][t] * X_s[m] + spread[t] * y[m]
+ * (connect as in B200_OUT_STREAMS), X_s at streams_in + s * streams_in_stride, X'_t at streams_out + t *
+ * streams_out_stride (NULL: not kept), u[m] = sum over t of take[t] * X'_t[m] (stored to u_out when given), and the
+ * layer norm of u (gamma, beta) to out, element type wtype (out NULL: no norm). */
+typedef struct b200_rows_streams_args {
+    const float *streams_in; long long streams_in_stride;
+    const float *y; long long y_ld;
+    const float *connect; int n_streams;
+    const float *gamma, *beta; float eps;
+    int rows, dim, ld, wtype;
+    float *streams_out; long long streams_out_stride;
+    float *u_out;
+    void *out;
+} b200_rows_streams_args;
+int b200_rows_streams(const b200_rows_streams_args *a, void *stream);
+/* The rows that all streams start from, x[m] = layer_norm(emb[tokens[m]] + emb_pos[pos0 + m]) * emb_gamma + emb_beta,
+ * and what the first reader makes of them, out[m] = layer_norm(*take * x[m]) * gamma + beta. */
+typedef struct b200_rows_start_args {
+    const float *emb, *emb_pos; const uint32_t *tokens; int vocab, pos_rows, pos0;
+    const float *emb_gamma, *emb_beta, *take, *gamma, *beta; float eps;
+    int rows, dim, ld, wtype;
+    float *x; void *out;
+} b200_rows_start_args;
+int b200_rows_start(const b200_rows_start_args *a, void *stream);
+/* out[m] = layer norm of x[index[m]] (index NULL: m) times gamma plus beta. */
+int b200_rows_layer_norm(const float *x, const int *index, int rows, int dim, int ld, float eps,
+                         const float *gamma, const float *beta, int wtype, void *out, void *stream);
 /* out[m] = grouped RMS norm of x[index[m]] times gamma; wtype: element type of out (BF16 or F32). */
 int b200_rows_norm(const float *x, const int *index, int rows, int dim, int ld, int groups, float eps,
                    const float *gamma, int wtype, void *out, void *stream);

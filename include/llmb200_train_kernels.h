@@ -40,6 +40,7 @@ typedef struct {
                             bounded wait runs out (the product is then incomplete) */
     void *Ch; long long ldch;   /* b200_gemm_bf16 only: when not NULL the result is stored here as bfloat16 and C is
                                    not written (R must be NULL) */
+    int relu2;           /* store max(x, 0)^2 of the result x: b200_gemm_f32, and b200_gemm_bf16 with Ch and alpha 1 */
 } b200_gemm_args;
 
 /* CUDA-core version: any shape, any of the stride combinations above. */

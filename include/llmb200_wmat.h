@@ -55,7 +55,7 @@ void metal_enqueue_grpo_policy_grad(MetalBuf *logits, MetalBuf *actions, MetalBu
                                     MetalBuf *dlogits, int N, int V, float clip_eps);
 
 /* ---- containers (layouts as in src/nn/wmat.h:10-56) ---- */
-typedef enum { MODEL_QWEN3, MODEL_GEMMA3, MODEL_MORILORN /* addition */ } ModelType;
+typedef enum { MODEL_QWEN3, MODEL_GEMMA3, MODEL_MORILORN, MODEL_ZIDEPEL /* additions */ } ModelType;
 
 typedef struct WMat {
     MetalBuf *mbuf;

@@ -22,8 +22,10 @@ c_u32_p = C.POINTER(C.c_uint32)
 B200_MAX_PEERS = 8
 B200_WT_Q8, B200_WT_F16, B200_WT_BF16, B200_WT_F32 = 0, 1, 2, 3
 B200_IN_VEC, B200_IN_RESID, B200_IN_EMBED, B200_IN_POSTNORM = 0, 1, 2, 3
-B200_OUT_STORE, B200_OUT_GLU, B200_OUT_GATED = 0, 1, 2
-MODEL_QWEN3, MODEL_GEMMA3, MODEL_MORILORN = 0, 1, 2
+B200_OUT_STORE, B200_OUT_GLU, B200_OUT_GATED, B200_OUT_STREAMS = 0, 1, 2, 3
+B200_ACT_SILU, B200_ACT_GELU_TANH, B200_ACT_RELU2 = 0, 1, 2
+B200_MAX_STREAMS = 8
+MODEL_QWEN3, MODEL_GEMMA3, MODEL_MORILORN, MODEL_ZIDEPEL = 0, 1, 2, 3
 LLMB200_HANDLE_BYTES = 64
 
 
@@ -61,6 +63,9 @@ class MatvecArgs(C.Structure):
         ("d_hist", C.c_void_p), ("hist_n", C.c_int), ("hist_stride", C.c_longlong), ("d_hist_coef", C.c_void_p),
         ("d_hist_out", C.c_void_p),
         ("glu_rows", C.c_int), ("d_out2", C.c_void_p), ("softcap", C.c_float),
+        ("d_norm_beta", C.c_void_p), ("d_slot_norm_beta", C.c_void_p), ("d_emb_pos", C.c_void_p), ("emb_pos_rows", C.c_int),
+        ("d_streams_in", C.c_void_p), ("streams_in_stride", C.c_longlong), ("d_streams_out", C.c_void_p), ("streams_out_stride", C.c_longlong),
+        ("d_connect", C.c_void_p), ("n_streams", C.c_int),
     ]
 
 
@@ -144,7 +149,7 @@ class GemmArgs(C.Structure):
                 ("C", C.c_void_p), ("ldc", C.c_longlong),
                 ("R", C.c_void_p), ("ldr", C.c_longlong),
                 ("M", C.c_int), ("N", C.c_int), ("K", C.c_int), ("alpha", C.c_float), ("d_err", C.c_void_p),
-                ("Ch", C.c_void_p), ("ldch", C.c_longlong)]
+                ("Ch", C.c_void_p), ("ldch", C.c_longlong), ("relu2", C.c_int)]
 
 
 class LatentArgs(C.Structure):
@@ -157,6 +162,40 @@ class LatentArgs(C.Structure):
                [(n, C.c_int) for n in ("n_split", "use_pdl", "n_rows", "pos0", "kv_row0")] + \
                [("proj_ld", C.c_longlong), ("d_q_rows", C.c_void_p), ("d_kv", C.c_void_p), ("kv_ld", C.c_longlong),
                 ("d_out_rows", C.c_void_p), ("out_ld", C.c_longlong)]
+
+
+class GqaArgs(C.Structure):
+    """b200_gqa_args (include/llmb200_kernels.h)."""
+    _fields_ = [(n, C.c_int) for n in ("wtype", "heads", "kv_heads", "dim", "vdim", "max_seq")] + \
+               [(n, C.c_float) for n in ("scale", "softcap", "eps")] + \
+               [(n, C.c_void_p) for n in ("d_q", "d_k", "d_v", "d_q_gamma", "d_k_gamma", "d_q_scale", "d_k_cache", "d_v_cache",
+                                          "d_part", "d_tickets", "d_out", "d_pos")] + \
+               [(n, C.c_int) for n in ("n_split", "use_pdl", "n_rows", "pos0")] + \
+               [("proj_ld", C.c_longlong), ("d_q_rows", C.c_void_p), ("d_out_rows", C.c_void_p), ("out_ld", C.c_longlong)]
+
+
+class GlaArgs(C.Structure):
+    """b200_gla_args (include/llmb200_kernels.h)."""
+    _fields_ = [(n, C.c_int) for n in ("wtype", "heads", "dim", "vdim", "rank", "n_slots")] + \
+               [(n, C.c_float) for n in ("tau", "q_scale", "eps")] + \
+               [(n, C.c_void_p) for n in ("d_q", "d_k", "d_v", "d_gate", "d_f", "d_a2", "d_a2_bias", "d_norm_gamma", "d_state", "d_out", "d_pos")] + \
+               [(n, C.c_int) for n in ("use_pdl", "n_rows", "pos0")] + [("proj_ld", C.c_longlong)] + \
+               [(n, C.c_void_p) for n in ("d_qd", "d_kd", "d_decay", "d_scores", "d_chunk_state", "d_o", "d_out_rows")] + [("out_ld", C.c_longlong)]
+
+
+class RowsStreamsArgs(C.Structure):
+    """b200_rows_streams_args (include/llmb200_kernels.h)."""
+    _fields_ = [("streams_in", C.c_void_p), ("streams_in_stride", C.c_longlong), ("y", C.c_void_p), ("y_ld", C.c_longlong),
+                ("connect", C.c_void_p), ("n_streams", C.c_int), ("gamma", C.c_void_p), ("beta", C.c_void_p), ("eps", C.c_float),
+                ("rows", C.c_int), ("dim", C.c_int), ("ld", C.c_int), ("wtype", C.c_int),
+                ("streams_out", C.c_void_p), ("streams_out_stride", C.c_longlong), ("u_out", C.c_void_p), ("out", C.c_void_p)]
+
+
+class RowsStartArgs(C.Structure):
+    """b200_rows_start_args (include/llmb200_kernels.h)."""
+    _fields_ = [("emb", C.c_void_p), ("emb_pos", C.c_void_p), ("tokens", C.c_void_p), ("vocab", C.c_int), ("pos_rows", C.c_int), ("pos0", C.c_int)] + \
+               [(n, C.c_void_p) for n in ("emb_gamma", "emb_beta", "take", "gamma", "beta")] + [("eps", C.c_float)] + \
+               [(n, C.c_int) for n in ("rows", "dim", "ld", "wtype")] + [("x", C.c_void_p), ("out", C.c_void_p)]
 
 
 class RowsPostnormArgs(C.Structure):
@@ -197,7 +236,9 @@ SYMBOLS_MAIN = {
                           "b200_attn_scratch_floats", "b200_attn_decode", "b200_attn_decode_static", "b200_tp_argmax_finalize", "b200_token_plan", "b200_token_chunks", "b200_decode_token", "b200_lora_decode", "b200_argmax_rows",
                           "b200_launch_count", "b200_launch_count_add",
                           "b200_latent_splits", "b200_latent_decode", "b200_latent_rows_prep", "b200_latent_rows_attend", "b200_rows_embed",
-                          "b200_rows_postnorm", "b200_rows_norm", "b200_rows_gelu_mul", "b200_rows_softcap"],
+                          "b200_rows_postnorm", "b200_rows_norm", "b200_rows_gelu_mul", "b200_rows_softcap",
+                          "b200_gqa_splits", "b200_gqa_decode", "b200_gqa_rows_prep", "b200_gqa_rows_attend", "b200_gla_decode", "b200_gla_rows",
+                          "b200_rows_streams", "b200_rows_start", "b200_rows_layer_norm"],
     "llmb200_inference.h": ["inference_state_create", "inference_state_create_gemma3", "inference_state_free",
                             "inference_generate", "inference_state_model_type", "inference_state_vocab_size",
                             "inference_state_reset", "inference_forward_token", "inference_state_load_eos",
@@ -316,6 +357,11 @@ def lib():
         "b200_rows_embed": (i, [vp, vp, i, i, i, fl, vp, vp, vp]), "b200_rows_postnorm": (i, [C.POINTER(RowsPostnormArgs), vp]),
         "b200_rows_norm": (i, [vp, vp, i, i, i, i, fl, vp, i, vp, vp]), "b200_rows_gelu_mul": (i, [vp, ll, i, i, i, vp, vp]),
         "b200_rows_softcap": (i, [vp, i, i, ll, fl, vp]),
+        "b200_gqa_splits": (i, [i, i, i, i, i, i]), "b200_gqa_decode": (i, [C.POINTER(GqaArgs), vp]),
+        "b200_gqa_rows_prep": (i, [C.POINTER(GqaArgs), vp]), "b200_gqa_rows_attend": (i, [C.POINTER(GqaArgs), vp]),
+        "b200_gla_decode": (i, [C.POINTER(GlaArgs), vp]), "b200_gla_rows": (i, [C.POINTER(GlaArgs), vp]),
+        "b200_rows_streams": (i, [C.POINTER(RowsStreamsArgs), vp]), "b200_rows_start": (i, [C.POINTER(RowsStartArgs), vp]),
+        "b200_rows_layer_norm": (i, [vp, vp, i, i, i, fl, vp, vp, i, vp, vp]),
         # ---- llmb200_train_kernels.h
         "b200_gemm_f32": (i, [C.POINTER(GemmArgs), vp]), "b200_gemm_tf32": (i, [C.POINTER(GemmArgs), vp]),
         "b200_gemm_f16": (i, [C.POINTER(GemmArgs), vp]), "b200_gemm_bf16": (i, [C.POINTER(GemmArgs), vp]), "b200_f32_to_f16": (i, [vp, sz, fl, vp, vp]),

@@ -23,9 +23,9 @@ OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libllmb200.so")
 LIB_SYNTH = os.path.join(HERE, "libllmb200_synth.so")
 
-CU_SOURCES = ["pack.cu", "matvec.cu", "matvec_ext.cu", "attention.cu", "decode_token.cu", "lora_decode.cu", "batch_kernels.cu", "gemm_f32.cu", "gemm_tf32.cu", "train_kernels.cu",
-              "latent_attention.cu", "row_kernels.cu"]
-C_SOURCES = ["weights.c", "decode_engine.c", "sft_engine.c", "batch_engine.c", "json.c", "tensor_file.c", "model_dir.c", "latent_model.c"]
+CU_SOURCES = ["pack.cu", "matvec.cu", "matvec_ext.cu", "matvec_streams.cu", "attention.cu", "decode_token.cu", "lora_decode.cu", "batch_kernels.cu", "gemm_f32.cu", "gemm_tf32.cu", "train_kernels.cu",
+              "latent_attention.cu", "gqa_attention.cu", "gla.cu", "row_kernels.cu"]
+C_SOURCES = ["weights.c", "decode_engine.c", "sft_engine.c", "batch_engine.c", "json.c", "tensor_file.c", "model_dir.c", "model_dir_common.c", "latent_model.c", "hybrid_model.c"]
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC"]

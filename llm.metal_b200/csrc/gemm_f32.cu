@@ -74,6 +74,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const b200_gemm_args p)
             if (gn >= p.N) continue;
             float v = p.alpha * acc[i][j];
             if (p.R) v += p.R[(long long)gm * p.ldr + gn];
+            if (p.relu2) { v = fmaxf(v, 0.0f); v *= v; }
             p.C[(long long)gm * p.ldc + gn] = v;
         }
     }

@@ -53,6 +53,7 @@ struct EpiArgs {
     int splits;        // CTAs sharing one output tile along k (gridDim.z); 1 = none
     unsigned *flags;   // one turn counter per output tile, zero between launches
     __nv_bfloat16 *Ch; long long ldch;   // bfloat16 result instead of C (never with splits > 1)
+    int relu2;         // store max(x, 0)^2 (bfloat16 results)
 };
 
 // Turn counters of the serial split-k epilogue (see the kernel): one word per output tile.
@@ -253,6 +254,10 @@ gemm_tf32_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 uint32_t r[32];
                 tmem_ld32(tmem_base + ((uint32_t)lane_base << 16) + (uint32_t)c, r);
                 if (row < p.M && p.Ch) {
+                    if (p.relu2) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(act_relu2(__uint_as_float(r[j])));
+                    }
                     __nv_bfloat16 *hrow = p.Ch + (long long)row * p.ldch + n0 + c;      // 16-byte aligned: checked by the host
                     if (cw == 32 && n0 + c + 32 <= p.N) {
 #pragma unroll
@@ -453,6 +458,7 @@ int launch(const CUtensorMap &ma, const CUtensorMap &mb, EpiArgs e, cudaStream_t
 static int gemm_tc(const b200_gemm_args *a, int f16, void *stream)
 {
     if (!a || !a->A || !a->B || (!a->C && !a->Ch) || a->M <= 0 || a->N <= 0 || a->K <= 0) return B200_E_BADARG;
+    if (a->relu2 && (!a->Ch || a->alpha != 1.0f)) return B200_E_BADARG;
     if (a->Ch && (f16 != 2 || a->R || (a->ldch & 7) || (reinterpret_cast<uintptr_t>(a->Ch) & 15))) return B200_E_BADARG;
     if (a->a_col != 1 || a->b_row != 1) return B200_E_UNSUPPORTED;
     const long long lda = a->a_row, ldb = a->b_col;
@@ -464,7 +470,7 @@ static int gemm_tc(const b200_gemm_args *a, int f16, void *stream)
 
     CUtensorMap ma, mb;
     EpiArgs e = {a->C, a->ldc, a->R, a->ldr, a->M, a->N, a->K, a->alpha, a->d_err, 128, 0, 0, f16, 1, 1, nullptr,
-                 static_cast<__nv_bfloat16 *>(a->Ch), a->ldch};
+                 static_cast<__nv_bfloat16 *>(a->Ch), a->ldch, a->relu2};
     // LLMB200_GEMM_BN=<n> overrides the tile width for experiments
     static int forced = -1;
     if (forced < 0) {

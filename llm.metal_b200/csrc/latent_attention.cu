@@ -10,15 +10,8 @@
 //   latent_value   merges the splits of a head, applies W_uv and the output gate
 //
 // Prompt portions: latent_prep writes cache rows and rotated queries of all rows; keys and values are expanded
-// by a product the caller runs; latent_attend_bf16 is a tiled online-softmax attention on the tensor cores
-// (mma.sync m16n8k16, bfloat16 operands, fp32 scores, weights and sums), latent_attend_f32 the same sum in
-// fp32 on the CUDA cores.
-#include "stream_core.cuh"
-#include "../../include/llmb200_kernels.h"
-
-#include <cuda_bf16.h>
-
-extern unsigned long long g_b200_launches;
+// by a product the caller runs; the attention over them is the tiled one of row_attention.cuh.
+#include "row_attention.cuh"
 
 namespace {
 
@@ -29,30 +22,6 @@ constexpr int ABSORB_PASSES = 4;   // row passes whose weights a warp of latent_
 constexpr int VALUE_ROWS = 16;     // value rows per block of latent_value, two per warp
 constexpr int MAX_SPLITS = 256;
 
-__host__ __device__ __forceinline__ int up8(int n) { return (n + 7) & ~7; }
-
-template <int WT> struct Elem;
-template <> struct Elem<B200_WT_BF16> {
-    using T = __nv_bfloat16;
-    static constexpr int E = 8;
-    static __device__ __forceinline__ float dot(const uint4 &w, const float *x) { return dot8_bf16(w, x); }
-    static __device__ __forceinline__ void unpack(const uint4 &w, float *x)
-    {
-        const uint32_t u[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-        for (int i = 0; i < 4; ++i) { const float2 f = bf16_pair(u[i]); x[2 * i] = f.x; x[2 * i + 1] = f.y; }
-    }
-};
-template <> struct Elem<B200_WT_F32> {
-    using T = float;
-    static constexpr int E = 4;
-    static __device__ __forceinline__ float dot(const uint4 &w, const float *x) { return dot4_f32(w, x); }
-    static __device__ __forceinline__ void unpack(const uint4 &w, float *x)
-    {
-        x[0] = __uint_as_float(w.x); x[1] = __uint_as_float(w.y); x[2] = __uint_as_float(w.z); x[3] = __uint_as_float(w.w);
-    }
-};
-
 // Element i of a rotated vector v whose first `dims` elements turn pairwise by the angles in rope (cos, sin).
 __device__ __forceinline__ float rotated(const float *v, int i, int dims, const float *rope)
 {
@@ -61,14 +30,6 @@ __device__ __forceinline__ float rotated(const float *v, int i, int dims, const 
     const float a = v[i & ~1], b = v[(i & ~1) + 1];
     return (i & 1) ? b * c + a * s : a * c - b * s;
 }
-
-__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool on)
-{
-    const int n = on ? 16 : 0;                               // 0: the 16 bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // The cache row of one token, by all 256 threads of a block. `wait` runs before anything an earlier kernel of the
 // same token wrote is read; norm weights and angles are fetched ahead of it. `red` holds >= 33 floats.
@@ -279,25 +240,6 @@ __global__ void __launch_bounds__(256) latent_scores_f32_kernel(const __grid_con
                 *reinterpret_cast<float4 *>(part + col + e) = make_float4(acc[c][e], acc[c][e + 1], acc[c][e + 2], acc[c][e + 3]);
     }
     if (half == 0 && lane == 0) { part[R8] = m; part[R8 + 1] = l; }
-}
-
-__device__ __forceinline__ void ldsm4(uint32_t a, uint32_t (&r)[4])
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t a, uint32_t (&r)[4])
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
-{
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi)
-{
-    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t *>(&h);
 }
 
 // bfloat16, on the tensor cores: sixteen heads are the rows of both products, so a cache row is read from shared
@@ -587,253 +529,6 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const __grid_constant_
     }
 }
 
-// fp32: one warp per (row, head), a lane per key, value columns over the lanes (256 per blockIdx.z).
-__global__ void __launch_bounds__(128) latent_attend_f32_kernel(const __grid_constant__ b200_latent_args p)
-{
-    extern __shared__ __align__(16) float qsh[];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int h = blockIdx.y * 4 + warp, m = blockIdx.x, c0 = blockIdx.z * 256;
-    if (h >= p.heads) return;                                // warps are independent of one another
-    const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), QS = dim8 + rot8, vd8 = up8(p.vdim), R8 = up8(p.kv_rank), CS = R8 + rot8;
-    float *q = qsh + (size_t)warp * QS;
-    const float *qg = static_cast<const float *>(p.d_q_rows) + ((size_t)m * p.heads + h) * QS;
-    for (int i = lane; i < QS; i += 32) q[i] = qg[i];
-    __syncwarp();
-    const int pos = p.pos0 + m;
-    const int lo = p.window > 0 && pos - p.window + 1 > 0 ? pos - p.window + 1 : 0;
-    const float *kv = static_cast<const float *>(p.d_kv) + (size_t)h * (dim8 + vd8);
-    const float *cache = static_cast<const float *>(p.d_cache);
-    float mx = -INFINITY, l = 0.0f, acc[8];
-#pragma unroll
-    for (int c = 0; c < 8; ++c) acc[c] = 0.0f;
-    for (int k0 = lo; k0 <= pos; k0 += 32) {
-        const int n = min(32, pos - k0 + 1), kp = k0 + lane;
-        float s = -INFINITY;
-        if (lane < n) {
-            const float *kn = kv + (size_t)(kp - p.kv_row0) * p.kv_ld, *kr = cache + (size_t)kp * CS + R8;
-            float a = 0.0f, b = 0.0f;
-            for (int d = 0; d < p.dim; ++d) a = fmaf(q[d], kn[d], a);
-            for (int d = 0; d < p.rot_dim; ++d) b = fmaf(q[dim8 + d], kr[d], b);
-            s = p.scale * (a + b);
-        }
-        const float mt = fmaxf(mx, warp_max(s));
-        const float w = lane < n ? expf(s - mt) : 0.0f;
-        const float corr = mx == -INFINITY ? 0.0f : expf(mx - mt);
-        l = l * corr + warp_sum(w);
-        mx = mt;
-#pragma unroll
-        for (int c = 0; c < 8; ++c) acc[c] *= corr;
-        for (int j = 0; j < n; ++j) {
-            const float wj = __shfl_sync(0xffffffffu, w, j);
-            const float *v = kv + (size_t)(k0 + j - p.kv_row0) * p.kv_ld + dim8;
-#pragma unroll
-            for (int c = 0; c < 8; ++c) {
-                const int col = c0 + c * 32 + lane;
-                if (col < p.vdim) acc[c] = fmaf(wj, v[col], acc[c]);
-            }
-        }
-    }
-    const float inv = 1.0f / l;
-    float *o = static_cast<float *>(p.d_out_rows) + (size_t)m * p.out_ld + (size_t)h * p.vdim;
-    const float *gate = p.d_gate + (size_t)m * p.proj_ld + (size_t)h * p.vdim;
-#pragma unroll
-    for (int c = 0; c < 8; ++c) {
-        const int col = c0 + c * 32 + lane;
-        if (col < p.vdim) o[col] = acc[c] * inv * sigmoid_f32(gate[col]);
-    }
-}
-
-// bfloat16 on the tensor cores. A block: NW warps of 16 query rows of one head; keys 32 at a time, the next tile's
-// copies in flight under the current one. DV value columns per blockIdx.z.
-constexpr int BKEY = 32;
-
-__device__ __forceinline__ float ex2(float x)                // 2^x, 2 ulp, 0 for -inf
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-template <int DV, int NW>
-__global__ void __launch_bounds__(NW * 32, 16 / NW) latent_attend_bf16_kernel(const __grid_constant__ b200_latent_args p, int dqs, int stages)
-{
-    // dqs: elements of a query / key row in shared memory; its first dqs - 8 are multiples of 16 and hold
-    // [unrotated | rotated | zeros]. Rows are 16 bytes off a multiple of 32: ldmatrix is conflict-free.
-    constexpr int VS = DV + 8, BQ = NW * 16, NT = NW * 32;
-    extern __shared__ __align__(16) unsigned char smem[];
-    const int dim8 = up8(p.dim), rot8 = up8(p.rot_dim), QS = dim8 + rot8, vd8 = up8(p.vdim), R8 = up8(p.kv_rank), CS = R8 + rot8;
-    const int dqk = dqs - 8;
-    __nv_bfloat16 *qsm = reinterpret_cast<__nv_bfloat16 *>(smem);
-    __nv_bfloat16 *ksm = qsm + (size_t)BQ * dqs;             // [stages][BKEY][dqs]
-    __nv_bfloat16 *vsm = ksm + (size_t)stages * BKEY * dqs;  // [stages][BKEY][VS]
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int h = blockIdx.y, m0 = blockIdx.x * BQ, c0 = blockIdx.z * DV;
-    const int rows = min(BQ, p.n_rows - m0);
-    const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(p.d_cache);
-    const __nv_bfloat16 *kv = static_cast<const __nv_bfloat16 *>(p.d_kv) + (size_t)h * (dim8 + vd8);
-    const __nv_bfloat16 *qg = static_cast<const __nv_bfloat16 *>(p.d_q_rows) + ((size_t)m0 * p.heads + h) * QS;
-
-    const int first = p.pos0 + m0, last = first + rows - 1;  // absolute positions of this block's queries
-    const int lo = p.window > 0 && first - p.window + 1 > 0 ? first - p.window + 1 : 0;
-    const int tiles = (last - lo) / BKEY + 1;
-    const int sq = dqk / 8;
-    constexpr int SV = DV / 8;
-    // 16-byte chunks of a [rows][sq] tile go round the threads: (row, chunk) of this thread and its step, no divisions
-    const int r_first = tid / sq, c_first = tid % sq, r_step = NT / sq, c_step = NT % sq;
-
-    for (int r = r_first, c = c_first; r < BQ;) {
-        const bool on = r < rows && c * 8 < QS;
-        cp16(smem_u32(qsm + r * dqs + c * 8), on ? qg + (size_t)r * p.heads * QS + c * 8 : qg, on);
-        r += r_step; c += c_step;
-        if (c >= sq) { c -= sq; ++r; }
-    }
-    auto stage = [&](int tile, int slot) {
-        const uint32_t kd = smem_u32(ksm + slot * BKEY * dqs), vd = smem_u32(vsm + slot * BKEY * VS);
-        const int k0 = lo + tile * BKEY, n = last - k0;      // rows past n hold zeros
-        const __nv_bfloat16 *kvt = kv + (long long)(k0 - p.kv_row0) * p.kv_ld, *crt = cache + (long long)k0 * CS + (R8 - dim8);
-        for (int r = r_first, c = c_first; r < BKEY;) {
-            const bool on = r <= n && c * 8 < QS;
-            const __nv_bfloat16 *src = c * 8 < dim8 ? kvt + (long long)r * p.kv_ld : crt + r * CS;
-            cp16(kd + (r * dqs + c * 8) * 2, on ? src + c * 8 : kv, on);
-            r += r_step; c += c_step;
-            if (c >= sq) { c -= sq; ++r; }
-        }
-#pragma unroll
-        for (int i = 0; i < (BKEY * SV + NT - 1) / NT; ++i) {
-            const int e = tid + i * NT, r = e / SV, c = e % SV;
-            if (BKEY * SV % NT == 0 || r < BKEY) {
-                const bool on = r <= n && c0 + c * 8 < vd8;
-                cp16(vd + (r * VS + c * 8) * 2, on ? kvt + (long long)r * p.kv_ld + dim8 + c0 + c * 8 : kv, on);
-            }
-        }
-        cp_commit();
-    };
-    stage(0, 0);
-
-    float o[DV / 8][4];
-#pragma unroll
-    for (int i = 0; i < DV / 8; ++i)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) o[i][k] = 0.0f;
-    float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};      // maxima of the unscaled scores
-    // this thread's rows: r0 and r0 + 8 of the warp's 16
-    const int r0 = warp * 16 + (lane >> 2);
-    const uint32_t qaddr = smem_u32(qsm + (warp * 16 + (lane & 15)) * dqs + (lane >> 4) * 8);
-    const float sc = p.scale * 1.4426950408889634f;          // weights as powers of two
-
-    for (int tile = 0; tile < tiles; ++tile) {
-        const int slot = stages == 2 ? tile & 1 : 0;
-        if (stages == 2 && tile + 1 < tiles) {
-            stage(tile + 1, slot ^ 1);
-            cp_wait<1>();
-        } else {
-            cp_wait<0>();
-        }
-        __syncthreads();
-        const int k0 = lo + tile * BKEY;
-        // the warp's queries see nothing of this tile: all of it is ahead of them, or has left their windows
-        const int w_first = first + warp * 16, w_last = w_first + 15;
-        const bool idle = k0 > w_last || (p.window > 0 && w_first - (k0 + BKEY - 1) >= p.window);
-        if (!idle) {
-            float s[BKEY / 8][4];
-#pragma unroll
-            for (int i = 0; i < BKEY / 8; ++i)
-#pragma unroll
-                for (int k = 0; k < 4; ++k) s[i][k] = 0.0f;
-            // key rows as the B operand: matrices (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, k 0-7), (keys 8-15, k 8-15)
-            const uint32_t kaddr = smem_u32(ksm + slot * BKEY * dqs + ((lane & 7) + ((lane >> 4) << 3)) * dqs + ((lane >> 3) & 1) * 8);
-#pragma unroll 4
-            for (int kk = 0; kk < dqk; kk += 16) {
-                uint32_t a[4];
-                ldsm4(qaddr + kk * 2, a);
-#pragma unroll
-                for (int n = 0; n < BKEY / 16; ++n) {
-                    uint32_t b[4];
-                    ldsm4(kaddr + (uint32_t)(n * 16 * dqs + kk) * 2, b);
-                    mma_bf16(s[2 * n], a, b[0], b[1]);
-                    mma_bf16(s[2 * n + 1], a, b[2], b[3]);
-                }
-            }
-            // only tiles at an edge of the warp's visible range need the mask
-            if (k0 + BKEY - 1 > w_first || (p.window > 0 && w_last - k0 >= p.window)) {
-                const int span = p.window > 0 ? p.window : 0x7fffffff;
-                const int d0 = first + r0 - k0 - (lane & 3) * 2;
-#pragma unroll
-                for (int n = 0; n < BKEY / 8; ++n)
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) {
-                        const int d = d0 + (k >> 1) * 8 - n * 8 - (k & 1);
-                        if (d < 0 || d >= span) s[n][k] = -INFINITY;
-                    }
-            }
-            float mt[2] = {mx[0], mx[1]};
-#pragma unroll
-            for (int n = 0; n < BKEY / 8; ++n) {
-                mt[0] = fmaxf(mt[0], fmaxf(s[n][0], s[n][1]));
-                mt[1] = fmaxf(mt[1], fmaxf(s[n][2], s[n][3]));
-            }
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 1));
-                mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 2));
-            }
-            // a row with nothing visible so far keeps its maximum at -inf: its weights and its correction are zero
-            // (differences first: the score at the maximum then weighs exactly one, whatever its size)
-            const float base[2] = {mt[0] == -INFINITY ? 0.0f : mt[0], mt[1] == -INFINITY ? 0.0f : mt[1]};
-            const float corr[2] = {ex2((mx[0] - base[0]) * sc), ex2((mx[1] - base[1]) * sc)};
-            const bool moved = mt[0] != mx[0] || mt[1] != mx[1];
-            mx[0] = mt[0]; mx[1] = mt[1];
-            float ls[2] = {0.0f, 0.0f};
-#pragma unroll
-            for (int n = 0; n < BKEY / 8; ++n)
-#pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    s[n][k] = ex2((s[n][k] - base[k >> 1]) * sc);
-                    ls[k >> 1] += s[n][k];
-                }
-            l[0] = fmaf(l[0], corr[0], ls[0]);
-            l[1] = fmaf(l[1], corr[1], ls[1]);
-            if (__any_sync(0xffffffffu, moved)) {
-#pragma unroll
-                for (int i = 0; i < DV / 8; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
-            }
-            // value rows as the B operand, transposed on load: (k 0-7, cols 0-7), (k 8-15, cols 0-7), (k 0-7, cols 8-15), ...
-            const uint32_t vaddr = smem_u32(vsm + slot * BKEY * VS + (lane & 15) * VS + (lane >> 4) * 8);
-#pragma unroll
-            for (int kk = 0; kk < BKEY / 16; ++kk) {
-                const uint32_t a[4] = {pack_bf16(s[2 * kk][0], s[2 * kk][1]), pack_bf16(s[2 * kk][2], s[2 * kk][3]),
-                                       pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3])};
-#pragma unroll
-                for (int n = 0; n < DV / 16; ++n) {
-                    uint32_t b[4];
-                    ldsm4_t(vaddr + (uint32_t)(kk * 16 * VS + n * 16) * 2, b);
-                    mma_bf16(o[2 * n], a, b[0], b[1]);
-                    mma_bf16(o[2 * n + 1], a, b[2], b[3]);
-                }
-            }
-        }
-        __syncthreads();                                     // the slot is overwritten by the next round's copies
-        if (stages == 1 && tile + 1 < tiles) stage(tile + 1, 0);
-    }
-
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
-        l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
-        if (r0 + 8 * r >= rows) continue;
-        const float inv = 1.0f / l[r];
-        const size_t m = (size_t)(m0 + r0 + 8 * r);
-        __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(p.d_out_rows) + m * p.out_ld + (size_t)h * p.vdim;
-        const float *gate = p.d_gate + m * p.proj_ld + (size_t)h * p.vdim;
-#pragma unroll
-        for (int i = 0; i < DV / 8; ++i)
-#pragma unroll
-            for (int k = 0; k < 2; ++k) {
-                const int col = c0 + i * 8 + (lane & 3) * 2 + k;
-                if (col < p.vdim) out[col] = __float2bfloat16_rn(o[i][2 * r + k] * inv * sigmoid_f32(gate[col]));
-            }
-    }
-}
-
 // ------------------------------------------------------------------------------------------------ host side
 
 bool shape_ok(const b200_latent_args *a)
@@ -859,13 +554,6 @@ int launch_pdl(K kern, int gx, int gy, size_t smem, int pdl, cudaStream_t st, Ar
     cfg.numAttrs = pdl ? 1 : 0;
     ++g_b200_launches;
     return (int)cudaLaunchKernelEx(&cfg, kern, args...);
-}
-
-template <typename K>
-int allow_smem(K kern, size_t smem)
-{
-    if (smem > 227 * 1024) return B200_E_TOOLARGE;
-    return smem > 48 * 1024 ? (int)cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) : 0;
 }
 
 template <int WT>
@@ -912,26 +600,20 @@ int decode(const b200_latent_args &a, cudaStream_t st)
     return launch_pdl(latent_value_kernel<WT>, a.heads * vchunks, 1, (size_t)sgroups * R8 * 4, a.use_pdl, st, a, vchunks, sgroups);
 }
 
-template <int DV, int NW>
-int attend_bf16(const b200_latent_args &a, cudaStream_t st)
+// the tiled attention over rows: keys [W_uk c | rotated part], values W_uv c, all heads with rows of their own
+RowAttn row_args(const b200_latent_args &a)
 {
-    const int dqk = (up8(a.dim) + up8(a.rot_dim) + 15) / 16 * 16, dqs = dqk + 8;
-    int stages = 2;
-    auto bytes = [&](int s) { return ((size_t)(NW * 16 + s * BKEY) * dqs + (size_t)s * BKEY * (DV + 8)) * 2; };
-    if (bytes(2) > 227 * 1024) stages = 1;
-    int rc = allow_smem(latent_attend_bf16_kernel<DV, NW>, bytes(stages));
-    if (rc) return rc;
-    const dim3 grid((a.n_rows + NW * 16 - 1) / (NW * 16), a.heads, (a.vdim + DV - 1) / DV);
-    latent_attend_bf16_kernel<DV, NW><<<grid, NW * 32, bytes(stages), st>>>(a, dqs, stages);
-    ++g_b200_launches;
-    return (int)cudaGetLastError();
-}
-
-// 128 query rows a block where that still fills the machine (a tile of keys serves twice the rows), 64 otherwise
-template <int DV>
-int attend_bf16(const b200_latent_args &a, cudaStream_t st)
-{
-    return (long long)((a.n_rows + 127) / 128) * a.heads >= 148 ? attend_bf16<DV, 8>(a, st) : attend_bf16<DV, 4>(a, st);
+    const int dim8 = up8(a.dim), rot8 = up8(a.rot_dim), vd8 = up8(a.vdim), R8 = up8(a.kv_rank), es = a.wtype == B200_WT_F32 ? 4 : 2;
+    RowAttn r = {};
+    r.n_rows = a.n_rows; r.pos0 = a.pos0; r.heads = a.heads; r.group = 1; r.window = a.window;
+    r.dim = a.dim; r.rot_dim = a.rot_dim; r.vdim = a.vdim; r.scale = a.scale;
+    r.q = a.d_q_rows;
+    r.k = a.d_kv; r.k_ld = a.kv_ld; r.k_head = dim8 + vd8; r.kv_row0 = a.kv_row0;
+    r.v = static_cast<const char *>(a.d_kv) + (size_t)dim8 * es; r.v_ld = a.kv_ld; r.v_head = dim8 + vd8;
+    r.k2 = static_cast<const char *>(a.d_cache) + (size_t)R8 * es; r.k2_ld = R8 + rot8;
+    r.gate = a.d_gate; r.gate_ld = a.proj_ld;
+    r.out = a.d_out_rows; r.out_ld = a.out_ld;
+    return r;
 }
 
 }  // namespace
@@ -979,14 +661,7 @@ extern "C" int b200_latent_rows_attend(const b200_latent_args *a, void *stream)
     cudaStream_t st = (cudaStream_t)stream;
     if (a->wtype == B200_WT_BF16) {
         if ((a->kv_ld & 7) || ((uintptr_t)a->d_kv & 15) || ((uintptr_t)a->d_q_rows & 15)) return B200_E_BADARG;
-        if (a->vdim <= 32) return attend_bf16<32>(*a, st);
-        if (a->vdim <= 64) return attend_bf16<64>(*a, st);
-        return attend_bf16<128>(*a, st);
+        return row_attend_bf16<false>(row_args(*a), st);
     }
-    const size_t smem = (size_t)4 * (up8(a->dim) + up8(a->rot_dim)) * 4;
-    int rc = allow_smem(latent_attend_f32_kernel, smem);
-    if (rc) return rc;
-    latent_attend_f32_kernel<<<dim3(a->n_rows, (a->heads + 3) / 4, (a->vdim + 255) / 256), 128, smem, st>>>(*a);
-    ++g_b200_launches;
-    return (int)cudaGetLastError();
+    return row_attend_f32(row_args(*a), st);
 }

@@ -61,14 +61,25 @@ extern "C" int b200_matvec(const b200_matvec_args *ap, void *stream)
         : a.in_mode == B200_IN_POSTNORM ? (!ext || !a.d_in_vec || !a.d_slot_norm_gamma || (a.d_mix_in && !a.d_mix_coef))
         : a.in_mode == B200_IN_EMBED ? (!a.d_emb || !a.d_tokens || !a.d_pos || a.emb_rows <= 0) : true)
         return B200_E_BADARG;
+    const bool streams = a.out_mode == B200_OUT_STREAMS || a.d_norm_beta || a.d_slot_norm_beta || a.d_emb_pos ||
+                         (a.out_mode == B200_OUT_STORE && a.act == B200_ACT_RELU2);
+    // one launch takes its optional parts from one family
+    if (streams && (!ext || a.in_mode == B200_IN_POSTNORM || a.out_mode == B200_OUT_GATED || a.out_mode == B200_OUT_GLU || a.hist_n ||
+                    a.softcap != 0.0f || (a.d_norm_gamma && !a.d_norm_beta)))
+        return B200_E_BADARG;
     if (!ext && (a.out_mode == B200_OUT_GATED || a.norm_dim || a.norm_groups || a.hist_n || a.glu_rows || a.softcap != 0.0f)) return B200_E_BADARG;
     if (ext && (a.norm_dim < 0 || a.norm_dim > a.cols || a.norm_groups < 0 ||
                 (a.norm_groups > 1 && (a.norm_dim > 0 ? a.norm_dim : a.cols) % a.norm_groups) ||
                 a.hist_n < 0 || (a.hist_n > 0 && (!a.d_hist || !a.d_hist_coef || !a.d_hist_out)) ||
                 (a.glu_rows && (a.out_mode != B200_OUT_GLU || a.glu_rows < 0 || a.glu_rows % 2 || a.glu_rows > a.rows || !a.d_out2)) ||
-                (a.in_mode == B200_IN_RESID && a.d_slot_norm_gamma)))
+                (a.in_mode == B200_IN_RESID && a.d_slot_norm_gamma) || (a.d_norm_beta && (!a.d_norm_gamma || a.norm_groups > 1)) ||
+                (a.d_slot_norm_beta && (a.in_mode != B200_IN_EMBED || !a.d_slot_norm_gamma)) ||
+                (a.d_emb_pos && (a.in_mode != B200_IN_EMBED || a.emb_pos_rows < 1)) ||
+                (a.out_mode == B200_OUT_STREAMS && (a.n_streams < 1 || a.n_streams > B200_MAX_STREAMS || !a.d_streams_in || !a.d_streams_out ||
+                                                    !a.d_connect))))
         return B200_E_BADARG;
     if (a.out_mode == B200_OUT_GATED ? (!a.d_out[0] || !a.d_out_resid || !a.d_out_gate || !a.d_out_gate_bias)
+        : a.out_mode == B200_OUT_STREAMS ? !a.d_out[0]
         : a.out_mode == B200_OUT_GLU ? (a.rows % 2 || !a.d_out[0]) : (a.out_mode != B200_OUT_STORE || a.n_out < 1 || a.n_out > B200_MAX_PEERS))
         return B200_E_BADARG;
     if (a.n_wait < 0 || a.n_wait > B200_MAX_PEERS || a.n_signal < 0 || a.n_signal > B200_MAX_PEERS ||
@@ -119,6 +130,7 @@ extern "C" int b200_matvec(const b200_matvec_args *ap, void *stream)
     cudaStream_t st = (cudaStream_t)stream;
     if (a.wtype == B200_WT_Q8)
         return spt == 1 ? launch_by_rows<B200_WT_Q8, 1>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_Q8, 2>(a, geo, rb, grid, st);
+    if (streams) return launch_streams(a, geo, spt, rb, grid, st);
     if (ext) return launch_ext(a, geo, spt, rb, grid, st);
     return spt == 1 ? launch_by_rows<B200_WT_F16, 1>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_F16, 2>(a, geo, rb, grid, st);
 }

@@ -23,8 +23,8 @@
 // (:133-157), residual_add (:369-375), silu_mul / gelu_mul (:337-363), the
 // embedding copy (src/nn/fast_inference.c:386-392) and argmax (:469-476).
 //
-// This header holds the kernel and its launchers; matvec.cu instantiates them for Q8_0 and F16 weights,
-// matvec_ext.cu for BF16 and F32 (two translation units: they compile side by side).
+// This header holds the kernel and its launchers; matvec.cu instantiates them for Q8_0 and F16 weights, matvec_ext.cu
+// and matvec_streams.cu for BF16 and F32 (translation units of their own: they compile side by side).
 #pragma once
 #include "stream_core.cuh"
 #include "../../include/llmb200_kernels.h"
@@ -67,12 +67,55 @@ __device__ __forceinline__ void norm_parts(float (&x)[SPT][E], const int (&col)[
     }
 }
 
-template <int WT, int SPT, int RB, int MAXT>
+// Layer norm (mean taken off, variance of the deviations, weight and bias) of the first `dim` elements, in place; the
+// columns past them hold zeros before and after (their weight and bias are zero).
+template <int SPT, int E>
+__device__ __forceinline__ void layer_norm(float (&x)[SPT][E], const int (&col)[SPT], const float (&gamma)[SPT][E],
+                                           const float (&beta)[SPT][E], int dim, float eps, float *gred, int bar_id, int T, int t)
+{
+    float sum = 0.0f;
+#pragma unroll
+    for (int s = 0; s < SPT; ++s)
+#pragma unroll
+        for (int e = 0; e < E; ++e) sum += x[s][e];
+    const float mean = group_sum(sum, gred, bar_id, T, t) / (float)dim;
+    float ss = 0.0f;
+#pragma unroll
+    for (int s = 0; s < SPT; ++s)
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+            if (col[s] + e < dim) { x[s][e] -= mean; ss = fmaf(x[s][e], x[s][e], ss); }
+    ss = group_sum(ss, gred, bar_id, T, t);
+    const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+    for (int s = 0; s < SPT; ++s)
+#pragma unroll
+        for (int e = 0; e < E; ++e) x[s][e] = fmaf(gamma[s][e], x[s][e] * inv, beta[s][e]);
+}
+
+template <int SPT, int E>
+__device__ __forceinline__ void load_slices(float (&v)[SPT][E], const float *src, const int (&col)[SPT], const bool (&on)[SPT])
+{
+#pragma unroll
+    for (int s = 0; s < SPT; ++s)
+#pragma unroll
+        for (int e = 0; e < E; e += 4) {
+            const float4 v4 = on[s] ? *reinterpret_cast<const float4 *>(src + col[s] + e) : make_float4(0, 0, 0, 0);
+            v[s][e] = v4.x; v[s][e + 1] = v4.y; v[s][e + 2] = v4.z; v[s][e + 3] = v4.w;
+        }
+}
+
+// Which of the optional parts an instantiation holds (registers decide how well the row loop runs): FAM_PLAIN the parts
+// every weight type has, FAM_POST post-norm inputs, gated outputs, depth sums and the logit cap, FAM_STREAMS layer
+// norms, learned positions, residual streams and the squared relu.
+enum { FAM_PLAIN = 0, FAM_POST = 1, FAM_STREAMS = 2 };
+
+template <int WT, int SPT, int RB, int MAXT, int FAM>
 __global__ void __launch_bounds__(MAXT)
 matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
 {
     constexpr int E = (WT == B200_WT_Q8) ? 16 : (WT == B200_WT_F32) ? 4 : 8;       // elements per 16-byte slice
-    constexpr bool EXT = WT == B200_WT_BF16 || WT == B200_WT_F32;   // post-norm inputs, gated outputs, depth sums
+    constexpr bool EXT = FAM == FAM_POST, STR = FAM == FAM_STREAMS;
     extern __shared__ __align__(128) unsigned char smem_raw[];
     const int T = geo.T, NG = geo.NG, nstage = geo.nstage, nwg = T >> 5, nC = NG * T;
     unsigned char *ring = smem_raw;
@@ -84,6 +127,7 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
     int *am_i = reinterpret_cast<int *>(am_v + NG * RB);        // [NG*RB]
     float *xs = reinterpret_cast<float *>(am_i + NG * RB);      // [SPT*T*E] when geo.share_x
     __shared__ int s_last;
+    __shared__ float s_conn[STR ? B200_MAX_STREAMS * (B200_MAX_STREAMS + 2) : 1];     // mix, out, next read of the streams
 
     const int tid = threadIdx.x;
     const int ralign = (p.out_mode == B200_OUT_GLU) ? 2 : 1;
@@ -168,6 +212,15 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
         }
     }
 
+    float gb[STR ? SPT : 1][E];                  // bias of a layer norm
+    if constexpr (STR) {
+        if (pre_gamma && p.d_norm_beta) load_slices<SPT, E>(gb, p.d_norm_beta, col, on);
+        if (p.out_mode == B200_OUT_STREAMS && wg == 0) {         // the epilogue warp of every group, same values
+            for (int i = lane; i < p.n_streams * (p.n_streams + 2); i += 32) s_conn[i] = p.d_connect[i];
+            __syncwarp();
+        }
+    }
+
     pdl_wait();
 
     // Tensor parallel: every rank's partial vector must have landed in `slots`
@@ -237,6 +290,22 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                     x[s][e] = v4.x * p.emb_scale; x[s][e + 1] = v4.y * p.emb_scale;
                     x[s][e + 2] = v4.z * p.emb_scale; x[s][e + 3] = v4.w * p.emb_scale;
                 }
+            if constexpr (STR) {
+                if (p.d_emb_pos) {
+                    float row[SPT][E];
+                    load_slices<SPT, E>(row, p.d_emb_pos + (long long)min(*p.d_pos, p.emb_pos_rows - 1) * p.cols, col, on);
+#pragma unroll
+                    for (int s = 0; s < SPT; ++s)
+#pragma unroll
+                        for (int e = 0; e < E; ++e) x[s][e] += row[s][e];
+                }
+                if (p.d_slot_norm_beta) {
+                    float w[SPT][E], b[SPT][E];
+                    load_slices<SPT, E>(w, p.d_slot_norm_gamma, col, on);
+                    load_slices<SPT, E>(b, p.d_slot_norm_beta, col, on);
+                    layer_norm<SPT, E>(x, col, w, b, p.norm_dim > 0 ? p.norm_dim : p.cols, p.eps, gred, 2 + g, T, t);
+                }
+            }
         } else {
             float sacc[SPT][E];
 #pragma unroll
@@ -288,8 +357,18 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                         *reinterpret_cast<float4 *>(p.d_resid_out + col[s] + e) =
                             make_float4(x[s][e], x[s][e + 1], x[s][e + 2], x[s][e + 3]);
         }
+        if constexpr (STR) {
+            if (p.in_mode == B200_IN_EMBED && p.d_mix_coef) {    // what the first reader takes of the streams, all equal here
+                const float c = *p.d_mix_coef;
+#pragma unroll
+                for (int s = 0; s < SPT; ++s)
+#pragma unroll
+                    for (int e = 0; e < E; ++e) x[s][e] *= c;
+            }
+        }
     }
-    if (EXT && p.d_norm_gamma) {
+    if ((EXT || STR) && p.d_norm_gamma) {
+        if constexpr (STR) layer_norm<SPT, E>(x, col, gm, gb, p.norm_dim > 0 ? p.norm_dim : p.cols, p.eps, gred, 2 + g, T, t);
         if constexpr (EXT)
             norm_parts<SPT, E>(x, col, gm, p.norm_dim > 0 ? p.norm_dim : p.cols, p.norm_groups > 1 ? p.norm_groups : 1, p.eps, gred, 2 + g, T, t);
     } else if (p.d_norm_gamma) {
@@ -358,6 +437,18 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                 o_gate = p.d_out_gate[row0 + lane] + p.d_out_gate_bias[row0 + lane];
             }
         }
+        // Streams: lane = row + RB * j holds streams j, j + 32/RB, ... of its row.
+        constexpr int LPR = 32 / RB, XS = (B200_MAX_STREAMS + LPR - 1) / LPR;
+        float old[STR ? XS : 1];
+        if constexpr (STR) {
+            if (p.out_mode == B200_OUT_STREAMS && wg == 0) {
+#pragma unroll
+                for (int k = 0; k < XS; ++k) {
+                    const int s = lane / RB + k * LPR, r = lane % RB;
+                    old[k] = s < p.n_streams && r < nr ? p.d_streams_in[s * p.streams_in_stride + row0 + r] : 0.0f;
+                }
+            }
+        }
         if (!mbar_wait(&full[slot], (i / nstage) & 1) && p.d_err) *p.d_err = 3;
         const uint32_t sb = ring_s + (uint32_t)slot * geo.slot_bytes;
         // Rows past nr hold stale bytes; they are computed like the others (no predicates in the
@@ -407,8 +498,29 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
                 }
             } else if (EXT && p.out_mode == B200_OUT_GATED) {
                 if (lane < nr) p.d_out[0][p.out_offset + row] = fmaf(p.resid_alpha, o_resid, sigmoid_f32(o_gate) * y);
+            } else if (STR && p.out_mode == B200_OUT_STREAMS) {
+                if constexpr (STR) {
+                    const int n = p.n_streams, r = lane % RB;
+                    const float yr = __shfl_sync(0xffffffffu, y, r);
+                    float next = 0.0f;
+                    for (int to = 0; to < n; ++to) {
+                        float a = 0.0f;
+#pragma unroll
+                        for (int k = 0; k < XS; ++k) {
+                            const int s = lane / RB + k * LPR;
+                            if (s < n) a = fmaf(s_conn[s * n + to], old[k], a);
+                        }
+#pragma unroll
+                        for (int o = RB; o < 32; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+                        a = fmaf(s_conn[n * n + to], yr, a);
+                        if (r < nr && lane / RB == to % LPR) p.d_streams_out[to * p.streams_out_stride + row0 + r] = a;
+                        next = fmaf(s_conn[n * n + n + to], a, next);
+                    }
+                    if (lane < nr) p.d_out[0][p.out_offset + row] = next;
+                }
             } else if (lane < nr) {
                 if (EXT && p.softcap > 0.0f) y = p.softcap * tanhf(y / p.softcap);
+                if (STR && p.act == B200_ACT_RELU2) y = act_relu2(y);
                 for (int q = 0; q < p.n_out; ++q) p.d_out[q][p.out_offset + row] = y;
                 if (better(y, row, best_v, best_i)) { best_v = y; best_i = row; }
             }
@@ -471,14 +583,14 @@ matvec_kernel(const __grid_constant__ b200_matvec_args p, const Geometry geo)
     }
 }
 
-template <int WT, int SPT, int RB, int MAXT>
+template <int WT, int SPT, int RB, int MAXT, int FAM>
 int launch(const b200_matvec_args &a, const Geometry &geo, int grid, cudaStream_t st)
 {
     const int nwg = geo.T / 32;
     const size_t smem = (size_t)geo.nstage * geo.slot_bytes + (size_t)geo.nstage * 16 +
                         ((size_t)geo.NG * 2 * nwg * RB + (size_t)geo.NG * 32 + (size_t)geo.NG * RB * 2) * sizeof(float) +
                         (geo.share_x ? (size_t)SPT * geo.T * (WT == B200_WT_Q8 ? 16 : WT == B200_WT_F32 ? 4 : 8) * sizeof(float) : 0);
-    auto kern = matvec_kernel<WT, SPT, RB, MAXT>;
+    auto kern = matvec_kernel<WT, SPT, RB, MAXT, FAM>;
     if (smem > 220 * 1024) return B200_E_TOOLARGE;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -498,27 +610,36 @@ int launch(const b200_matvec_args &a, const Geometry &geo, int grid, cudaStream_
     return (int)cudaLaunchKernelEx(&cfg, kern, a, geo);
 }
 
-template <int WT, int SPT, int RB>
+template <int WT, int SPT, int RB, int FAM>
 int launch_by_size(const b200_matvec_args &a, const Geometry &geo, int grid, cudaStream_t st)
 {
     const int threads = geo.NG * geo.T + 32;
-    if (threads <= 672) return launch<WT, SPT, RB, 672>(a, geo, grid, st);
-    return launch<WT, SPT, RB, 1024>(a, geo, grid, st);
+    if (threads <= 672) return launch<WT, SPT, RB, 672, FAM>(a, geo, grid, st);
+    return launch<WT, SPT, RB, 1024, FAM>(a, geo, grid, st);
 }
 
-template <int WT, int SPT>
+template <int WT, int SPT, int FAM = FAM_PLAIN>
 int launch_by_rows(const b200_matvec_args &a, const Geometry &geo, int rb, int grid, cudaStream_t st)
 {
     switch (rb) {
-    case 8: return launch_by_size<WT, SPT, 8>(a, geo, grid, st);
-    case 4: return launch_by_size<WT, SPT, 4>(a, geo, grid, st);
-    case 2: return launch_by_size<WT, SPT, 2>(a, geo, grid, st);
-    default: return launch_by_size<WT, SPT, 1>(a, geo, grid, st);
+    case 8: return launch_by_size<WT, SPT, 8, FAM>(a, geo, grid, st);
+    case 4: return launch_by_size<WT, SPT, 4, FAM>(a, geo, grid, st);
+    case 2: return launch_by_size<WT, SPT, 2, FAM>(a, geo, grid, st);
+    default: return launch_by_size<WT, SPT, 1, FAM>(a, geo, grid, st);
     }
 }
 
 
-// BF16 / F32 weights (matvec_ext.cu)
-int launch_ext(const b200_matvec_args &a, const Geometry &geo, int spt, int rb, int grid, cudaStream_t st);
+// BF16 / F32 weights
+template <int FAM>
+int launch_typed(const b200_matvec_args &a, const Geometry &geo, int spt, int rb, int grid, cudaStream_t st)
+{
+    if (a.wtype == B200_WT_BF16)
+        return spt == 1 ? launch_by_rows<B200_WT_BF16, 1, FAM>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_BF16, 2, FAM>(a, geo, rb, grid, st);
+    return spt == 1 ? launch_by_rows<B200_WT_F32, 1, FAM>(a, geo, rb, grid, st)
+         : spt == 2 ? launch_by_rows<B200_WT_F32, 2, FAM>(a, geo, rb, grid, st) : launch_by_rows<B200_WT_F32, 4, FAM>(a, geo, rb, grid, st);
+}
+int launch_ext(const b200_matvec_args &a, const Geometry &geo, int spt, int rb, int grid, cudaStream_t st);        // matvec_ext.cu
+int launch_streams(const b200_matvec_args &a, const Geometry &geo, int spt, int rb, int grid, cudaStream_t st);    // matvec_streams.cu
 
 } // namespace b200_mv

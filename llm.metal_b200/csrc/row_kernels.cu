@@ -1,5 +1,5 @@
 // Row-wise steps of a prompt portion (sm_100a): embedding, grouped RMS norms after a gated, scaled residual sum,
-// the depth average over earlier layers' results, GeGLU and the logit cap. One block per row; every sum is formed
+// the depth average over earlier layers' results, layer norms, residual streams, GeGLU and the logit cap. One block per row; every sum is formed
 // in a fixed order. Results that a tensor-core product reads next are written as bfloat16 too.
 #include "stream_core.cuh"
 #include "../../include/llmb200_kernels.h"
@@ -79,6 +79,120 @@ rows_norm_kernel(const float *x, const int *index, int dim, int ld, int groups, 
     part_scales(row, dim, groups, eps, red, inv);
     const int len = dim / groups;
     for (int i = threadIdx.x; i < ld; i += 256) out[m * ld + i] = (T)(i < dim ? gamma[i] * (row[i] * inv[i / len]) : 0.0f);
+}
+
+__device__ __forceinline__ void store4(float *out, const float4 &v) { *reinterpret_cast<float4 *>(out) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16 *out, const float4 &v)
+{
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(out) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+
+// Layer norm of row[0 .. dim) (shared memory; this thread wrote quads threadIdx.x + 256 k, `sum` is the sum of what it
+// wrote, elements past dim are zeros). Every quad below ld goes through `put` with its normalised value.
+template <typename Put>
+__device__ __forceinline__ void layer_norm_row(float *row, float sum, int dim, int ld, float eps, const float *gamma, const float *beta,
+                                               float *red, Put put)
+{
+    const float mean = block_sum(sum, red) / (float)dim;
+    float ss = 0.0f;
+    for (int i = 4 * threadIdx.x; i < ld; i += 1024)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+            if (i + e < dim) { const float d = row[i + e] - mean; ss = fmaf(d, d, ss); }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dim + eps);
+    for (int i = 4 * threadIdx.x; i < ld; i += 1024) {
+        const float4 x = *reinterpret_cast<const float4 *>(row + i), g = *reinterpret_cast<const float4 *>(gamma + i), b = *reinterpret_cast<const float4 *>(beta + i);
+        put(i, make_float4(fmaf(g.x, (x.x - mean) * inv, b.x), fmaf(g.y, (x.y - mean) * inv, b.y),
+                           fmaf(g.z, (x.z - mean) * inv, b.z), fmaf(g.w, (x.w - mean) * inv, b.w)));
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) rows_streams_kernel(const b200_rows_streams_args p)
+{
+    extern __shared__ __align__(16) float row[];             // [ld]
+    __shared__ float red[33], conn[B200_MAX_STREAMS * (B200_MAX_STREAMS + 2)];
+    const int n = p.n_streams;
+    if ((int)threadIdx.x < n * (n + 2)) conn[threadIdx.x] = p.connect[threadIdx.x];
+    __syncthreads();
+    const size_t m = blockIdx.x;
+    const float *xin = p.streams_in + m * p.ld, *y = p.y + m * p.y_ld;
+    float sum = 0.0f;
+    for (int i = 4 * threadIdx.x; i < p.ld; i += 1024) {
+        float4 x[B200_MAX_STREAMS];
+#pragma unroll
+        for (int s = 0; s < B200_MAX_STREAMS; ++s)
+            if (s < n) x[s] = *reinterpret_cast<const float4 *>(xin + s * p.streams_in_stride + i);
+        const float4 yv = *reinterpret_cast<const float4 *>(y + i);
+        float4 u = make_float4(0, 0, 0, 0);
+        for (int t = 0; t < n; ++t) {
+            const float c = conn[n * n + t], take = conn[n * n + n + t];
+            float4 a = make_float4(c * yv.x, c * yv.y, c * yv.z, c * yv.w);
+#pragma unroll
+            for (int s = 0; s < B200_MAX_STREAMS; ++s)
+                if (s < n) {
+                    const float w = conn[s * n + t];
+                    a.x = fmaf(w, x[s].x, a.x); a.y = fmaf(w, x[s].y, a.y); a.z = fmaf(w, x[s].z, a.z); a.w = fmaf(w, x[s].w, a.w);
+                }
+            if (p.streams_out) *reinterpret_cast<float4 *>(p.streams_out + t * p.streams_out_stride + m * p.ld + i) = a;
+            u.x = fmaf(take, a.x, u.x); u.y = fmaf(take, a.y, u.y); u.z = fmaf(take, a.z, u.z); u.w = fmaf(take, a.w, u.w);
+        }
+        if (p.u_out) *reinterpret_cast<float4 *>(p.u_out + m * p.ld + i) = u;
+        *reinterpret_cast<float4 *>(row + i) = u;
+        sum += (u.x + u.y) + (u.z + u.w);
+    }
+    if (!p.out) return;
+    T *out = static_cast<T *>(p.out) + m * p.ld;
+    layer_norm_row(row, sum, p.dim, p.ld, p.eps, p.gamma, p.beta, red, [&](int i, const float4 &v) { store4(out + i, v); });
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) rows_start_kernel(const b200_rows_start_args p)
+{
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[33];
+    const size_t m = blockIdx.x;
+    uint32_t t = p.tokens[m];
+    if (t >= (uint32_t)p.vocab) t = 0;                       // never outside the table
+    const float *e = p.emb + (size_t)t * p.ld, *q = p.emb_pos + (size_t)min(p.pos0 + (int)m, p.pos_rows - 1) * p.ld;
+    float sum = 0.0f;
+    for (int i = 4 * threadIdx.x; i < p.ld; i += 1024) {
+        const float4 a = *reinterpret_cast<const float4 *>(e + i), b = *reinterpret_cast<const float4 *>(q + i);
+        const float4 v = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+        *reinterpret_cast<float4 *>(row + i) = v;
+        sum += (v.x + v.y) + (v.z + v.w);
+    }
+    const float take = *p.take;
+    float *x = p.x + m * p.ld, next = 0.0f;
+    layer_norm_row(row, sum, p.dim, p.ld, p.eps, p.emb_gamma, p.emb_beta, red, [&](int i, const float4 &v) {
+        store4(x + i, v);
+        const float4 u = make_float4(take * v.x, take * v.y, take * v.z, take * v.w);
+        *reinterpret_cast<float4 *>(row + i) = u;            // this thread's own quad
+        next += (u.x + u.y) + (u.z + u.w);
+    });
+    T *out = static_cast<T *>(p.out) + m * p.ld;
+    layer_norm_row(row, next, p.dim, p.ld, p.eps, p.gamma, p.beta, red, [&](int i, const float4 &v) { store4(out + i, v); });
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+rows_layer_norm_kernel(const float *x, const int *index, int dim, int ld, float eps, const float *gamma, const float *beta, T *out)
+{
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[33];
+    const size_t m = blockIdx.x, src = index ? (size_t)index[m] : m;
+    float sum = 0.0f;
+    for (int i = 4 * threadIdx.x; i < ld; i += 1024) {
+        float4 v = *reinterpret_cast<const float4 *>(x + src * ld + i);
+        float *e = &v.x;
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+            if (i + k >= dim) e[k] = 0.0f;
+        *reinterpret_cast<float4 *>(row + i) = v;
+        sum += (v.x + v.y) + (v.z + v.w);
+    }
+    layer_norm_row(row, sum, dim, ld, eps, gamma, beta, red, [&](int i, const float4 &v) { store4(out + m * ld + i, v); });
 }
 
 template <typename T>
@@ -172,5 +286,61 @@ extern "C" int b200_rows_softcap(float *x, int rows, int dim, long long ld, floa
 {
     if (!x || rows <= 0 || dim <= 0 || ld < dim || !(cap > 0.0f)) return B200_E_BADARG;
     rows_softcap_kernel<<<grid_for((size_t)rows * dim), 256, 0, (cudaStream_t)stream>>>(x, rows, dim, ld, cap);
+    return done();
+}
+
+static bool typed(int wtype) { return wtype == B200_WT_BF16 || wtype == B200_WT_F32; }
+
+extern "C" int b200_rows_streams(const b200_rows_streams_args *a, void *stream)
+{
+    if (!a || !a->streams_in || !a->y || !a->connect || a->n_streams < 1 || a->n_streams > B200_MAX_STREAMS || a->rows <= 0 || a->dim <= 0 ||
+        a->ld < a->dim || (a->ld & 3) || (a->y_ld & 3) || a->y_ld < a->ld || (a->streams_in_stride & 3) || (a->streams_out_stride & 3) ||
+        (a->out && (!a->gamma || !a->beta || !typed(a->wtype))) || (!a->out && !a->streams_out && !a->u_out))
+        return B200_E_BADARG;
+    const size_t smem = (size_t)a->ld * 4;
+    cudaStream_t st = (cudaStream_t)stream;
+    int rc;
+    if (a->wtype == B200_WT_F32) {
+        if ((rc = row_smem(rows_streams_kernel<float>, smem)) != 0) return rc;
+        rows_streams_kernel<float><<<a->rows, 256, smem, st>>>(*a);
+    } else {
+        if ((rc = row_smem(rows_streams_kernel<__nv_bfloat16>, smem)) != 0) return rc;
+        rows_streams_kernel<__nv_bfloat16><<<a->rows, 256, smem, st>>>(*a);
+    }
+    return done();
+}
+
+extern "C" int b200_rows_start(const b200_rows_start_args *a, void *stream)
+{
+    if (!a || !a->emb || !a->emb_pos || !a->tokens || !a->emb_gamma || !a->emb_beta || !a->take || !a->gamma || !a->beta || !a->x || !a->out ||
+        a->rows <= 0 || a->dim <= 0 || a->ld < a->dim || (a->ld & 3) || a->vocab <= 0 || a->pos_rows <= 0 || a->pos0 < 0 || !typed(a->wtype))
+        return B200_E_BADARG;
+    const size_t smem = (size_t)a->ld * 4;
+    cudaStream_t st = (cudaStream_t)stream;
+    int rc;
+    if (a->wtype == B200_WT_F32) {
+        if ((rc = row_smem(rows_start_kernel<float>, smem)) != 0) return rc;
+        rows_start_kernel<float><<<a->rows, 256, smem, st>>>(*a);
+    } else {
+        if ((rc = row_smem(rows_start_kernel<__nv_bfloat16>, smem)) != 0) return rc;
+        rows_start_kernel<__nv_bfloat16><<<a->rows, 256, smem, st>>>(*a);
+    }
+    return done();
+}
+
+extern "C" int b200_rows_layer_norm(const float *x, const int *index, int rows, int dim, int ld, float eps,
+                                    const float *gamma, const float *beta, int wtype, void *out, void *stream)
+{
+    if (!x || !gamma || !beta || !out || rows <= 0 || dim <= 0 || ld < dim || (ld & 3) || !typed(wtype)) return B200_E_BADARG;
+    const size_t smem = (size_t)ld * 4;
+    cudaStream_t st = (cudaStream_t)stream;
+    int rc;
+    if (wtype == B200_WT_F32) {
+        if ((rc = row_smem(rows_layer_norm_kernel<float>, smem)) != 0) return rc;
+        rows_layer_norm_kernel<float><<<rows, 256, smem, st>>>(x, index, dim, ld, eps, gamma, beta, static_cast<float *>(out));
+    } else {
+        if ((rc = row_smem(rows_layer_norm_kernel<__nv_bfloat16>, smem)) != 0) return rc;
+        rows_layer_norm_kernel<__nv_bfloat16><<<rows, 256, smem, st>>>(x, index, dim, ld, eps, gamma, beta, static_cast<__nv_bfloat16 *>(out));
+    }
     return done();
 }

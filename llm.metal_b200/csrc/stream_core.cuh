@@ -137,6 +137,8 @@ __device__ __forceinline__ float act_gelu_tanh(float g)
     return 0.5f * g * (1.0f + tanhf(inner));
 }
 
+__device__ __forceinline__ float act_relu2(float g) { const float r = fmaxf(g, 0.0f); return r * r; }
+
 __device__ __forceinline__ bool better(float v, int i, float bv, int bi)
 {
     return v > bv || (v == bv && i < bi);

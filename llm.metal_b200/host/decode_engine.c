@@ -1143,7 +1143,6 @@ static int generate_one(InferenceState *s, const uint32_t *prompt, int prompt_le
      * reads the ids back in groups: one small copy and one event per TOK_BATCH forwards (a copy after every
      * forward sits between two launches on the stream and cost 0.8 % of the decode rate), two groups in flight.
      * After an EOS id the forwards already launched are simply not used. */
-    enum { TOK_BATCH = 4 };
     int max_fw = max_gen_len - 1;
     if (max_fw > s->max_seq - P) max_fw = s->max_seq - P;
     int launched = 0, done = 0, copied = 0, b_enq = 0, b_done = 0, stop = is_eos(s, next) || max_fw <= 0;

@@ -20,6 +20,11 @@ typedef struct {
 
 enum { K_QKV = 0, K_ATTN, K_O, K_GATEUP, K_DOWN, K_LM, K_KINDS };
 
+/* The generate loop lets forwards run ahead of the ids it has read: ids are read in groups of TOK_BATCH, two groups in
+ * flight, and after an end id the forwards already launched are not used. State that is not addressed by position has to
+ * reach RUN_AHEAD positions back. */
+enum { TOK_BATCH = 4, RUN_AHEAD = 2 * TOK_BATCH };
+
 /* What a model type brings to the engine. The engine owns the control words, the per-token graphs, the generate
  * loop, positions, EOS handling and measurement; a model type enqueues its kernels. */
 typedef struct {

@@ -20,8 +20,8 @@
  *   rows        a portion of several tokens, up to ROW_CHUNK at a time: the same matrices as tensor-core products
  *               (fp32: CUDA-core products) with row kernels in between.
  *
- * Layouts: up8(n) = n rounded up to a multiple of 8. Matrices get zero padding columns up to up8(cols) and sections
- * of fused matrices zero padding rows up to up8(rows), vectors zero padding to match, so every size works.
+ * Layouts: llmb200_up8(n) = n rounded up to a multiple of 8. Matrices get zero padding columns up to llmb200_up8(cols) and sections
+ * of fused matrices zero padding rows up to llmb200_up8(rows), vectors zero padding to match, so every size works.
  */
 #include "model_dir.h"
 #include "../../include/llmb200_train_kernels.h"
@@ -30,18 +30,16 @@
 #include <stdlib.h>
 #include <string.h>
 
-enum { ROW_CHUNK = 2048, WANT_CHUNK = 256 };
-
 typedef struct {
     int heads, dim, rot_dim, rot_dims, vdim, kv_rank, window, ff;
     float scale;
     double rot_base;
     PackedMat in, uk_t, kv, o, gu, down;
     int o_dkv, o_gate, o_rg1;        /* row offsets in `in`; q is at 0 */
-    int ffp;                         /* up8(ff): gate/up pairs 0 .. 2 ffp, residual gate after them */
+    int ffp;                         /* llmb200_up8(ff): gate/up pairs 0 .. 2 ffp, residual gate after them */
     float *dkv_gamma, *norm1, *norm2, *b1, *b2, *dwa;
     const float *rope;
-    void *cache;                     /* [max_seq][up8(kv_rank) + up8(rot_dim)] */
+    void *cache;                     /* [max_seq][llmb200_up8(kv_rank) + llmb200_up8(rot_dim)] */
     int n_split;
 } LLayer;
 
@@ -55,60 +53,14 @@ typedef struct {
     void *qlat;
     float *proj, *part, *attn, *z, *u, *rg2, *act, *hist, *mix, *x;
     /* rows (allocated at the first portion) */
-    int chunk;
-    float *r_proj, *r_hist, *r_x, *r_u, *r_y, *r_gu, *r_logits;
-    void *r_xh, *r_q, *r_kv, *r_attn, *r_act, *r_last;
-    int *d_want, *h_want;
+    RowPath rows;
+    float *r_proj, *r_hist, *r_x, *r_u, *r_y, *r_gu;
+    void *r_xh, *r_q, *r_kv, *r_attn, *r_act;
 } Latent;
 
-static int up8(int n) { return (n + 7) & ~7; }
 static int imax(int a, int b) { return a > b ? a : b; }
 
 /* ------------------------------------------------------------ loading */
-
-/* rows x up8(cols), zero; at least 64 rows, the narrowest matrix the tensor-core product takes */
-static int new_mat(InferenceState *s, PackedMat *m, int rows, int cols)
-{
-    m->rows = imax(64, up8(rows));
-    m->cols = up8(cols);
-    m->stride = (long long)b200_packed_row_stride(s->wtype, m->cols);
-    m->w = llmb200_dev_zero((size_t)m->stride * m->rows);
-    return m->w ? 0 : -1;
-}
-
-static int put_rows(InferenceState *s, PackedMat *m, const float *src, int rows, int cols, int row0, int step)
-{
-    return llmb200_upload_packed(s->wtype, src, cols, rows, 0, cols, m->w, m->stride, row0, step);
-}
-
-typedef struct { const llmb200_tensor_file *file; int layer; int failed; } Source;
-
-/* Tensor "l<layer>.<name>" (layer < 0: "<name>") as fp32 on the host; the caller frees it. */
-static float *tensor(Source *src, const char *name, long long d0, long long d1)
-{
-    char full[128];
-    if (src->layer >= 0) snprintf(full, sizeof(full), "l%d.%s", src->layer, name);
-    else snprintf(full, sizeof(full), "%s", name);
-    float *t = llmb200_tensor_f32(src->file, full, d0, d1);
-    if (!t) src->failed = 1;
-    return t;
-}
-
-static void load_rows(InferenceState *s, Source *src, PackedMat *m, const char *name, int rows, int cols, int row0, int step)
-{
-    float *t = tensor(src, name, rows, cols);
-    if (t && put_rows(s, m, t, rows, cols, row0, step) != 0) src->failed = 1;
-    free(t);
-}
-
-/* A vector of n elements, zero-padded to `padded` on the device. */
-static float *load_vec(Source *src, const char *name, int n, int padded)
-{
-    float *t = tensor(src, name, n, 0), *d = t ? llmb200_dev_zero((size_t)padded * 4) : NULL;
-    if (!d || llmb200_upload_f32_into(d, t, (size_t)n) != 0) src->failed = 1;
-    free(t);
-    return d;
-}
 
 /* (cos, sin) of pos * base^(-2i/dims), formed in double; one table per distinct (base, dims). */
 static const float *rope_table(InferenceState *s, Latent *m, int layer)
@@ -136,50 +88,50 @@ static const float *rope_table(InferenceState *s, Latent *m, int layer)
 static int load_layer(InferenceState *s, Latent *m, int li, const llmb200_tensor_file *file)
 {
     LLayer *y = &m->layers[li];
-    Source src = { file, li, 0 };
-    const int D = s->D, H = y->heads, R = y->kv_rank, dim8 = up8(y->dim), vd8 = up8(y->vdim), per = dim8 + vd8;
+    TensorSource src = { file, li, 0 };
+    const int D = s->D, H = y->heads, R = y->kv_rank, dim8 = llmb200_up8(y->dim), vd8 = llmb200_up8(y->vdim), per = dim8 + vd8;
     const int q_rows = H * (y->dim + y->rot_dim), hv = H * y->vdim;
-    y->o_dkv = up8(q_rows);
-    y->o_gate = y->o_dkv + up8(R + y->rot_dim);
-    y->o_rg1 = y->o_gate + up8(hv);
-    if (new_mat(s, &y->in, y->o_rg1 + m->Dp, D) || new_mat(s, &y->uk_t, H * R, y->dim) || new_mat(s, &y->kv, H * per, R) ||
-        new_mat(s, &y->o, D, hv))
+    y->o_dkv = llmb200_up8(q_rows);
+    y->o_gate = y->o_dkv + llmb200_up8(R + y->rot_dim);
+    y->o_rg1 = y->o_gate + llmb200_up8(hv);
+    if (llmb200_new_mat(s, &y->in, y->o_rg1 + m->Dp, D) || llmb200_new_mat(s, &y->uk_t, H * R, y->dim) || llmb200_new_mat(s, &y->kv, H * per, R) ||
+        llmb200_new_mat(s, &y->o, D, hv))
         return -1;
-    load_rows(s, &src, &y->in, "mix.q", q_rows, D, 0, 1);
-    load_rows(s, &src, &y->in, "mix.dkv", R + y->rot_dim, D, y->o_dkv, 1);
-    load_rows(s, &src, &y->in, "mix.g", hv, D, y->o_gate, 1);
-    load_rows(s, &src, &y->in, "rg1", D, D, y->o_rg1, 1);
-    load_rows(s, &src, &y->o, "mix.o", D, hv, 0, 1);
+    llmb200_load_rows(s, &src, &y->in, "mix.q", q_rows, D, 0, 1);
+    llmb200_load_rows(s, &src, &y->in, "mix.dkv", R + y->rot_dim, D, y->o_dkv, 1);
+    llmb200_load_rows(s, &src, &y->in, "mix.g", hv, D, y->o_gate, 1);
+    llmb200_load_rows(s, &src, &y->in, "rg1", D, D, y->o_rg1, 1);
+    llmb200_load_rows(s, &src, &y->o, "mix.o", D, hv, 0, 1);
 
     /* the two expansions: side by side per head for the rows path, W_uk transposed per head for one token */
-    float *uk = tensor(&src, "mix.uk", (long long)H * y->dim, R), *uv = tensor(&src, "mix.uv", hv, R);
+    float *uk = llmb200_source_tensor(&src, "mix.uk", (long long)H * y->dim, R), *uv = llmb200_source_tensor(&src, "mix.uv", hv, R);
     float *t = malloc((size_t)R * y->dim * sizeof(float));
     if (uk && uv && t)
         for (int h = 0; h < H && !src.failed; ++h) {
             const float *k = uk + (size_t)h * y->dim * R;
             for (int d = 0; d < y->dim; ++d)
                 for (int r = 0; r < R; ++r) t[(size_t)r * y->dim + d] = k[(size_t)d * R + r];
-            if (put_rows(s, &y->uk_t, t, R, y->dim, h * R, 1) || put_rows(s, &y->kv, k, y->dim, R, h * per, 1) ||
-                put_rows(s, &y->kv, uv + (size_t)h * y->vdim * R, y->vdim, R, h * per + dim8, 1))
+            if (llmb200_put_rows(s, &y->uk_t, t, R, y->dim, h * R, 1) || llmb200_put_rows(s, &y->kv, k, y->dim, R, h * per, 1) ||
+                llmb200_put_rows(s, &y->kv, uv + (size_t)h * y->vdim * R, y->vdim, R, h * per + dim8, 1))
                 src.failed = 1;
         }
     free(uk); free(uv); free(t);
 
-    y->dkv_gamma = load_vec(&src, "mix.dkv.norm", R, up8(R));
-    y->norm1 = load_vec(&src, "norm1", D, m->Dp);
-    y->b1 = load_vec(&src, "rg1.b", D, m->Dp);
-    y->dwa = load_vec(&src, "dwa", li + 2, li + 2);
+    y->dkv_gamma = llmb200_load_vec(&src, "mix.dkv.norm", R, llmb200_up8(R));
+    y->norm1 = llmb200_load_vec(&src, "norm1", D, m->Dp);
+    y->b1 = llmb200_load_vec(&src, "rg1.b", D, m->Dp);
+    y->dwa = llmb200_load_vec(&src, "dwa", li + 2, li + 2);
     if (y->ff) {
-        y->ffp = up8(y->ff);
-        if (new_mat(s, &y->gu, 2 * y->ffp + m->Dp, D) || new_mat(s, &y->down, D, y->ff)) return -1;
-        load_rows(s, &src, &y->gu, "mlp.gate", y->ff, D, 0, 2);
-        load_rows(s, &src, &y->gu, "mlp.up", y->ff, D, 1, 2);
-        load_rows(s, &src, &y->gu, "rg2", D, D, 2 * y->ffp, 1);
-        load_rows(s, &src, &y->down, "mlp.down", D, y->ff, 0, 1);
-        y->norm2 = load_vec(&src, "norm2", D, m->Dp);
-        y->b2 = load_vec(&src, "rg2.b", D, m->Dp);
+        y->ffp = llmb200_up8(y->ff);
+        if (llmb200_new_mat(s, &y->gu, 2 * y->ffp + m->Dp, D) || llmb200_new_mat(s, &y->down, D, y->ff)) return -1;
+        llmb200_load_rows(s, &src, &y->gu, "mlp.gate", y->ff, D, 0, 2);
+        llmb200_load_rows(s, &src, &y->gu, "mlp.up", y->ff, D, 1, 2);
+        llmb200_load_rows(s, &src, &y->gu, "rg2", D, D, 2 * y->ffp, 1);
+        llmb200_load_rows(s, &src, &y->down, "mlp.down", D, y->ff, 0, 1);
+        y->norm2 = llmb200_load_vec(&src, "norm2", D, m->Dp);
+        y->b2 = llmb200_load_vec(&src, "rg2.b", D, m->Dp);
     }
-    const size_t row = (size_t)(up8(R) + up8(y->rot_dim)) * m->es;
+    const size_t row = (size_t)(llmb200_up8(R) + llmb200_up8(y->rot_dim)) * m->es;
     y->cache = llmb200_dev_zero(row * s->max_seq);
     y->rope = rope_table(s, m, li);
     y->n_split = b200_latent_splits(H, y->window, s->max_seq);
@@ -192,35 +144,29 @@ static int load_layer(InferenceState *s, Latent *m, int li, const llmb200_tensor
     return 0;
 }
 
-static int bad_config(const char *where, const char *what)
-{
-    fprintf(stderr, "[FastGen] config.json: %s: %s\n", where, what);
-    return -1;
-}
-
 static int parse_layer(const json *e, int i, LLayer *y)
 {
     char where[32];
     snprintf(where, sizeof(where), "layer %d", i);
     const char *type = json_string(e, "type");
-    if (!type || strcmp(type, "latent_attention")) return bad_config(where, "the mixer type is not latent_attention");
+    if (!type || strcmp(type, "latent_attention")) return llmb200_bad_config(where, "the mixer type is not latent_attention");
     const json *x = json_get(e, "mixer"), *rot = json_get(x, "rot"), *mask = json_get(x, "mask"), *mlp = json_get(e, "mlp");
     double scale;
     if (json_int(x, "heads", &y->heads) || json_int(x, "dim", &y->dim) || json_int(x, "rot_dim", &y->rot_dim) ||
         json_int(x, "vdim", &y->vdim) || json_int(x, "kv_rank", &y->kv_rank) || json_number(x, "scale", &scale) ||
         json_number(rot, "base", &y->rot_base))
-        return bad_config(where, "a size or constant of the mixer is missing");
+        return llmb200_bad_config(where, "a size or constant of the mixer is missing");
     y->scale = (float)scale;
     if (json_int(rot, "dims", &y->rot_dims)) y->rot_dims = y->rot_dim;
     if (mask && mask->type != JSON_NULL && (json_int(mask, "size", &y->window) || y->window < 1))
-        return bad_config(where, "mask.size must be a positive integer");
+        return llmb200_bad_config(where, "mask.size must be a positive integer");
     if (y->heads < 1 || y->dim < 1 || y->rot_dim < 1 || y->vdim < 1 || y->kv_rank < 1 || y->rot_dims < 0 || y->rot_dims > y->rot_dim ||
         y->rot_dims % 2 || !(y->rot_base > 0))
-        return bad_config(where, "a size of the mixer is out of range");
+        return llmb200_bad_config(where, "a size of the mixer is out of range");
     if (mlp && mlp->type != JSON_NULL) {
         const char *kind = json_string(mlp, "kind");
-        if (!kind || strcmp(kind, "dense")) return bad_config(where, "the feed-forward kind is not dense");
-        if (json_int(mlp, "ff", &y->ff) || y->ff < 1) return bad_config(where, "mlp.ff must be a positive integer");
+        if (!kind || strcmp(kind, "dense")) return llmb200_bad_config(where, "the feed-forward kind is not dense");
+        if (json_int(mlp, "ff", &y->ff) || y->ff < 1) return llmb200_bad_config(where, "mlp.ff must be a positive integer");
     }
     return 0;
 }
@@ -236,11 +182,11 @@ static int parse(InferenceState *s, Latent *m, const json *c)
     double eps, alpha, emb, cap = 0.0;
     if (json_int(c, "vocab", &s->V) || json_int(c, "width", &s->D) || json_number(norm, "eps", &eps) ||
         json_number(c, "postln_alpha", &alpha) || json_number(json_get(c, "embedding"), "scale", &emb))
-        return bad_config("model", "a size or constant is missing");
+        return llmb200_bad_config("model", "a size or constant is missing");
     if (json_int(norm, "groups", &m->groups)) m->groups = 1;
     json_number(c, "logit_softcap", &cap);
-    if (s->V < 1 || s->D < 1 || m->groups < 1 || s->D % m->groups) return bad_config("model", "a size is out of range");
-    if (!layers || layers->type != JSON_ARRAY || layers->n < 1) return bad_config("model", "layers must be a list");
+    if (s->V < 1 || s->D < 1 || m->groups < 1 || s->D % m->groups) return llmb200_bad_config("model", "a size is out of range");
+    if (!layers || layers->type != JSON_ARRAY || layers->n < 1) return llmb200_bad_config("model", "layers must be a list");
     m->eps = (float)eps; m->alpha = (float)alpha; m->softcap = (float)cap;
     s->emb_scale = (float)emb;
     s->L = layers->n;
@@ -255,42 +201,30 @@ static int parse(InferenceState *s, Latent *m, const json *c)
 
 InferenceState *llmb200_create_morilorn(const json *config, const llmb200_tensor_file *tensors, int max_seq_len, int wtype)
 {
-    if (fast_metal_init() != 0) { fprintf(stderr, "[FastGen] CUDA init failed\n"); return NULL; }
-    InferenceState *s = calloc(1, sizeof(*s));
-    Latent *m = s ? calloc(1, sizeof(*m)) : NULL;
-    if (!m) { free(s); fast_metal_shutdown(); return NULL; }
-    s->ops = &morilorn_ops;
-    s->model = m;
-    s->mt = MODEL_MORILORN;
-    s->wtype = wtype;
-    s->max_seq = max_seq_len;
-    llmb200_engine_tp(&s->tp_rank, &s->tp_size);
-    if (s->tp_size != 1) { fprintf(stderr, "[FastGen] this model type runs on one GPU\n"); s->tp_rank = 0; s->tp_size = 1; goto fail; }
+    Latent *m = calloc(1, sizeof(*m));
+    InferenceState *s = m ? llmb200_dir_state(&morilorn_ops, MODEL_MORILORN, m, max_seq_len, wtype) : NULL;
+    if (!s) return NULL;
     if (parse(s, m, config) != 0) goto fail;
     m->es = wtype == B200_WT_F32 ? 4 : 2;
-    m->Dp = up8(s->D);
+    m->Dp = llmb200_up8(s->D);
     s->V_l = s->V;
-    if (cudaDeviceGetAttribute(&s->n_sm, cudaDevAttrMultiProcessorCount, g_rt.device) != cudaSuccess || s->n_sm <= 0) goto fail;
 
     int proj = 0, qlat = 0, part = 0, attn = 0, act = 8;
     for (int i = 0; i < s->L; ++i) {
         if (load_layer(s, m, i, tensors) != 0) { fprintf(stderr, "[FastGen] loading layer %d failed\n", i); goto fail; }
         const LLayer *y = &m->layers[i];
         proj = imax(proj, y->in.rows);
-        qlat = imax(qlat, y->heads * (up8(y->kv_rank) + up8(y->rot_dim)));
-        part = imax(part, y->heads * y->n_split * (up8(y->kv_rank) + 8));
+        qlat = imax(qlat, y->heads * (llmb200_up8(y->kv_rank) + llmb200_up8(y->rot_dim)));
+        part = imax(part, y->heads * y->n_split * (llmb200_up8(y->kv_rank) + 8));
         attn = imax(attn, y->o.cols);
         act = imax(act, y->ffp);
     }
-    Source src = { tensors, -1, 0 };
-    if (new_mat(s, &m->head, s->V, s->D) != 0) goto fail;
-    load_rows(s, &src, &m->head, "head", s->V, s->D, 0, 1);
+    TensorSource src = { tensors, -1, 0 };
+    if (llmb200_new_mat(s, &m->head, s->V, s->D) != 0) goto fail;
+    llmb200_load_rows(s, &src, &m->head, "head", s->V, s->D, 0, 1);
     s->weight_bytes += (unsigned long long)m->head.stride * s->V;
-    s->g_final = load_vec(&src, "final.norm", s->D, m->Dp);
-    float *emb = tensor(&src, "embed", s->V, s->D);
-    s->emb = llmb200_dev_zero((size_t)s->V * m->Dp * 4);
-    if (!emb || !s->emb || llmb200_upload_packed(B200_WT_F32, emb, s->D, s->V, 0, s->D, s->emb, (long long)m->Dp * 4, 0, 1) != 0) src.failed = 1;
-    free(emb);
+    s->g_final = llmb200_load_vec(&src, "final.norm", s->D, m->Dp);
+    s->emb = llmb200_load_table(&src, "embed", s->V, s->D, m->Dp);
     if (src.failed) goto fail;
 
     m->proj = llmb200_dev_zero((size_t)proj * 4); m->qlat = llmb200_dev_zero((size_t)qlat * 4);
@@ -319,9 +253,9 @@ static void free_model(InferenceState *s)
     }
     for (int i = 0; i < m->n_rope; ++i) cudaFree(m->rope_tab[i]);
     void *b[] = { m->head.w, m->proj, m->qlat, m->part, m->attn, m->z, m->u, m->rg2, m->act, m->hist, m->mix, m->x, m->r_proj, m->r_hist,
-                  m->r_x, m->r_u, m->r_y, m->r_gu, m->r_logits, m->r_xh, m->r_q, m->r_kv, m->r_attn, m->r_act, m->r_last, m->d_want };
+                  m->r_x, m->r_u, m->r_y, m->r_gu, m->r_xh, m->r_q, m->r_kv, m->r_attn, m->r_act };
     for (size_t k = 0; k < sizeof(b) / sizeof(b[0]); ++k) cudaFree(b[k]);
-    if (m->h_want) cudaFreeHost(m->h_want);
+    llmb200_row_path_free(&m->rows);
     free(m->layers);
     free(m->rope_tab);
     free(m);
@@ -451,8 +385,8 @@ static int enqueue_token(InferenceState *s, int with_lm, int pdl)
 
 static int rows_ready(InferenceState *s, Latent *m)
 {
-    if (m->chunk) return 0;
-    const int M = s->max_seq < ROW_CHUNK ? s->max_seq : ROW_CHUNK, Dp = m->Dp, es = m->es;
+    if (m->rows.chunk) return 0;
+    const int M = llmb200_row_chunk(s), Dp = m->Dp, es = m->es;
     size_t proj = 0, q = 0, kv = 0, attn = 0, gu = 0, act = 0;
     for (int i = 0; i < s->L; ++i) {
         const LLayer *y = &m->layers[i];
@@ -460,51 +394,28 @@ static int rows_ready(InferenceState *s, Latent *m)
         long long span = y->window > 0 ? (long long)M + y->window - 1 : s->max_seq;
         if (span > s->max_seq) span = s->max_seq;
         MAXI(proj, y->in.rows);
-        MAXI(q, y->heads * (up8(y->dim) + up8(y->rot_dim)));
+        MAXI(q, y->heads * (llmb200_up8(y->dim) + llmb200_up8(y->rot_dim)));
         MAXI(kv, span * y->kv.rows);
         MAXI(attn, y->o.cols);
         if (y->ff) { MAXI(gu, y->gu.rows); MAXI(act, y->ffp); }
 #undef MAXI
     }
-    const size_t wc = s->max_seq < WANT_CHUNK ? s->max_seq : WANT_CHUNK;
     m->r_proj = llmb200_dev_zero(M * proj * 4); m->r_hist = llmb200_dev_zero((size_t)(s->L + 1) * M * Dp * 4);
     m->r_x = llmb200_dev_zero((size_t)M * Dp * 4); m->r_u = llmb200_dev_zero((size_t)M * Dp * 4);
     m->r_y = llmb200_dev_zero((size_t)M * imax(64, Dp) * 4); m->r_gu = llmb200_dev_zero(M * gu * 4);
     m->r_xh = llmb200_dev_zero((size_t)M * Dp * 2); m->r_q = llmb200_dev_zero(M * q * es); m->r_kv = llmb200_dev_zero(kv * es);
     m->r_attn = llmb200_dev_zero(M * attn * es); m->r_act = llmb200_dev_zero(M * act * es);
-    m->r_last = llmb200_dev_zero(wc * Dp * es); m->r_logits = llmb200_dev_zero(wc * m->head.rows * 4);
-    m->d_want = (int *)llmb200_dev_zero(wc * 4);
-    if (!m->r_proj || !m->r_hist || !m->r_x || !m->r_u || !m->r_y || !m->r_gu || !m->r_xh || !m->r_q || !m->r_kv || !m->r_attn || !m->r_act ||
-        !m->r_last || !m->r_logits || !m->d_want)
+    if (!m->r_proj || !m->r_hist || !m->r_x || !m->r_u || !m->r_y || !m->r_gu || !m->r_xh || !m->r_q || !m->r_kv || !m->r_attn || !m->r_act)
         return -1;
-    if (!m->h_want) CU_TRY(cudaMallocHost((void **)&m->h_want, wc * 4), return -1);
-    m->chunk = M;
-    return 0;
-}
-
-/* C[M, w->rows] = A[M, K] x w^T; A has the matrices' element type, K columns (padding included) lda apart. Ch: the
- * result in that element type instead of C. */
-static int rows_product(InferenceState *s, const void *A, long long lda, const PackedMat *w, int M, float *C, long long ldc, void *Ch)
-{
-    const int f32 = s->wtype == B200_WT_F32;
-    b200_gemm_args g;
-    memset(&g, 0, sizeof(g));
-    g.A = A; g.a_row = lda; g.a_col = 1;
-    g.B = w->w; g.b_row = 1; g.b_col = w->stride / (f32 ? 4 : 2);
-    g.ldc = ldc; g.M = M; g.N = w->rows; g.K = w->cols; g.alpha = 1.0f;
-    g.d_err = (unsigned *)s->d_err;
-    if (Ch && !f32) { g.Ch = Ch; g.ldch = ldc; }
-    else g.C = Ch ? Ch : C;
-    const int rc = f32 ? b200_gemm_f32(&g, g_rt.stream) : b200_gemm_bf16(&g, g_rt.stream);
-    if (rc) fprintf(stderr, "[FastGen] row product %d x %d x %d failed: code %d\n", M, w->rows, w->cols, rc);
-    return rc;
+    return llmb200_row_path_ready(s, &m->rows, &m->head, Dp, M);
 }
 
 /* M tokens from position pos0 on, whose ids are in d_tokens; x of the last layer is left in r_x. */
-static int chunk_rows(InferenceState *s, Latent *m, int pos0, int M)
+static int chunk_rows(InferenceState *s, int pos0, int M)
 {
+    Latent *m = s->model;
     const int Dp = m->Dp, f32 = s->wtype == B200_WT_F32;
-    const size_t hs = (size_t)m->chunk * Dp;                 /* one layer's result of a chunk in r_hist */
+    const size_t hs = (size_t)m->rows.chunk * Dp;                 /* one layer's result of a chunk in r_hist */
     void *st = g_rt.stream;
     /* the operand of a product is the bfloat16 copy, or the vector itself in fp32 */
     void *xh = f32 ? NULL : m->r_xh;
@@ -513,7 +424,7 @@ static int chunk_rows(InferenceState *s, Latent *m, int pos0, int M)
         const LLayer *y = &m->layers[l];
         const float *x = l ? m->r_x : m->r_hist;
         const long long pld = y->in.rows;
-        if (rows_product(s, f32 ? (const void *)x : xh, Dp, &y->in, M, m->r_proj, pld, NULL)) return -1;
+        if (llmb200_rows_product(s, f32 ? (const void *)x : xh, Dp, &y->in, M, m->r_proj, pld, NULL, 0)) return -1;
 
         b200_latent_args at;
         latent_args(s, m, y, m->r_proj, &at);
@@ -522,11 +433,11 @@ static int chunk_rows(InferenceState *s, Latent *m, int pos0, int M)
         at.d_q_rows = m->r_q; at.d_kv = m->r_kv; at.kv_ld = y->kv.rows;
         at.d_out_rows = m->r_attn; at.out_ld = y->o.cols;
         K_TRY(b200_latent_rows_prep(&at, st), return -1);
-        const long long cs = up8(y->kv_rank) + up8(y->rot_dim);
-        if (rows_product(s, (const char *)y->cache + (size_t)at.kv_row0 * cs * m->es, cs, &y->kv, pos0 + M - at.kv_row0, NULL, y->kv.rows, m->r_kv))
+        const long long cs = llmb200_up8(y->kv_rank) + llmb200_up8(y->rot_dim);
+        if (llmb200_rows_product(s, (const char *)y->cache + (size_t)at.kv_row0 * cs * m->es, cs, &y->kv, pos0 + M - at.kv_row0, NULL, y->kv.rows, m->r_kv, 0))
             return -1;
         K_TRY(b200_latent_rows_attend(&at, st), return -1);
-        if (rows_product(s, m->r_attn, y->o.cols, &y->o, M, m->r_y, y->o.rows, NULL)) return -1;
+        if (llmb200_rows_product(s, m->r_attn, y->o.cols, &y->o, M, m->r_y, y->o.rows, NULL, 0)) return -1;
 
         b200_rows_postnorm_args pn;
         memset(&pn, 0, sizeof(pn));
@@ -537,9 +448,9 @@ static int chunk_rows(InferenceState *s, Latent *m, int pos0, int M)
         if (y->ff) {
             pn.norm_out = m->r_u; pn.out = m->r_u;
             K_TRY(b200_rows_postnorm(&pn, st), return -1);
-            if (rows_product(s, f32 ? (const void *)m->r_u : xh, Dp, &y->gu, M, m->r_gu, y->gu.rows, NULL)) return -1;
+            if (llmb200_rows_product(s, f32 ? (const void *)m->r_u : xh, Dp, &y->gu, M, m->r_gu, y->gu.rows, NULL, 0)) return -1;
             K_TRY(b200_rows_gelu_mul(m->r_gu, y->gu.rows, M, y->ffp, s->wtype, m->r_act, st), return -1);
-            if (rows_product(s, m->r_act, y->ffp, &y->down, M, m->r_y, y->down.rows, NULL)) return -1;
+            if (llmb200_rows_product(s, m->r_act, y->ffp, &y->down, M, m->r_y, y->down.rows, NULL, 0)) return -1;
             pn.y_ld = y->down.rows;
             pn.x = m->r_u; pn.gate = m->r_gu + 2 * y->ffp; pn.gate_ld = y->gu.rows; pn.gate_bias = y->b2; pn.gamma = y->norm2;
         }
@@ -551,29 +462,16 @@ static int chunk_rows(InferenceState *s, Latent *m, int pos0, int M)
     return 0;
 }
 
+static int last_rows(InferenceState *s, const int *index, int n, void *out)
+{
+    const Latent *m = s->model;
+    K_TRY(b200_rows_norm(m->r_x, index, n, s->D, m->Dp, m->groups, m->eps, s->g_final, s->wtype, out, g_rt.stream), return -1);
+    return 0;
+}
+
 static int forward_rows(InferenceState *s, const uint32_t *tokens, int n, const int *want, int n_want, float *logits)
 {
     Latent *m = s->model;
     if (rows_ready(s, m) != 0) { fprintf(stderr, "[FastGen] no memory for the row path\n"); return -1; }
-    int w = 0;
-    const size_t wc = s->max_seq < WANT_CHUNK ? s->max_seq : WANT_CHUNK;
-    for (int c0 = 0; c0 < n; c0 += m->chunk) {
-        const int M = n - c0 < m->chunk ? n - c0 : m->chunk, pos0 = s->cur_len + c0;
-        if (llmb200_set_control(s, pos0, s->max_seq + 2, tokens + c0, pos0, M) != 0) return -1;
-        if (chunk_rows(s, m, pos0, M) != 0) return -1;
-        while (w < n_want && want[w] < c0 + M) {
-            int k = 0;
-            CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1);           /* h_want may still be in flight */
-            while (k < (int)wc && w + k < n_want && want[w + k] < c0 + M) { m->h_want[k] = want[w + k] - c0; ++k; }
-            CU_TRY(cudaMemcpyAsync(m->d_want, m->h_want, (size_t)k * 4, cudaMemcpyHostToDevice, g_rt.stream), return -1);
-            K_TRY(b200_rows_norm(m->r_x, m->d_want, k, s->D, m->Dp, m->groups, m->eps, s->g_final, s->wtype, m->r_last, g_rt.stream), return -1);
-            if (rows_product(s, m->r_last, m->Dp, &m->head, k, m->r_logits, m->head.rows, NULL)) return -1;
-            if (m->softcap > 0.0f) K_TRY(b200_rows_softcap(m->r_logits, k, s->V, m->head.rows, m->softcap, g_rt.stream), return -1);
-            CU_TRY(cudaMemcpy2DAsync(logits + (size_t)w * s->V, (size_t)s->V * 4, m->r_logits, (size_t)m->head.rows * 4, (size_t)s->V * 4, (size_t)k,
-                                     cudaMemcpyDeviceToHost, g_rt.stream), return -1);
-            w += k;
-        }
-    }
-    CU_TRY(cudaStreamSynchronize(g_rt.stream), return -1);
-    return 0;
+    return llmb200_row_path_run(s, &m->rows, chunk_rows, last_rows, m->softcap, tokens, n, want, n_want, logits);
 }

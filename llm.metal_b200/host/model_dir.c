@@ -13,6 +13,7 @@ static const struct {
     InferenceState *(*create)(const json *config, const llmb200_tensor_file *tensors, int max_seq_len, int wtype);
 } registry[] = {
     { "Morilorn", llmb200_create_morilorn },
+    { "Zidepel", llmb200_create_zidepel },
 };
 
 InferenceState *inference_state_create_from_dir(const char *dir, int max_seq_len, int wtype)

@@ -104,3 +104,12 @@ float *llmb200_tensor_f32(const llmb200_tensor_file *f, const char *name, long l
         for (size_t i = 0; i < n; ++i) out[i] = half_to_f32((uint16_t)(src[2 * i] | src[2 * i + 1] << 8));
     return out;
 }
+
+long long llmb200_tensor_dim(const llmb200_tensor_file *f, const char *name, int axis)
+{
+    const json *shape = json_get(json_get(f->header, name), "shape");
+    if (!shape || shape->type != JSON_ARRAY || axis < 0 || axis >= shape->n) return -1;
+    const json *d = shape->child;
+    while (axis-- > 0) d = d->next;
+    return d->type == JSON_NUMBER && d->number >= 0 && d->number < 9e15 ? (long long)d->number : -1;
+}
