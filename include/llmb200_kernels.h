@@ -349,7 +349,7 @@ typedef struct b200_gla_args {
     int n_rows, pos0;
     long long proj_ld;
     float *d_qd, *d_kd;                  /* [n_chunks * 64][heads][up8(dim)]: queries and keys times their decays */
-    float *d_decay;                      /* [n_chunks][heads][up8(dim)]: decay over a whole chunk */
+    float *d_decay;                      /* [n_chunks][heads][up8(dim)]: logarithm of the decay over a whole chunk */
     float *d_scores;                     /* [n_chunks][heads][64][64] */
     float *d_chunk_state;                /* [n_chunks][heads][dim][up8(vdim)] */
     float *d_o;                          /* [n_rows][heads * vdim]; vdim > 128 only */

@@ -34,6 +34,17 @@ __host__ __device__ __forceinline__ int up8(int n) { return (n + 7) & ~7; }
 __device__ __forceinline__ float log_logistic(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float silu_f32(float z) { return z * sigmoid_f32(z); }
 
+// A decay factor exp(x), x <= 0, as the pair (m, keep) for S <- keep S + (m S + u). Near one the factor's own rounding,
+// the same for every token of a slow channel, would add up over hundreds of tokens, so there m = exp(x) - 1 and keep = 1;
+// elsewhere m = exp(x) and keep = 0.
+struct Decay { float m, keep; };
+__device__ __forceinline__ Decay decay_of(float x)
+{
+    const float m = expm1f(x);
+    return m > -0.5f ? Decay{m, 1.0f} : Decay{expf(x), 0.0f};
+}
+__device__ __forceinline__ float decayed(float s, const Decay &a, float u) { return fmaf(a.keep, s, fmaf(a.m, s, u)); }
+
 __device__ __forceinline__ float dot4(const float4 &a, const float4 &b, float acc)
 {
     return fmaf(a.w, b.w, fmaf(a.z, b.z, fmaf(a.y, b.y, fmaf(a.x, b.x, acc))));
@@ -58,7 +69,8 @@ __global__ void __launch_bounds__(THREADS) gla_decode_kernel(const __grid_consta
     const int h = blockIdx.x / cluster_size, rank = blockIdx.x % cluster_size;
     const int dim = p.dim, v8 = up8(p.vdim), R4 = up4(p.rank), w16 = (R4 / 4) | 1;      // odd: rows 16 bytes apart mod 32
     const int VW = 4 * vg, c0 = rank * VW, RG = THREADS / vg, rg = tid / vg, col = c0 + 4 * (tid % vg);
-    float *sa = sh, *sk = sa + up4(dim), *sq = sk + up4(dim), *so = sq + up4(dim), *w2 = so + (THREADS / 32) * VW;
+    Decay *sa = reinterpret_cast<Decay *>(sh);
+    float *sk = sh + 2 * up4(dim), *sq = sk + up4(dim), *so = sq + up4(dim), *w2 = so + (THREADS / 32) * VW;
     const int pos = *p.d_pos;
     const size_t slot = (size_t)p.heads * dim * v8;
     const float *s_in = p.d_state + (size_t)(max(pos, 0) % p.n_slots) * slot + (size_t)h * dim * v8;
@@ -96,15 +108,16 @@ __global__ void __launch_bounds__(THREADS) gla_decode_kernel(const __grid_consta
         float z = d == tid ? bias0 : p.d_a2_bias[h * dim + d];
         for (int c = 0; c < R4 / 4; ++c)
             z = dot4(*reinterpret_cast<const float4 *>(w2 + ((size_t)d * w16 + c) * 4), *reinterpret_cast<const float4 *>(p.d_f + 4 * c), z);
-        sa[d] = expf(log_logistic(z) / p.tau);
+        sa[d] = decay_of(log_logistic(z) / p.tau);
         sk[d] = k;
         sq[d] = q * p.q_scale;
     }
     __syncthreads();
     float4 o = zero;
     auto step = [&](float4 s, int d) {
-        const float a = sa[d], k = sk[d], q = sq[d];
-        s.x = fmaf(a, s.x, k * v.x); s.y = fmaf(a, s.y, k * v.y); s.z = fmaf(a, s.z, k * v.z); s.w = fmaf(a, s.w, k * v.w);
+        const Decay a = sa[d];
+        const float k = sk[d], q = sq[d];
+        s.x = decayed(s.x, a, k * v.x); s.y = decayed(s.y, a, k * v.y); s.z = decayed(s.z, a, k * v.z); s.w = decayed(s.w, a, k * v.w);
         *reinterpret_cast<float4 *>(s_out + (size_t)d * v8 + col) = s;
         o.x = fmaf(q, s.x, o.x); o.y = fmaf(q, s.y, o.y); o.z = fmaf(q, s.z, o.z); o.w = fmaf(q, s.w, o.w);
     };
@@ -218,7 +231,7 @@ __global__ void __launch_bounds__(THREADS) gla_prep_kernel(const __grid_constant
                 p.d_kd[at] = k[i] * expf(end - c[i]);
             }
         }
-        if (tg == 0 && d0 + d < d8) p.d_decay[((size_t)chunk * p.heads + h) * d8 + d0 + d] = expf(end);
+        if (tg == 0 && d0 + d < d8) p.d_decay[((size_t)chunk * p.heads + h) * d8 + d0 + d] = end;
         __syncthreads();
         // references: c just before each sixteen
 #pragma unroll
@@ -327,18 +340,18 @@ __global__ void __launch_bounds__(THREADS) gla_scan_kernel(const __grid_constant
     if (p.pos0 > 0) s = *reinterpret_cast<const float4 *>(p.d_state + (size_t)(p.pos0 % p.n_slots) * per + e * 4);
     for (int c0 = 0; c0 < n_chunks; c0 += AHEAD) {
         float4 u[AHEAD];
-        float g[AHEAD];
+        Decay g[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
             if (c0 + i < n_chunks) {
                 u[i] = *reinterpret_cast<const float4 *>(p.d_chunk_state + (size_t)(c0 + i) * per + e * 4);
-                g[i] = p.d_decay[(size_t)(c0 + i) * p.heads * d8 + ch];
+                g[i] = decay_of(p.d_decay[(size_t)(c0 + i) * p.heads * d8 + ch]);
             }
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
             if (c0 + i < n_chunks) {
                 *reinterpret_cast<float4 *>(p.d_chunk_state + (size_t)(c0 + i) * per + e * 4) = s;
-                s.x = fmaf(g[i], s.x, u[i].x); s.y = fmaf(g[i], s.y, u[i].y); s.z = fmaf(g[i], s.z, u[i].z); s.w = fmaf(g[i], s.w, u[i].w);
+                s.x = decayed(s.x, g[i], u[i].x); s.y = decayed(s.y, g[i], u[i].y); s.z = decayed(s.z, g[i], u[i].z); s.w = decayed(s.w, g[i], u[i].w);
             }
     }
     *reinterpret_cast<float4 *>(p.d_state + (size_t)((p.pos0 + p.n_rows) % p.n_slots) * per + e * 4) = s;
@@ -476,7 +489,7 @@ extern "C" int b200_gla_decode(const b200_gla_args *a, void *stream)
     while (vg < (quads + cl - 1) / cl) vg <<= 1;
     if (vg > 32) return B200_E_TOOLARGE;
     const int R4 = up4(a->rank);
-    const size_t smem = ((size_t)3 * up4(a->dim) + THREADS / 32 * 4 * vg + (size_t)a->dim * ((R4 / 4) | 1) * 4) * 4;
+    const size_t smem = ((size_t)4 * up4(a->dim) + THREADS / 32 * 4 * vg + (size_t)a->dim * ((R4 / 4) | 1) * 4) * 4;
     const int rc = allow_smem(gla_decode_kernel, smem);
     if (rc) return rc;
     cudaLaunchConfig_t cfg = {};

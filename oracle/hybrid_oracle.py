@@ -134,3 +134,82 @@ def forward(config, weights, tokens):
                               lambda h: feed_forward(h, sub(w, p + "mlp.")))
         after.append(streams.sum(axis=0))
     return layer_norm(streams.sum(axis=0), w["final.norm"], w["final.norm.b"], eps) @ w["head"].T, after
+
+
+# ------------------------------------------------------------------ models
+
+def attention_layer(heads, kv_heads, dim, vdim, ff, scale=None, cap=25.0, temp=(0.3, 64)):
+    mix = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale or dim ** -0.5, "softcap": cap,
+           "q_temp": {"coef": temp[0], "every": temp[1]} if temp else None}
+    return {"type": "attention", "mixer": mix, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def gla_layer(heads, dim, vdim, ff, tau, rank):
+    """`rank` is no key of a configuration: it is the shape of a tensor (tensor_shapes reads it)."""
+    return {"type": "gla", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}, "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "_rank": rank}
+
+
+def model_config(width, vocab, streams, layers, loop=None, eps=1e-5, max_positions=512):
+    """-> config.json's content and the ranks of the layers' decays."""
+    ranks = [layer.get("_rank") for layer in layers]
+    clean = [{k: v for k, v in layer.items() if k != "_rank"} for layer in layers]
+    return {"architecture": "Zidepel", "vocab": vocab, "width": width, "streams": streams, "max_positions": max_positions, "norm": {"eps": eps},
+            "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None, "layers": clean}, ranks
+
+
+def tensor_shapes(config, ranks):
+    D, V, n = config["width"], config["vocab"], config["streams"]
+    s = {"embed": (V, D), "pos": (config["max_positions"], D), "head": (V, D)}
+    for name in ("embed.norm", "final.norm"):
+        s.update({name: (D,), name + ".b": (D,)})
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}."
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        for q in range(1, 3 if layer["mlp"] else 2):
+            s.update({f"{p}norm{q}": (D,), f"{p}norm{q}.b": (D,), f"{p}hc{q}.in": (n,), f"{p}hc{q}.out": (n,), f"{p}hc{q}.mix": (n, n)})
+        s.update({p + "mix.q": (H * d, D), p + "mix.o": (D, H * dv)})
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            s.update({p + "mix.k": (G * d, D), p + "mix.v": (G * dv, D), p + "mix.q.norm": (d,), p + "mix.k.norm": (d,)})
+        else:
+            r = ranks[i]
+            s.update({p + "mix.k": (H * d, D), p + "mix.v": (H * dv, D), p + "mix.g": (H * dv, D), p + "mix.norm": (dv,), p + "mix.a1": (r, D),
+                      p + "mix.a2": (H * d, r), p + "mix.a2.b": (H * d,)})
+        if layer["mlp"]:
+            F = layer["mlp"]["ff"]
+            s.update({p + "mlp.up": (F, D), p + "mlp.down": (D, F)})
+    return s
+
+
+def random_model(config, ranks, seed, sharp=1.2):
+    """Weights that keep every part in play: scores of spread about sharp^2, decays from a token to hundreds, stream
+    connections away from their trivial values. The recurrences' keys lean towards their queries, so that a head's result
+    is not a difference of nearly equal numbers before its norm. All are bfloat16 values."""
+    rng = np.random.default_rng(seed)
+    n, w = config["streams"], {}
+    for name, shape in tensor_shapes(config, ranks).items():
+        leaf = name.split(".", 1)[1] if name[0] == "l" else name
+        z = rng.standard_normal(shape)
+        if leaf.endswith(".in"):
+            v = 1.0 / n + 0.1 * z
+        elif leaf.endswith(".out"):
+            v = 1.0 + 0.3 * z
+        elif leaf.startswith("hc"):
+            v = 0.8 * np.eye(n) + 0.2 * n ** -0.5 * z
+        elif leaf == "mix.a2.b":
+            v = 2.0 + 2.0 * z
+        elif leaf.endswith(".b"):
+            v = 0.2 * z
+        elif leaf in ("mix.q.norm", "mix.k.norm"):
+            v = sharp * (1.0 + 0.3 * z)
+        elif len(shape) == 1:
+            v = 1.0 + 0.2 * z
+        elif leaf in ("embed", "pos"):
+            v = 0.5 * z
+        else:
+            v = z * shape[1] ** -0.5 * (2.0 if leaf == "head" else 1.0)
+            if leaf == "mix.k" and config["layers"][int(name[1:name.index(".")])]["type"] == "gla":
+                v = 0.7 * w[name[:-1] + "q"] + 0.7 * v
+        w[name] = bf16(v)
+    return w
