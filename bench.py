@@ -35,9 +35,11 @@ import argparse
 import ctypes as C
 import json
 import os
+import shutil
 import statistics
 import subprocess
 import sys
+import tempfile
 import threading
 import time
 
@@ -438,6 +440,204 @@ def batch_main(args, rank, local_rank, world):
     return 0
 
 
+HYBRID_WORKLOADS = {
+    # name: sizes, each beside a Morilorn model of the same width, layer runs, heads, feed-forward and vocabulary; prompt portion,
+    # generated tokens. A group is one linear-attention layer and three attention layers; the first group runs twice.
+    "zidepel": ([dict(width=2048, groups=2, heads=16, kv_heads=4, dim=128, vdim=128, gla_dim=64, rank=16, ff=6144, vocab=32768, streams=4),
+                 dict(width=2560, groups=2, heads=32, kv_heads=8, dim=128, vdim=128, gla_dim=64, rank=16, ff=9728, vocab=65536, streams=4),
+                 dict(width=4096, groups=1, heads=32, kv_heads=8, dim=128, vdim=128, gla_dim=128, rank=16, ff=12288, vocab=65536, streams=2)], 2048, 256),
+    "tiny-zidepel": ([dict(width=256, groups=1, heads=4, kv_heads=1, dim=48, vdim=64, gla_dim=24, rank=8, ff=512, vocab=1024, streams=2)], 128, 32),
+}
+
+
+def write_hybrid_model(folder, z, seed, pattern=None, loop=True, vocab=None):
+    """A Zidepel model folder of the sizes z; pattern: the layers' kinds ("a", "r"), by default groups of r a a a with the first one
+    looped twice."""
+    D, V, F, H, G, n = z["width"], vocab or z["vocab"], z["ff"], z["heads"], z["kv_heads"], z["streams"]
+    pattern = pattern or "raaa" * z["groups"]
+    attn = {"type": "attention", "mlp": {"kind": "dense", "ff": F},
+            "mixer": {"heads": H, "kv_heads": G, "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "softcap": 40.0,
+                      "q_temp": {"coef": 0.1, "every": 1000}}}
+    rec = {"type": "gla", "mlp": {"kind": "dense", "ff": F}, "mixer": {"heads": H, "dim": z["gla_dim"], "vdim": z["vdim"], "tau": 16.0}}
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump({"architecture": "Zidepel", "vocab": V, "width": D, "streams": n, "max_positions": 4096, "norm": {"eps": 1e-6},
+                   "loop": {"start": 0, "stop": 4, "times": 2} if loop else None, "layers": [attn if c == "a" else rec for c in pattern]}, f)
+    shapes = {"embed": (V, D), "pos": (4096, D), "head": (V, D)}
+    for k in ("embed.norm", "final.norm"):
+        shapes.update({k: (D,), k + ".b": (D,)})
+    for i, c in enumerate(pattern):
+        d, p = z["dim"] if c == "a" else z["gla_dim"], f"l{i}."
+        for q in (1, 2):
+            shapes.update({f"{p}norm{q}": (D,), f"{p}norm{q}.b": (D,), f"{p}hc{q}.in": (n,), f"{p}hc{q}.out": (n,), f"{p}hc{q}.mix": (n, n)})
+        shapes.update({p + "mix.q": (H * d, D), p + "mix.o": (D, H * z["vdim"]), p + "mlp.up": (F, D), p + "mlp.down": (D, F)})
+        if c == "a":
+            shapes.update({p + "mix.k": (G * d, D), p + "mix.v": (G * z["vdim"], D), p + "mix.q.norm": (d,), p + "mix.k.norm": (d,)})
+        else:
+            shapes.update({p + "mix.k": (H * d, D), p + "mix.v": (H * z["vdim"], D), p + "mix.g": (H * z["vdim"], D), p + "mix.norm": (z["vdim"],),
+                           p + "mix.a1": (z["rank"], D), p + "mix.a2": (H * d, z["rank"]), p + "mix.a2.b": (H * d,)})
+
+    def special(k):
+        return "identity" if k.endswith(".mix") else "zeros" if k.endswith(".b") else "ones" if "norm" in k or ".hc" in k else None
+    return write_random_tensors(folder, shapes, seed, special)
+
+
+def hybrid_kernel_bytes(z, kind, P):
+    """Bytes that one layer's decode kernels have to move at position P (streams of the o / down products included)."""
+    D, H, G, n, hv = z["width"], z["heads"], z["kv_heads"], z["streams"], z["heads"] * z["vdim"]
+    join = 4 * (2 * n + 1) * D
+    if kind == "a":
+        rows, mixer = (H + G) * z["dim"] + G * z["vdim"], 2 * P * G * (z["dim"] + z["vdim"])
+    else:
+        rows, mixer = 2 * H * z["gla_dim"] + 2 * hv + z["rank"], 4 * H * z["gla_dim"] * (2 * z["vdim"] + z["rank"])
+    return {"in": 2 * rows * D, "attention": mixer, "o": 2 * D * hv + join, "gateup": 2 * z["ff"] * D, "down": 2 * D * z["ff"] + join,
+            "lm_head": 2 * z["vocab"] * D}
+
+
+def hybrid_kernel_timings(pkg, L, torch, z, M, peaks):
+    """Prompt-portion kernels alone at these sizes: the attention of one layer, the linear attention of one layer (all its launches),
+    the stream update; beside the row norm of the closest model (its attention: latent_kernel_timings)."""
+    up8 = lambda v: (v + 7) // 8 * 8
+    D, H, G, d, dv, n = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["streams"]
+    hbm, tc = peaks
+    st, out, keep = torch.cuda.current_stream().cuda_stream, {}, []
+
+    def buf(*shape, dt=torch.float32):
+        keep.append(torch.randn(*shape, device="cuda").to(dt))
+        return keep[-1].data_ptr()
+
+    def run(name, fn, arg, flops=0.0, nbytes=0.0):
+        def call():
+            if fn(C.byref(arg), st) != 0:
+                raise RuntimeError(name)
+        ms = timed_flushed(torch, call)
+        out[name] = {"us": 1e3 * ms}
+        if flops:
+            out[name].update(tflops=flops / ms / 1e9, frac_of_tensor_peak=flops / ms / 1e9 / tc)
+        if nbytes:
+            out[name].update(bytes=nbytes, gbs=nbytes / ms / 1e6, frac_of_hbm=nbytes / ms / 1e6 / hbm)
+
+    a = pkg.GqaArgs()
+    ld = (H + G) * d + G * dv
+    a.wtype, a.heads, a.kv_heads, a.dim, a.vdim, a.max_seq, a.scale, a.softcap, a.eps = 2, H, G, d, dv, M, d ** -0.5, 40.0, 1e-6
+    a.d_q = buf(M, ld)
+    a.d_k, a.d_v, a.proj_ld = a.d_q + 4 * H * d, a.d_q + 4 * (H + G) * d, ld
+    a.d_q_gamma, a.d_k_gamma, a.d_q_scale = buf(d), buf(d), buf(M)
+    a.d_k_cache, a.d_v_cache = buf(G, M, up8(d), dt=torch.bfloat16), buf(G, M, up8(dv), dt=torch.bfloat16)
+    a.d_q_rows, a.d_out_rows, a.out_ld, a.n_rows = buf(M, H, up8(d), dt=torch.bfloat16), buf(M, H * dv, dt=torch.bfloat16), H * dv, M
+    run("attention_rows_prep", L.b200_gqa_rows_prep, a, nbytes=M * (4.0 * ld + 2.0 * ld))
+    run("attention_rows", L.b200_gqa_rows_attend, a, flops=2.0 * (M * (M + 1) / 2) * H * (d + dv))
+    a.softcap = 0.0
+    run("attention_rows_without_cap", L.b200_gqa_rows_attend, a, flops=2.0 * (M * (M + 1) / 2) * H * (d + dv))
+    g, d, nc, r4 = pkg.GlaArgs(), z["gla_dim"], (M + 63) // 64, (z["rank"] + 3) // 4 * 4
+    ld = 2 * H * d + 2 * H * dv + z["rank"]
+    g.wtype, g.heads, g.dim, g.vdim, g.rank, g.n_slots, g.tau, g.q_scale, g.eps = 2, H, d, dv, z["rank"], 2, 16.0, d ** -0.5, 1e-6
+    g.d_q = buf(M, ld)
+    g.proj_ld = ld
+    g.d_k, g.d_v, g.d_gate, g.d_f = (g.d_q + 4 * o for o in (H * d, 2 * H * d, 2 * H * d + H * dv, 2 * H * d + 2 * H * dv))
+    g.d_a2, g.d_a2_bias, g.d_norm_gamma, g.d_state = buf(H * d, r4), buf(H * d), buf(dv), buf(2, H, d, up8(dv))
+    g.d_qd, g.d_kd, g.d_decay, g.d_scores = buf(nc * 64, H, up8(d)), buf(nc * 64, H, up8(d)), buf(nc, H, up8(d)), buf(nc, H, 64, 64)
+    g.d_chunk_state, g.d_o, g.d_out_rows, g.out_ld, g.n_rows = buf(nc, H, d, up8(dv)), buf(M, H * dv), buf(M, H * dv, dt=torch.bfloat16), H * dv, M
+    run("linear_attention_rows", L.b200_gla_rows, g, nbytes=M * (4.0 * ld + 2.0 * H * dv))
+    s = pkg.RowsStreamsArgs()
+    s.streams_in, s.streams_in_stride, s.y, s.y_ld, s.connect, s.n_streams = buf(n, M, D), M * D, buf(M, D), D, buf(n * (n + 2)), n
+    s.gamma, s.beta, s.eps, s.rows, s.dim, s.ld, s.wtype, s.streams_out, s.streams_out_stride, s.out = (
+        buf(D), buf(D), 1e-6, M, D, D, 2, buf(n, M, D), M * D, buf(M, D, dt=torch.bfloat16))
+    run("rows_streams", L.b200_rows_streams, s, nbytes=M * D * (4.0 * (2 * n + 1) + 2.0))
+    p = pkg.RowsPostnormArgs()
+    p.x, p.y, p.y_ld, p.gate, p.gate_ld, p.gate_bias, p.gamma = buf(M, D), buf(M, D), D, buf(M, D), D, buf(D), buf(D)
+    p.alpha, p.eps, p.rows, p.dim, p.ld, p.groups, p.norm_out, p.out, p.out_h = 1.5, 1e-6, M, D, D, 4, buf(M, D), None, buf(M, D, dt=torch.bfloat16)
+    p.out = p.norm_out
+    run("rows_postnorm_closest_model", L.b200_rows_postnorm, p, nbytes=M * D * (4.0 * 4 + 2.0))
+    u = pkg.GemmArgs()
+    u.A, u.a_row, u.a_col, u.B, u.b_row, u.b_col = buf(M, D, dt=torch.bfloat16), D, 1, buf(z["ff"], D, dt=torch.bfloat16), 1, D
+    u.Ch, u.ldch, u.M, u.N, u.K, u.alpha, u.relu2 = buf(M, z["ff"], dt=torch.bfloat16), z["ff"], M, z["ff"], D, 1.0, 1
+    run("up_product_squared_relu", L.b200_gemm_bf16, u, flops=2.0 * M * z["ff"] * D)
+    return out
+
+
+def hybrid_main(args, rank, local_rank, world):
+    """Zidepel: prompt portions and decode at several sizes, each beside a Morilorn model of equal width, layer runs, heads,
+    feed-forward and vocabulary. The line's value is the first size's decode rate."""
+    if args.impl == "reference" or world > 1:
+        if rank == 0:
+            emit(json.dumps({"impl": args.impl, "unavailable": "the reference has no such model; the workload runs on one GPU"}))
+        return 0
+    import torch
+    torch.cuda.set_device(local_rank)
+    sizes, P, G = HYBRID_WORKLOADS[args.workload]
+    P, G = args.prompt_len or P, args.gen_len or G
+    pkg = entry.load_package()
+    L, S = pkg.lib(), pkg.synth()
+    peak, peak_kind = measured_peaks()
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tc = float(json.load(f)["bf16_tflops"])
+    except Exception:
+        tc = 1590.0
+    rows, launches = [], 0
+    sampler = ClockSampler(local_rank)
+    for zi, z in enumerate(sizes):
+        z = dict(z, groups=args.layers or z["groups"])
+        m = open_folder_model(pkg, lambda folder: write_hybrid_model(folder, z, 7 + zi), P + G + 8)
+        if zi == 0:
+            sampler.start()
+        r = measure_folder_model(pkg, L, S, m, P, G, args.warmup, args.steps)
+        launches += r["launches"]
+        if L.llmb200_state_error(m.state):
+            raise RuntimeError("a device-side wait timed out")
+        m.close()
+        n_rec, n_att = z["groups"] + 1, 3 * (z["groups"] + 1)         # runs: the first group counts twice
+        kb = {c: hybrid_kernel_bytes(z, c, P + G // 2) for c in "ar"}
+        token_bytes = kb["a"]["lm_head"] + sum(cnt * sum(b for k, b in kb[c].items() if k != "lm_head") for c, cnt in (("r", n_rec), ("a", n_att)))
+        us, pf = r["decode_us"], r["prefill_ms"]
+        in_rows = {"a": (z["heads"] + z["kv_heads"]) * z["dim"] + z["kv_heads"] * z["vdim"],
+                   "r": 2 * z["heads"] * (z["gla_dim"] + z["vdim"]) + z["rank"]}
+        flops = 2.0 * P * z["width"] * sum(cnt * (in_rows[c] + z["heads"] * z["vdim"] + 2 * z["ff"]) for c, cnt in (("r", n_rec), ("a", n_att)))
+        res = {"sizes": z, "runs": {"linear_attention": n_rec, "attention": n_att},
+               "decode": {"tokens_per_s": 1e6 / us, "us_per_token": us, "bytes_per_token": token_bytes, "frac_of_hbm": token_bytes / us / 1e3 / peak,
+                          "launches_per_token": r["graph"]},
+               "decode_e2e_tokens_per_s": r["e2e_tokens_per_s"],
+               "prefill": {"tokens": P, "ms": pf, "tokens_per_s": P / pf * 1e3, "product_tflops": flops / pf / 1e9,
+                           "frac_of_tensor_peak": flops / pf / 1e9 / tc}}
+        # decode kernels alone: models of one kind of layer
+        for c, name in (("a", "attention_layers"), ("r", "linear_attention_layers")):
+            m = open_folder_model(pkg, lambda folder: write_hybrid_model(folder, z, 17 + zi, c * 6, False), P + G + 8)
+            res["decode"][name] = time_folder_kinds(L, m, r["prompt"], hybrid_kernel_bytes(z, c, P), peak)
+            m.close()
+        res["kernels_alone"] = hybrid_kernel_timings(pkg, L, torch, z, P, (peak, tc))
+        # the closest model at equal size
+        near = dict(width=z["width"], layers=n_rec + n_att, heads=z["heads"], dim=z["dim"], rot_dim=64 if z["dim"] >= 64 else 16, vdim=z["vdim"],
+                    kv_rank=4 * z["dim"], ff=z["ff"], vocab=z["vocab"], window=P + G)
+        m = open_folder_model(pkg, lambda folder: write_latent_model(folder, near, 27 + zi), P + G + 8)
+        q = measure_folder_model(pkg, L, S, m, P, G, args.warmup, args.steps)
+        qk = latent_kernel_bytes(near, P)
+        qb = sum(b * (near["layers"] if k != "lm_head" else 1) for k, b in qk.items())
+        kinds = time_folder_kinds(L, m, q["prompt"], qk, peak, lambda k: 3 if k == "attention" else 1)
+        m.close()
+        alone = latent_kernel_timings(pkg, L, torch, near, P, (peak, tc))
+        res["closest_model"] = {"what": "Morilorn, same width / layer runs / heads / feed-forward / vocabulary", "sizes": near,
+                                "decode": {"tokens_per_s": 1e6 / q["decode_us"], "us_per_token": q["decode_us"], "bytes_per_token": qb,
+                                           "frac_of_hbm": qb / q["decode_us"] / 1e3 / peak, "kernels": kinds},
+                                "prefill": {"tokens": P, "ms": q["prefill_ms"], "tokens_per_s": P / q["prefill_ms"] * 1e3},
+                                "kernels_alone": {k: alone[k] for k in ("attention_rows", "attention_rows_prep", "gateup_product_bf16")}}
+        rows.append(res)
+    clocks = sampler.stop()
+    r0 = rows[0]
+    emit(json.dumps({
+        "metric": "decode_tokens_per_s", "value": r0["decode"]["tokens_per_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": r0["decode"]["us_per_token"] * (G - 1) / 1e3, "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
+        "dtype": "bf16 matrices and products, f32 accumulate, norms, scores, recurrence and residual streams", "data": "synthetic",
+        "config": {"workload": f"Zidepel decoder, one linear-attention to three attention layers: prompt portion of {P} tokens in one pass, "
+                               f"{G - 1} decode steps, sizes in 'sizes'",
+                   "prompt_len": P, "gen_len": G, "parallelism": "tp1", "l2": "inputs larger than L2 (all weights streamed per token); kernels alone: L2 flushed"},
+        "e2e": {"value": r0["decode_e2e_tokens_per_s"], "unit": "tok/s", "h2d_bytes_per_step": int(P * 4 + 8), "d2h_bytes_per_step": int(G * 4)},
+        "gpu_launches": int(launches),
+        "roofline": {"bound": "hbm", "kernel": "one token, all kernels", "achieved": r0["decode"]["bytes_per_token"] / r0["decode"]["us_per_token"] / 1e3,
+                     "peak": peak, "unit": "GB/s", "frac": r0["decode"]["frac_of_hbm"], "peak_source": peak_kind, "traffic": None},
+        "clocks": clocks, "sizes": rows}))
+    return 0
+
+
 LATENT_WORKLOADS = {
     # name: sizes of (width, layers, heads, dim, rot_dim, vdim, kv_rank, ff, vocab, window), each beside a Qwen3 model of the same
     # width, layers, heads x 128, feed-forward and vocabulary; prompt portion, generated tokens
@@ -465,6 +665,12 @@ def write_latent_model(folder, z, seed):
             "mix.uk": (H * z["dim"], R), "mix.uv": (H * z["vdim"], R), "mix.g": (H * z["vdim"], D), "mix.o": (D, H * z["vdim"]),
             "mlp.gate": (F, D), "mlp.up": (F, D), "mlp.down": (D, F), "rg1": (D, D), "rg1.b": (D,), "rg2": (D, D), "rg2.b": (D,),
             "dwa": (i + 2,)}.items()})
+    return write_random_tensors(folder, shapes, seed, lambda k: "ones" if "norm" in k else "depth" if k.endswith("dwa") else None)
+
+
+def write_random_tensors(folder, shapes, seed, special):
+    """model.safetensors: matrices N(0, 0.02) cut from one random block; special(name): "ones", "zeros", "identity", "depth" (0.1, the
+    last 1) or None."""
     header, at = {}, 0
     for k, v in shapes.items():
         n = 2 * int(np.prod(v))
@@ -476,15 +682,13 @@ def write_latent_model(folder, z, seed):
     with open(os.path.join(folder, "model.safetensors"), "wb") as f:
         f.write(len(text).to_bytes(8, "little") + text)
         for k, v in shapes.items():
-            n = int(np.prod(v))
-            if k.endswith("dwa"):
-                w = np.full(n, 0.1, dtype=np.float32)
-                w[-1] = 1.0
-            elif "norm" in k:
-                w = np.ones(n, dtype=np.float32)
-            else:
-                w = None
-            if w is not None:
+            n, kind = int(np.prod(v)), special(k)
+            if kind:
+                w = np.ones(n, dtype=np.float32) if kind == "ones" else np.zeros(n, dtype=np.float32)
+                if kind == "identity":
+                    w = np.eye(v[0], dtype=np.float32).ravel()
+                if kind == "depth":
+                    w[:], w[-1] = 0.1, 1.0
                 f.write((w.view(np.uint32) >> 16).astype("<u2").tobytes())
                 continue
             o = int(rng.integers(0, block.size))
@@ -493,6 +697,84 @@ def write_latent_model(folder, z, seed):
                 f.write(block[o:o + m].tobytes())
                 n, o = n - m, 0
     return folder
+
+
+def timed_flushed(torch, fn, reps=10):
+    """Median milliseconds of fn, L2 flushed before every run."""
+    for _ in range(3):
+        fn()
+    flush = torch.empty(1 << 28, dtype=torch.uint8, device="cuda")
+    ms = []
+    for _ in range(reps):
+        flush.zero_()                                        # larger than L2
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        fn()
+        e1.record()
+        e1.synchronize()
+        ms.append(e0.elapsed_time(e1))
+    return statistics.median(ms)
+
+
+FOLDER_KINDS = ["in", "attention", "o", "gateup", "down", "lm_head"]
+
+
+def open_folder_model(pkg, write, max_tokens):
+    folder = tempfile.mkdtemp(prefix="model-")
+    try:
+        write(folder)
+        return pkg.DirModel(folder, max_tokens, "bfloat16")
+    finally:
+        shutil.rmtree(folder)
+
+
+def measure_folder_model(pkg, L, S, m, P, G, warmup, steps):
+    """Prompt portion of P tokens, G - 1 decode steps timed on the device, and the same through inference_generate."""
+    prompt = np.zeros(P, dtype=np.uint32)
+    S.llmb200_synth_tokens(prompt.ctypes.data, P, 4321, m.vocab)
+    pp = prompt.ctypes.data_as(pkg.c_u32_p)
+    L.llmb200_state_set_eos(m.state, None, 0)
+    out = np.zeros(G, dtype=np.uint32)
+    op = out.ctypes.data_as(pkg.c_u32_p)
+    prefill, decode, e2e, launches = [], [], [], 0
+    graph = L.llmb200_state_graph_kernels(m.state, 1)
+    for it in range(warmup + steps):
+        m.reset()
+        L.metal_flush()
+        t0 = time.perf_counter()
+        if L.inference_forward_tokens(m.state, pp, P, None, 0, None) != 0:
+            raise RuntimeError("prompt portion failed")
+        t1 = time.perf_counter()
+        ms = L.llmb200_state_run_device_steps(m.state, G - 1)
+        if ms <= 0:
+            raise RuntimeError("device steps failed")
+        n = L.inference_generate(m.state, pp, P, op, G)
+        nd = C.c_int(0)
+        dms = L.llmb200_last_decode_ms(m.state, C.byref(nd))
+        if n != G:
+            raise RuntimeError("generate failed")
+        if it >= warmup:
+            prefill.append((t1 - t0) * 1e3)
+            decode.append(ms)
+            e2e.append(dms)
+            launches += graph * (G - 1)
+    return {"prefill_ms": statistics.median(prefill), "decode_us": 1e3 * statistics.median(decode) / (G - 1),
+            "e2e_tokens_per_s": (G - 1) / statistics.median(e2e) * 1e3, "launches": launches, "graph": graph, "prompt": prompt}
+
+
+def time_folder_kinds(L, m, prompt, kbytes, peak, launches_of=lambda k: 1):
+    """Every kind of decode kernel alone: microseconds (of all its launches of a layer), bytes and fraction of HBM."""
+    m.reset()
+    m.feed(prompt.tolist())
+    kinds = {}
+    for k, name in enumerate(FOLDER_KINDS):
+        if name not in kbytes:
+            continue
+        cnt = C.c_int(0)
+        ms = L.llmb200_state_time_kind(m.state, k, 8 if k < 5 else 24, C.byref(cnt))
+        us = 1e3 * ms / cnt.value * launches_of(name)
+        kinds[name] = {"us": us, "bytes": kbytes[name], "gbs": kbytes[name] / us / 1e3, "frac_of_hbm": kbytes[name] / us / 1e3 / peak}
+    return kinds
 
 
 def latent_kernel_timings(pkg, L, torch, z, M, peaks):
@@ -504,19 +786,7 @@ def latent_kernel_timings(pkg, L, torch, z, M, peaks):
     out = {}
 
     def timed(fn, reps=10):
-        for _ in range(3):
-            fn()
-        flush = torch.empty(1 << 28, dtype=torch.uint8, device="cuda")
-        ms = []
-        for _ in range(reps):
-            flush.zero_()                                        # larger than L2
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            fn()
-            e1.record()
-            e1.synchronize()
-            ms.append(e0.elapsed_time(e1))
-        return statistics.median(ms)
+        return timed_flushed(torch, fn, reps)
 
     st = torch.cuda.current_stream().cuda_stream
     for name, fn, dt in (("gateup_product_bf16", L.b200_gemm_bf16, torch.bfloat16), ("gateup_product_f16_closest_model", L.b200_gemm_f16, torch.float16)):
@@ -576,6 +846,17 @@ def latent_kernel_timings(pkg, L, torch, z, M, peaks):
     return out
 
 
+def latent_in_rows(z):
+    return z["heads"] * (z["dim"] + z["rot_dim"]) + z["kv_rank"] + z["rot_dim"] + z["heads"] * z["vdim"] + z["width"]
+
+
+def latent_kernel_bytes(z, P):
+    """Bytes that one layer's decode kernels have to move at position P."""
+    D, H, cs, W = z["width"], z["heads"], z["kv_rank"] + z["rot_dim"], min(z["window"], P)
+    return {"in": 2 * latent_in_rows(z) * D, "attention": 2 * (H * z["kv_rank"] * (z["dim"] + z["vdim"]) + W * cs), "o": 2 * D * H * z["vdim"],
+            "gateup": 2 * (2 * z["ff"] + D) * D, "down": 2 * D * z["ff"], "lm_head": 2 * z["vocab"] * D}
+
+
 def latent_main(args, rank, local_rank, world):
     """Morilorn: prompt portions and decode at several sizes, each beside a Qwen3 (binary16) model of equal width, depth, heads,
     feed-forward and vocabulary on this library. The line's value is the first size's decode rate."""
@@ -583,8 +864,6 @@ def latent_main(args, rank, local_rank, world):
         if rank == 0:
             emit(json.dumps({"impl": args.impl, "unavailable": "the reference has no such model; the workload runs on one GPU"}))
         return 0
-    import shutil
-    import tempfile
     import torch
     torch.cuda.set_device(local_rank)
     sizes, P, G = LATENT_WORKLOADS[args.workload]
@@ -598,68 +877,28 @@ def latent_main(args, rank, local_rank, world):
     except Exception:
         tc = 1590.0
     threads = max(1, min(32, os.cpu_count() or 8))
-    kinds = ["in", "attention", "o", "gateup", "down", "lm_head"]
+    kinds = FOLDER_KINDS
     rows, launches = [], 0
     sampler = ClockSampler(local_rank)
     for zi, z in enumerate(sizes):
         z = dict(z, layers=args.layers or z["layers"])
-        folder = tempfile.mkdtemp(prefix="morilorn-")
-        try:
-            write_latent_model(folder, z, 7 + zi)
-            m = pkg.DirModel(folder, P + G + 8, "bfloat16")
-        finally:
-            shutil.rmtree(folder)
+        m = open_folder_model(pkg, lambda folder: write_latent_model(folder, z, 7 + zi), P + G + 8)
         D, nl, H, V = z["width"], z["layers"], z["heads"], z["vocab"]
-        prompt = np.zeros(P, dtype=np.uint32)
-        S.llmb200_synth_tokens(prompt.ctypes.data, P, 4321, V)
-        pp = prompt.ctypes.data_as(pkg.c_u32_p)
-        L.llmb200_state_set_eos(m.state, None, 0)
-        out = np.zeros(G, dtype=np.uint32)
-        op = out.ctypes.data_as(pkg.c_u32_p)
         if zi == 0:
             sampler.start()
-        prefill, decode, e2e = [], [], []
-        graph = L.llmb200_state_graph_kernels(m.state, 1)
-        for it in range(args.warmup + args.steps):
-            m.reset()
-            L.metal_flush()
-            t0 = time.perf_counter()
-            if L.inference_forward_tokens(m.state, pp, P, None, 0, None) != 0:
-                raise RuntimeError("prompt portion failed")
-            t1 = time.perf_counter()
-            ms = L.llmb200_state_run_device_steps(m.state, G - 1)
-            if ms <= 0:
-                raise RuntimeError("device steps failed")
-            n = L.inference_generate(m.state, pp, P, op, G)
-            nd = C.c_int(0)
-            dms = L.llmb200_last_decode_ms(m.state, C.byref(nd))
-            if n != G:
-                raise RuntimeError("generate failed")
-            if it >= args.warmup:
-                prefill.append((t1 - t0) * 1e3); decode.append(ms); e2e.append(dms)
-                launches += graph * (G - 1)
-        per_kind = {}
-        m.reset()
-        m.feed(prompt.tolist())
-        for k, name in enumerate(kinds):
-            cnt = C.c_int(0)
-            ms = L.llmb200_state_time_kind(m.state, k, 8 if k < 5 else 24, C.byref(cnt))
-            per_layer = 3 if name == "attention" else 1
-            per_kind[name] = {"us": 1e3 * ms / cnt.value * per_layer}
-        up8 = lambda v: (v + 7) // 8 * 8
-        in_rows = H * (z["dim"] + z["rot_dim"]) + z["kv_rank"] + z["rot_dim"] + H * z["vdim"] + D
-        cs, W = z["kv_rank"] + z["rot_dim"], min(z["window"], P)
-        kbytes = {"in": 2 * in_rows * D, "attention": 2 * (H * z["kv_rank"] * (z["dim"] + z["vdim"]) + W * cs), "o": 2 * D * H * z["vdim"],
-                  "gateup": 2 * (2 * z["ff"] + D) * D, "down": 2 * D * z["ff"], "lm_head": 2 * V * D}
-        for name, b in kbytes.items():
-            per_kind[name].update(bytes=b, gbs=b / per_kind[name]["us"] / 1e3, frac_of_hbm=b / per_kind[name]["us"] / 1e3 / peak)
+        r = measure_folder_model(pkg, L, S, m, P, G, args.warmup, args.steps)
+        prompt, pp, graph = r["prompt"], r["prompt"].ctypes.data_as(pkg.c_u32_p), r["graph"]
+        launches += r["launches"]
+        op = np.zeros(G, dtype=np.uint32).ctypes.data_as(pkg.c_u32_p)
+        in_rows = latent_in_rows(z)
+        kbytes = latent_kernel_bytes(z, P)
+        per_kind = time_folder_kinds(L, m, prompt, kbytes, peak, lambda k: 3 if k == "attention" else 1)
         token_bytes = sum(b * (nl if k != "lm_head" else 1) for k, b in kbytes.items())
-        us = 1e3 * statistics.median(decode) / (G - 1)
-        pf = statistics.median(prefill)
+        us, pf = r["decode_us"], r["prefill_ms"]
         row_flops = 2.0 * P * nl * (in_rows * D + H * z["kv_rank"] * (z["dim"] + z["vdim"]) + D * H * z["vdim"] + (3 * z["ff"] + D) * D)
         res = {"sizes": z, "decode": {"tokens_per_s": 1e6 / us, "us_per_token": us, "bytes_per_token": token_bytes,
                                       "frac_of_hbm": token_bytes / us / 1e3 / peak, "kernels": per_kind, "launches_per_token": graph},
-               "decode_e2e_tokens_per_s": (G - 1) / statistics.median(e2e) * 1e3,
+               "decode_e2e_tokens_per_s": r["e2e_tokens_per_s"],
                "prefill": {"tokens": P, "ms": pf, "tokens_per_s": P / pf * 1e3, "product_tflops": row_flops / pf / 1e9,
                            "frac_of_tensor_peak": row_flops / pf / 1e9 / tc}}
         if L.llmb200_state_error(m.state):
@@ -1039,7 +1278,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="qwen3-4b-q8",
-                    choices=sorted(WORKLOADS) + sorted(SFT_WORKLOADS) + sorted(BATCH_WORKLOADS) + sorted(LATENT_WORKLOADS) + ["matvec-sweep"])
+                    choices=sorted(WORKLOADS) + sorted(SFT_WORKLOADS) + sorted(BATCH_WORKLOADS) + sorted(LATENT_WORKLOADS) + sorted(HYBRID_WORKLOADS) + ["matvec-sweep"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-secondary", action="store_true", help="skip the secondary configurations and the parity stamp")
     ap.add_argument("--prompt-len", type=int, default=0, help="override the workload's prompt length (profiling runs)")
@@ -1054,6 +1293,8 @@ def main():
         return sft_main(args, rank, local_rank, world)
     if args.workload in BATCH_WORKLOADS:
         return batch_main(args, rank, local_rank, world)
+    if args.workload in HYBRID_WORKLOADS:
+        return hybrid_main(args, rank, local_rank, world)
     if args.workload in LATENT_WORKLOADS:
         return latent_main(args, rank, local_rank, world)
     if args.workload == "matvec-sweep":

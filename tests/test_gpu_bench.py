@@ -1,7 +1,7 @@
 """The benchmark's contract on its small workloads: exactly one JSON line on stdout with the agreed keys.
 
 Every workload family runs once (decode Q8_0, Gemma3 binary16 decode, LoRA SFT step, batched binary16
-decode, latent-attention decode) so that a change that breaks a family's timing path or its reporting shows up as a test failure.
+decode, latent-attention decode, attention and recurrence over streams) so that a change that breaks a family's timing path or its reporting shows up as a test failure.
 """
 import json
 import os
@@ -32,6 +32,7 @@ def run_bench(*extra):
     ("tiny-qwen3-sft-lora", "sft_tokens_per_s"),
     ("tiny-qwen3-f16-batch8", "batched_decode_tokens_per_s"),
     ("tiny-morilorn", "decode_tokens_per_s"),
+    ("tiny-zidepel", "decode_tokens_per_s"),
 ])
 def test_one_json_line_with_the_contract_keys(workload, metric):
     d = run_bench("--workload", workload)
