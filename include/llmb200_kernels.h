@@ -314,7 +314,7 @@ typedef struct b200_gqa_args {
     void *d_out_rows; long long out_ld;  /* [n_rows] rows of heads * vdim, out_ld elements apart */
 } b200_gqa_args;
 
-/* Splits of the sequence worth launching for this shape (1 .. 256). */
+/* Clusters of blocks that share the sequence for this shape (1 .. 64). */
 int b200_gqa_splits(int wtype, int heads, int kv_heads, int dim, int vdim, int max_seq);
 int b200_gqa_decode(const b200_gqa_args *a, void *stream);
 int b200_gqa_rows_prep(const b200_gqa_args *a, void *stream);

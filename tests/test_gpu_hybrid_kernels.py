@@ -313,18 +313,17 @@ def test_attention_options(lib, pkg, wtype, cap, temp):
 
 
 @pytest.mark.parametrize("wtype", TYPES)
-def test_attention_over_many_splits(lib, pkg, wtype):
-    """Positions around every border of the decode kernel's shares of a long sequence; a far key per share."""
-    n = 2400
-    far = [(i, (i * 37) % (i - 1)) for i in (2111, 2112, 2113, 2303, 2304, 2305, 2399)]
-    t = Attn(lib, pkg, wtype, 4, 2, 64, 32, n, 28.0, {"coef": 0.25, "every": 300}, 13, far=far)
-    assert t.splits > 20
+def test_attention_over_clusters_of_blocks(lib, pkg, wtype):
+    """Positions around every border of the decode kernel's shares of a long sequence (a block's, a cluster's), a far key each."""
+    n, lone = 4200, [2047, 2048, 2049, 2050, 2303, 2304, 3000, 4095, 4096, 4097, 4098, 4199]
+    t = Attn(lib, pkg, wtype, 2, 2, 64, 32, n, 28.0, {"coef": 0.25, "every": 300}, 13, far=[(i, (i * 37) % (i - 1)) for i in lone])
+    assert t.splits == 2
     got = t.rows(0, n)
     tol = 2e-2 if wtype == BF16 else 3e-5
     close(got, t.want, tol, t.size)
-    for i in (0, 1, 62, 63, 64, 65, 127, 128, 129, 1000, 2111, 2112, 2113, 2303, 2304, 2305, 2398, 2399):
+    for i in [0, 1, 7, 8, 9, 15, 16, 17, 62, 63, 64, 65, 127, 128, 129, 511, 512, 513, 1000] + lone:
         close(t.one(i)[None], t.want[i:i + 1], tol, t.size)
-    one = [t.one(2399) for _ in range(3)]
+    one = [t.one(4199) for _ in range(3)]
     assert np.array_equal(one[0], one[1]) and np.array_equal(one[0], one[2])
 
 
