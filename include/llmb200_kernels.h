@@ -331,7 +331,7 @@ int b200_gqa_rows_attend(const b200_gqa_args *a, void *stream);
  * [n_slots][heads][dim][up8(vdim)] (padding zero) and the one after it goes to the next slot, so running a position again gives the
  * same result, as with a key cache. Before position 0 the state is zero, whatever the slot holds.
  * Decode (b200_gla_decode, one launch): the token at *d_pos. Rows (b200_gla_rows): n_rows tokens from position
- * pos0 on, cut into chunks of 64 that are summed in parallel and joined by a scan over their states.
+ * pos0 on, cut into chunks of 64: their scores in parallel, then the states chunk by chunk, then all outputs.
  * ---------------------------------------------------------------------- */
 #define B200_GLA_CHUNK 64
 typedef struct b200_gla_args {
@@ -348,10 +348,10 @@ typedef struct b200_gla_args {
     /* rows; n_chunks = (n_rows + 63) / 64 */
     int n_rows, pos0;
     long long proj_ld;
-    float *d_qd, *d_kd;                  /* [n_chunks * 64][heads][up8(dim)]: queries and keys times their decays */
-    float *d_decay;                      /* [n_chunks][heads][up8(dim)]: logarithm of the decay over a whole chunk */
-    float *d_scores;                     /* [n_chunks][heads][64][64] */
-    float *d_chunk_state;                /* [n_chunks][heads][dim][up8(vdim)] */
+    float *d_qd, *d_kd;                  /* [n_chunks][heads]: queries [up8(dim)][64], keys [64][up8(dim)], times their decays */
+    float *d_decay;                      /* [n_chunks][heads][up8(dim)]: log2 of the decay over a whole chunk */
+    float *d_scores;                     /* [n_chunks][heads][64][64], by key, then query */
+    float *d_chunk_state;                /* [n_chunks][heads][dim][up8(vdim)]: the state before each chunk */
     float *d_o;                          /* [n_rows][heads * vdim]; vdim > 128 only */
     void *d_out_rows; long long out_ld;  /* [n_rows] rows of heads * vdim, out_ld elements apart */
 } b200_gla_args;

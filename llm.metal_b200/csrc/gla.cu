@@ -8,9 +8,10 @@
 // Prompt portions: chunks of 64 tokens in parallel. With c_t the running sum of the log decays inside a chunk,
 //   o_t = (q_t exp(c_t)) S_in + sum over s <= t of (sum over channels q_t k_s exp(c_t - c_s)) v_s
 //   S_out = exp(c_end) S_in + sum over s of (k_s exp(c_end - c_s)) v_s^T
-// gla_prep forms the decayed queries and keys and the score matrix, gla_chunk_state every chunk's own sum,
-// gla_scan joins the chunks, gla_out forms the outputs. Every exponent that is taken is <= 0: inside sixteen tokens the
-// differences c_t - c_s are exponentiated pair by pair, across sixteens through the value of c between the two.
+// gla_prep forms the decayed queries and keys and the score matrix, gla_states walks the chunks with a tile of the state
+// in registers and leaves the state before each, gla_out forms the outputs. Every exponent that is taken is <= 0: inside
+// eight tokens the differences c_t - c_s are exponentiated pair by pair, across eights and sixteens as a product through
+// the value of c between the two.
 #include "stream_core.cuh"
 #include "../../include/llmb200_kernels.h"
 
@@ -161,25 +162,51 @@ __global__ void __launch_bounds__(THREADS) gla_decode_kernel(const __grid_consta
 // ------------------------------------------------------------------------------------------------ rows
 
 constexpr int DT = 32, RS = DT + 4;                          // channels of a pass; row of a tile: 16 bytes off a multiple of 32
+constexpr int EIGHT_PAIRS = 36, N_PAIRS = C / 8 * EIGHT_PAIRS;       // s <= t inside eight tokens; of a chunk
 
-// One block per chunk and head. Shared: f [C][R4], then [C][RS] each: c (running log decay), q, k, q from the start of
-// its sixteen; and k up to the starts of the second, third and fourth sixteen, [16 + 32 + 48][RS].
+// The pair (t, s) number e of a chunk's eights.
+__device__ __forceinline__ void pair_of(int e, int &t, int &s)
+{
+    const int base = e / EIGHT_PAIRS * 8;
+    int k = e % EIGHT_PAIRS, row = 0;
+    while (k > row) { k -= row + 1; ++row; }
+    t = base + row;
+    s = base + k;
+}
+__device__ __forceinline__ float score4(const float4 &q, const float4 &k, const float4 &ct, const float4 &cs, float acc)
+{
+    const float4 w = make_float4(exp2f(ct.x - cs.x), exp2f(ct.y - cs.y), exp2f(ct.z - cs.z), exp2f(ct.w - cs.w));
+    return dot4(make_float4(q.x * k.x, q.y * k.y, q.z * k.z, q.w * k.w), w, acc);
+}
+__device__ __forceinline__ float4 row4(const float *tile, int row, int col) { return *reinterpret_cast<const float4 *>(tile + row * RS + col); }
+
+// One block per chunk and head. Shared: f [C][R4], then tiles of rows RS apart: c (running log2 of the decay), q, k [C];
+// q from the start of its sixteen [C]; k up to the starts of the second, third and fourth sixteen [16 + 32 + 48]; q of the
+// second eights and k of the first eights through the boundary between them [32] each.
 __global__ void __launch_bounds__(THREADS) gla_prep_kernel(const __grid_constant__ b200_gla_args p)
 {
     extern __shared__ __align__(16) float sh[];
     __shared__ float tot[8][DT];
     const int R4 = up4(p.rank), d8 = up8(p.dim), tid = threadIdx.x;
-    float *fs = sh, *cs = fs + C * R4, *qs = cs + C * RS, *ks = qs + C * RS, *qh = ks + C * RS, *kh = qh + C * RS, *ws = kh + 96 * RS;
+    float *fs = sh, *cs = fs + C * R4, *qs = cs + C * RS, *ks = qs + C * RS, *qh = ks + C * RS, *kh = qh + C * RS;
+    float *q8 = kh + 96 * RS, *k8 = q8 + C / 2 * RS, *ws = k8 + C / 2 * RS;
     const int chunk = blockIdx.x, h = blockIdx.y, m0 = chunk * C, n = min(C, p.n_rows - m0);
+    const size_t ch = (size_t)chunk * p.heads + h;
     const int w16 = (R4 / 4) | 1;
     for (int e = tid; e < C * R4; e += THREADS) {
         const int t = e / R4, r = e % R4;
         fs[e] = t < n && r < p.rank ? p.d_f[(size_t)(m0 + t) * p.proj_ld + r] : 0.0f;
     }
-    const int ti = tid / SUB, si = tid % SUB;
-    float acc[10];                                           // (i, j) of the lower triangle of sixteens, j <= i
+    // this thread's scores: one of every pair of sixteens i > j, one across the eights of a sixteen, one or two pairs of an eight
+    const int ti = tid % SUB, si = tid / SUB;
+    const int et = tid % 8, es = tid / 8 % 8, eb = tid / 64;
+    int pt[2], ps[2];
+    pair_of(tid, pt[0], ps[0]);
+    pair_of(min(THREADS + tid, N_PAIRS - 1), pt[1], ps[1]);
+    const bool two = THREADS + tid < N_PAIRS;
+    float far[6], mid = 0.0f, near[2] = {0.0f, 0.0f};
 #pragma unroll
-    for (int x = 0; x < 10; ++x) acc[x] = 0.0f;
+    for (int x = 0; x < 6; ++x) far[x] = 0.0f;
 
     for (int d0 = 0; d0 < p.dim; d0 += DT) {
         __syncthreads();
@@ -210,9 +237,10 @@ __global__ void __launch_bounds__(THREADS) gla_prep_kernel(const __grid_constant
             for (int i = 0; i < 8; ++i) c[i] = dot4(w, *reinterpret_cast<const float4 *>(fs + (tg * 8 + i) * R4 + 4 * r), c[i]);
         }
         float run = 0.0f;
+        const float unit = 1.4426950408889634f / p.tau;
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-            if (on && tg * 8 + i < n) run += log_logistic(c[i]) / p.tau;
+            if (on && tg * 8 + i < n) run += log_logistic(c[i]) * unit;
             c[i] = run;
         }
         tot[tg][d] = run;
@@ -225,56 +253,105 @@ __global__ void __launch_bounds__(THREADS) gla_prep_kernel(const __grid_constant
             const int t = tg * 8 + i;
             c[i] += before;
             cs[t * RS + d] = c[i]; qs[t * RS + d] = q[i]; ks[t * RS + d] = k[i];
-            if (d0 + d < d8) {
-                const size_t at = ((size_t)m0 + t) * p.heads * d8 + (size_t)h * d8 + d0 + d;
-                p.d_qd[at] = q[i] * expf(c[i]);
-                p.d_kd[at] = k[i] * expf(end - c[i]);
-            }
+            if (d0 + d < d8) p.d_kd[((ch * C) + t) * d8 + d0 + d] = k[i] * exp2f(end - c[i]);
         }
-        if (tg == 0 && d0 + d < d8) p.d_decay[((size_t)chunk * p.heads + h) * d8 + d0 + d] = end;
+        if (d0 + d < d8) {
+            float *out = p.d_qd + (ch * d8 + d0 + d) * C + tg * 8;
+#pragma unroll
+            for (int i = 0; i < 8; i += 4)
+                *reinterpret_cast<float4 *>(out + i) = make_float4(q[i] * exp2f(c[i]), q[i + 1] * exp2f(c[i + 1]), q[i + 2] * exp2f(c[i + 2]), q[i + 3] * exp2f(c[i + 3]));
+            if (tg == 0) p.d_decay[ch * d8 + d0 + d] = end;
+        }
         __syncthreads();
-        // references: c just before each sixteen
+        {   // through the boundaries: c just before each sixteen, c at the end of each first eight (this thread's tokens are one eight)
+            const int u = tg / 2;
+            const float start = u > 0 ? cs[(u * SUB - 1) * RS + d] : 0.0f, half = cs[(u * SUB + 7) * RS + d];
+            float next[3];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int t = tg * 8 + i, u = t / SUB;
-            if (u > 0) qh[t * RS + d] = q[i] * expf(c[i] - cs[(u * SUB - 1) * RS + d]);
+            for (int v = 1; v < 4; ++v) next[v - 1] = cs[(v * SUB - 1) * RS + d];
 #pragma unroll
-            for (int v = 1; v < 4; ++v)
-                if (u < v) kh[(v * (v - 1) * SUB / 2 + t) * RS + d] = k[i] * expf(cs[(v * SUB - 1) * RS + d] - c[i]);
+            for (int i = 0; i < 8; ++i) {
+                const int t = tg * 8 + i;
+                if (u > 0) qh[t * RS + d] = q[i] * exp2f(c[i] - start);
+                if (tg & 1) q8[(u * 8 + i) * RS + d] = q[i] * exp2f(c[i] - half);
+                else k8[(u * 8 + i) * RS + d] = k[i] * exp2f(half - c[i]);
+#pragma unroll
+                for (int v = 1; v < 4; ++v)
+                    if (u < v) kh[(v * (v - 1) * SUB / 2 + t) * RS + d] = k[i] * exp2f(next[v - 1] - c[i]);
+            }
         }
         __syncthreads();
 #pragma unroll 2
         for (int x = 0; x < DT; x += 4) {
 #pragma unroll
-            for (int i = 0, at = 0; i < 4; ++i) {
-                if (i > 0) {
-                    const float4 a = *reinterpret_cast<const float4 *>(qh + (i * SUB + ti) * RS + x);
+            for (int i = 1, at = 0; i < 4; ++i) {
+                const float4 a = row4(qh, i * SUB + ti, x);
 #pragma unroll
-                    for (int j = 0; j < i; ++j, ++at)
-                        acc[at] = dot4(a, *reinterpret_cast<const float4 *>(kh + (i * (i - 1) * SUB / 2 + j * SUB + si) * RS + x), acc[at]);
-                }
-                const float4 a = *reinterpret_cast<const float4 *>(qs + (i * SUB + ti) * RS + x), b = *reinterpret_cast<const float4 *>(ks + (i * SUB + si) * RS + x);
-                const float4 e = *reinterpret_cast<const float4 *>(cs + (i * SUB + ti) * RS + x), f = *reinterpret_cast<const float4 *>(cs + (i * SUB + si) * RS + x);
-                if (si <= ti) {
-                    const float4 w = make_float4(__expf(e.x - f.x), __expf(e.y - f.y), __expf(e.z - f.z), __expf(e.w - f.w));
-                    acc[at] = dot4(make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w), w, acc[at]);
-                }
-                ++at;
+                for (int j = 0; j < i; ++j, ++at) far[at] = dot4(a, row4(kh, i * (i - 1) * SUB / 2 + j * SUB + si, x), far[at]);
             }
+            mid = dot4(row4(q8, eb * 8 + et, x), row4(k8, eb * 8 + es, x), mid);
+            near[0] = score4(row4(qs, pt[0], x), row4(ks, ps[0], x), row4(cs, pt[0], x), row4(cs, ps[0], x), near[0]);
+            if (two) near[1] = score4(row4(qs, pt[1], x), row4(ks, ps[1], x), row4(cs, pt[1], x), row4(cs, ps[1], x), near[1]);
         }
     }
-    float *out = p.d_scores + ((size_t)chunk * p.heads + h) * C * C;
+    // [s][t], zeros where s > t
+    float *out = p.d_scores + ch * C * C;
 #pragma unroll
     for (int i = 0, at = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j <= i; ++j, ++at) out[(i * SUB + ti) * C + j * SUB + si] = acc[at];
+        for (int j = 0; j < 4; ++j) {
+            if (i > j) out[(j * SUB + si) * C + i * SUB + ti] = far[at++];
+            else if (i < j) out[(j * SUB + si) * C + i * SUB + ti] = 0.0f;
+        }
+    out[(eb * SUB + es) * C + eb * SUB + 8 + et] = mid;
+    out[(eb * SUB + 8 + es) * C + eb * SUB + et] = 0.0f;
+    out[ps[0] * C + pt[0]] = near[0];
+    if (pt[0] != ps[0]) out[pt[0] * C + ps[0]] = 0.0f;
+    if (two) {
+        out[ps[1] * C + pt[1]] = near[1];
+        if (pt[1] != ps[1]) out[pt[1] * C + ps[1]] = 0.0f;
+    }
 }
 
-// Tile product: acc[4][4 * TN] += A[k][m] B[k][n] over kn rows of shared tiles, thread (ty, tx): rows 4 ty.., columns 4 tx + 64 g..
+__device__ __forceinline__ void cp16_if(float *dst, const float *src, bool on)
+{
+    const int n = on ? 16 : 0;                               // 0: zero-filled
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void cp4_if(float *dst, const float *src, bool on)
+{
+    const int n = on ? 4 : 0;
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// Rows t0 .. t0 + ROWS of a chunk's values, columns j0 .. j0 + W of head h, to dst [ROWS][ld]. vec: 16-byte pieces are aligned.
+template <int ROWS, int W, int NT>
+__device__ __forceinline__ void fetch_values(const b200_gla_args &p, float *dst, int ld, int m0, int t0, int n, int h, int j0, bool vec)
+{
+    const float *src = p.d_v + (size_t)(m0 + t0) * p.proj_ld + (size_t)h * p.vdim + j0;
+    if (vec) {
+#pragma unroll 4
+        for (int e = threadIdx.x; e < ROWS * W / 4; e += NT) {
+            const int t = e / (W / 4), j = e % (W / 4) * 4;
+            const bool on = t0 + t < n && j0 + j < p.vdim;
+            cp16_if(dst + t * ld + j, on ? src + (size_t)t * p.proj_ld + j : p.d_v, on);
+        }
+    } else {
+        for (int e = threadIdx.x; e < ROWS * W; e += NT) {
+            const int t = e / W, j = e % W;
+            const bool on = t0 + t < n && j0 + j < p.vdim;
+            cp4_if(dst + t * ld + j, on ? src + (size_t)t * p.proj_ld + j : p.d_v, on);
+        }
+    }
+}
+
+// acc[4][4 * TN] += A[k][m] B[k][n] over kn rows of shared tiles, thread (ty, tx): rows 4 ty.., columns 4 tx + 64 g..
 template <int TN>
 __device__ __forceinline__ void tile_product(const float *A, int lda, const float *B, int ldb, int kn, int ty, int tx, float (&acc)[4][4 * TN])
 {
-#pragma unroll 4
+#pragma unroll 8
     for (int k = 0; k < kn; ++k) {
         const float4 a4 = *reinterpret_cast<const float4 *>(A + k * lda + 4 * ty);
         const float a[4] = {a4.x, a4.y, a4.z, a4.w};
@@ -290,115 +367,110 @@ __device__ __forceinline__ void tile_product(const float *A, int lda, const floa
     }
 }
 
-// A chunk's own sum: 64 channels x 64 TN columns per block.
-template <int TN>
-__global__ void __launch_bounds__(THREADS) gla_chunk_state_kernel(const __grid_constant__ b200_gla_args p, int vtiles)
+// The states before every chunk and after the last: a block walks the chunks with 32 channels x 64 columns of one head's
+// state in registers, the operands of the next chunks in flight.
+constexpr int SD = 32, SV = 64, S_THREADS = 128, S_STAGES = 4, S_TILE = C * SD + C * SV;
+__global__ void __launch_bounds__(S_THREADS) gla_states_kernel(const __grid_constant__ b200_gla_args p, int n_chunks, int vec)
 {
-    __shared__ __align__(16) float ks[C][64 + 4], vs[C / 2][64 * TN + 4];
-    const int chunk = blockIdx.x, h = blockIdx.y, d0 = blockIdx.z / vtiles * 64, j0 = blockIdx.z % vtiles * 64 * TN;
-    const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16, d8 = up8(p.dim), v8 = up8(p.vdim), m0 = chunk * C, n = min(C, p.n_rows - m0);
-    for (int e = tid; e < C * 16; e += THREADS) {
-        const int t = e / 16, d = e % 16 * 4;
-        *reinterpret_cast<float4 *>(&ks[t][d]) = d0 + d < d8 ? *reinterpret_cast<const float4 *>(p.d_kd + ((size_t)m0 + t) * p.heads * d8 + (size_t)h * d8 + d0 + d)
-                                                            : make_float4(0, 0, 0, 0);
-    }
-    float acc[4][4 * TN];
+    extern __shared__ __align__(16) float sh[];              // [S_STAGES] x { keys [C][SD], values [C][SV] }
+    const int h = blockIdx.z, d0 = blockIdx.x * SD, j0 = blockIdx.y * SV, tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
+    const int d8 = up8(p.dim), v8 = up8(p.vdim), j = j0 + 4 * tx;
+    const size_t slot = (size_t)p.heads * p.dim * v8;
+    auto fetch = [&](int chunk) {
+        float *kt = sh + (size_t)(chunk % S_STAGES) * S_TILE, *vt = kt + C * SD;
+        const float *src = p.d_kd + ((size_t)chunk * p.heads + h) * C * d8 + d0;
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int j = 0; j < 4 * TN; ++j) acc[i][j] = 0.0f;
-    for (int t0 = 0; t0 < C; t0 += C / 2) {
-        __syncthreads();
-        for (int e = tid; e < C / 2 * 64 * TN; e += THREADS) {
-            const int t = e / (64 * TN), j = e % (64 * TN);
-            vs[t][j] = t0 + t < n && j0 + j < p.vdim ? p.d_v[(size_t)(m0 + t0 + t) * p.proj_ld + (size_t)h * p.vdim + j0 + j] : 0.0f;
+        for (int e = tid; e < C * SD / 4; e += S_THREADS) {
+            const int t = e / (SD / 4), d = e % (SD / 4) * 4;
+            cp16_if(kt + t * SD + d, d0 + d < d8 ? src + (size_t)t * d8 + d : p.d_kd, d0 + d < d8);
         }
-        __syncthreads();
-        tile_product<TN>(&ks[t0][0], 64 + 4, &vs[0][0], 64 * TN + 4, C / 2, ty, tx, acc);
+        fetch_values<C, SV, S_THREADS>(p, vt, SV, chunk * C, 0, min(C, p.n_rows - chunk * C), h, j0, vec);
+    };
+    for (int c = 0; c < S_STAGES - 1; ++c) {
+        if (c < n_chunks) fetch(c);
+        cp_commit();
     }
-    float *out = p.d_chunk_state + ((size_t)chunk * p.heads + h) * p.dim * v8;
+    float s[4][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 4; ++i) {
+        const int d = d0 + 4 * ty + i;
+        float4 v = make_float4(0, 0, 0, 0);
+        if (p.pos0 > 0 && d < p.dim && j < v8)
+            v = *reinterpret_cast<const float4 *>(p.d_state + (size_t)(p.pos0 % p.n_slots) * slot + ((size_t)h * p.dim + d) * v8 + j);
+        s[i][0] = v.x; s[i][1] = v.y; s[i][2] = v.z; s[i][3] = v.w;
+    }
+    auto store = [&](float *base) {
 #pragma unroll
-        for (int g = 0; g < TN; ++g) {
-            const int d = d0 + 4 * ty + i, j = j0 + 64 * g + 4 * tx;
-            if (d < p.dim && j < v8)
-                *reinterpret_cast<float4 *>(out + (size_t)d * v8 + j) = make_float4(acc[i][4 * g], acc[i][4 * g + 1], acc[i][4 * g + 2], acc[i][4 * g + 3]);
+        for (int i = 0; i < 4; ++i) {
+            const int d = d0 + 4 * ty + i;
+            if (d < p.dim && j < v8) *reinterpret_cast<float4 *>(base + ((size_t)h * p.dim + d) * v8 + j) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
         }
-}
-
-// Replaces every chunk's own sum by the state before it; the state after the last one goes to its slot. A thread: one quad.
-__global__ void __launch_bounds__(THREADS) gla_scan_kernel(const __grid_constant__ b200_gla_args p, int n_chunks)
-{
-    constexpr int AHEAD = 8;
-    const int v8 = up8(p.vdim), d8 = up8(p.dim), quads = v8 / 4;
-    const size_t e = (size_t)blockIdx.x * THREADS + threadIdx.x, total = (size_t)p.heads * p.dim * quads, per = total * 4;
-    if (e >= total) return;
-    const size_t row = e / quads;                            // head * dim + channel
-    const size_t ch = row / p.dim * d8 + row % p.dim;
-    float4 s = make_float4(0, 0, 0, 0);
-    if (p.pos0 > 0) s = *reinterpret_cast<const float4 *>(p.d_state + (size_t)(p.pos0 % p.n_slots) * per + e * 4);
-    for (int c0 = 0; c0 < n_chunks; c0 += AHEAD) {
-        float4 u[AHEAD];
-        Decay g[AHEAD];
+    };
+    for (int c = 0; c < n_chunks; ++c) {
+        store(p.d_chunk_state + (size_t)c * slot);
+        const float4 g4 = d0 + 4 * ty < d8 ? *reinterpret_cast<const float4 *>(p.d_decay + ((size_t)c * p.heads + h) * d8 + d0 + 4 * ty) : make_float4(0, 0, 0, 0);
+        cp_wait<S_STAGES - 2>();
+        __syncthreads();                                     // this chunk's tiles are there; everybody is done with the previous one's
+        if (c + S_STAGES - 1 < n_chunks) fetch(c + S_STAGES - 1);
+        cp_commit();
+        const float *kt = sh + (size_t)(c % S_STAGES) * S_TILE, *vt = kt + C * SD;
+        float u[4][4] = {};
+        tile_product<1>(kt, SD, vt, SV, C, ty, tx, u);
+        const float g[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
-        for (int i = 0; i < AHEAD; ++i)
-            if (c0 + i < n_chunks) {
-                u[i] = *reinterpret_cast<const float4 *>(p.d_chunk_state + (size_t)(c0 + i) * per + e * 4);
-                g[i] = decay_of(p.d_decay[(size_t)(c0 + i) * p.heads * d8 + ch]);
-            }
+        for (int i = 0; i < 4; ++i) {
+            const Decay a = decay_of(g[i] * 0.6931471805599453f);
 #pragma unroll
-        for (int i = 0; i < AHEAD; ++i)
-            if (c0 + i < n_chunks) {
-                *reinterpret_cast<float4 *>(p.d_chunk_state + (size_t)(c0 + i) * per + e * 4) = s;
-                s.x = decayed(s.x, g[i], u[i].x); s.y = decayed(s.y, g[i], u[i].y); s.z = decayed(s.z, g[i], u[i].z); s.w = decayed(s.w, g[i], u[i].w);
-            }
+            for (int k = 0; k < 4; ++k) s[i][k] = decayed(s[i][k], a, u[i][k]);
+        }
     }
-    *reinterpret_cast<float4 *>(p.d_state + (size_t)((p.pos0 + p.n_rows) % p.n_slots) * per + e * 4) = s;
+    store(p.d_state + (size_t)((p.pos0 + p.n_rows) % p.n_slots) * slot);
 }
 
 // Outputs of a chunk, 64 tokens x 64 TN columns per block: decayed queries times the state before the chunk, scores times
-// values. FUSED: the columns are the whole head, so the norm and the gate follow here.
+// values, 32 rows of the contraction at a time. FUSED: the columns are the whole head, so the norm and the gate follow here.
+constexpr int KB = 32, O_STAGES = 3;
 template <int TN, bool FUSED, typename T>
-__global__ void __launch_bounds__(THREADS) gla_out_kernel(const __grid_constant__ b200_gla_args p)
+__global__ void __launch_bounds__(THREADS) gla_out_kernel(const __grid_constant__ b200_gla_args p, int vec)
 {
-    constexpr int KB = 32, BW = 64 * TN + 4;
-    __shared__ __align__(16) float as[KB][C + 4], bs[KB][BW];
-    const int chunk = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 64 * TN;
+    constexpr int BW = 64 * TN, TILE = KB * C + KB * BW;
+    extern __shared__ __align__(16) float sh[];              // [O_STAGES] x { A [KB][C], B [KB][BW] }
+    const int chunk = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * BW;
     const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16, d8 = up8(p.dim), v8 = up8(p.vdim), m0 = chunk * C, n = min(C, p.n_rows - m0);
-    const float *S = p.d_chunk_state + ((size_t)chunk * p.heads + h) * p.dim * v8;
-    const float *A = p.d_scores + ((size_t)chunk * p.heads + h) * C * C;
-    float acc[4][4 * TN];
+    const size_t ch = (size_t)chunk * p.heads + h;
+    const float *S = p.d_chunk_state + ch * p.dim * v8, *Q = p.d_qd + ch * d8 * C, *A = p.d_scores + ch * C * C;
+    const int steps_s = chunk == 0 && p.pos0 == 0 ? 0 : (p.dim + KB - 1) / KB, steps = steps_s + C / KB;
+    auto fetch = [&](int i) {
+        float *at = sh + (size_t)(i % O_STAGES) * TILE, *bt = at + KB * C;
+        const bool state = i < steps_s;
+        const int k0 = state ? i * KB : (i - steps_s) * KB, kn = state ? d8 : C;
+        const float *src = state ? Q : A;
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+        for (int e = tid; e < KB * C / 4; e += THREADS) {
+            const int k = e / (C / 4), t = e % (C / 4) * 4;
+            cp16_if(at + k * C + t, k0 + k < kn ? src + (size_t)(k0 + k) * C + t : src, k0 + k < kn);
+        }
+        if (!state) fetch_values<KB, BW, THREADS>(p, bt, BW, m0, k0, n, h, j0, vec);
+        else
 #pragma unroll
-        for (int j = 0; j < 4 * TN; ++j) acc[i][j] = 0.0f;
-    for (int k0 = 0; k0 < p.dim; k0 += KB) {
-        __syncthreads();
-        for (int e = tid; e < C * KB; e += THREADS) {        // lanes over channels: coalesced; rows of `as` 4 banks apart
-            const int t = e / KB, k = e % KB;
-            as[k][t] = k0 + k < d8 ? p.d_qd[((size_t)m0 + t) * p.heads * d8 + (size_t)h * d8 + k0 + k] : 0.0f;
-        }
-        for (int e = tid; e < KB * 16 * TN; e += THREADS) {
-            const int k = e / (16 * TN), j = e % (16 * TN) * 4;
-            *reinterpret_cast<float4 *>(&bs[k][j]) = k0 + k < p.dim && j0 + j < v8 ? *reinterpret_cast<const float4 *>(S + (size_t)(k0 + k) * v8 + j0 + j)
-                                                                                  : make_float4(0, 0, 0, 0);
-        }
-        __syncthreads();
-        tile_product<TN>(&as[0][0], C + 4, &bs[0][0], BW, KB, ty, tx, acc);
+            for (int e = tid; e < KB * BW / 4; e += THREADS) {
+                const int k = e / (BW / 4), j = e % (BW / 4) * 4;
+                const bool on = k0 + k < p.dim && j0 + j < v8;
+                cp16_if(bt + k * BW + j, on ? S + (size_t)(k0 + k) * v8 + j0 + j : S, on);
+            }
+    };
+    for (int i = 0; i < O_STAGES - 1; ++i) {
+        if (i < steps) fetch(i);
+        cp_commit();
     }
-    for (int k0 = 0; k0 < C; k0 += KB) {
+    float acc[4][4 * TN] = {};
+    for (int i = 0; i < steps; ++i) {
+        cp_wait<O_STAGES - 2>();
         __syncthreads();
-        for (int e = tid; e < C * KB; e += THREADS) {
-            const int t = e / KB, k = e % KB;
-            as[k][t] = (k0 + k) / SUB <= t / SUB ? A[t * C + k0 + k] : 0.0f;       // sixteens above the diagonal are not stored
-        }
-        for (int e = tid; e < KB * 64 * TN; e += THREADS) {
-            const int k = e / (64 * TN), j = e % (64 * TN);
-            bs[k][j] = k0 + k < n && j0 + j < p.vdim ? p.d_v[(size_t)(m0 + k0 + k) * p.proj_ld + (size_t)h * p.vdim + j0 + j] : 0.0f;
-        }
-        __syncthreads();
-        tile_product<TN>(&as[0][0], C + 4, &bs[0][0], BW, KB, ty, tx, acc);
+        if (i + O_STAGES - 1 < steps) fetch(i + O_STAGES - 1);
+        cp_commit();
+        const float *at = sh + (size_t)(i % O_STAGES) * TILE;
+        tile_product<TN>(at, C, at + KB * C, BW, KB, ty, tx, acc);
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -460,16 +532,20 @@ int allow_smem(K kern, size_t smem)
 }
 
 template <int TN, typename T>
-int out_rows(const b200_gla_args &a, int n_chunks, cudaStream_t st)
+int out_rows(const b200_gla_args &a, int n_chunks, int vec, cudaStream_t st)
 {
     const int tiles = (a.vdim + 64 * TN - 1) / (64 * TN);
+    const size_t smem = (size_t)O_STAGES * (KB * C + KB * 64 * TN) * 4;
     const dim3 grid(n_chunks, a.heads, tiles);
+    int rc;
     if (tiles == 1) {
-        gla_out_kernel<TN, true, T><<<grid, THREADS, 0, st>>>(a);
+        if ((rc = allow_smem(gla_out_kernel<TN, true, T>, smem)) != 0) return rc;
+        gla_out_kernel<TN, true, T><<<grid, THREADS, smem, st>>>(a, vec);
         ++g_b200_launches;
         return (int)cudaGetLastError();
     }
-    gla_out_kernel<TN, false, T><<<grid, THREADS, 0, st>>>(a);
+    if ((rc = allow_smem(gla_out_kernel<TN, false, T>, smem)) != 0) return rc;
+    gla_out_kernel<TN, false, T><<<grid, THREADS, smem, st>>>(a, vec);
     const size_t warps = (size_t)a.n_rows * a.heads;
     gla_gate_kernel<T><<<(unsigned)((warps + 7) / 8), THREADS, 0, st>>>(a);
     g_b200_launches += 2;
@@ -516,21 +592,16 @@ extern "C" int b200_gla_rows(const b200_gla_args *ap, void *stream)
         return B200_E_BADARG;
     const b200_gla_args &a = *ap;
     cudaStream_t st = (cudaStream_t)stream;
-    const int n_chunks = (a.n_rows + C - 1) / C, R4 = up4(a.rank), v8 = up8(a.vdim);
-    const size_t smem = ((size_t)C * R4 + (size_t)(4 * C + 96) * RS + (size_t)DT * ((R4 / 4) | 1) * 4) * 4;
-    int rc = allow_smem(gla_prep_kernel, smem);
+    const int n_chunks = (a.n_rows + C - 1) / C, R4 = up4(a.rank);
+    const int vec = a.vdim % 4 == 0 && a.proj_ld % 4 == 0 && ((uintptr_t)a.d_v & 15) == 0;
+    const size_t prep = ((size_t)C * R4 + (size_t)(5 * C + 96) * RS + (size_t)DT * ((R4 / 4) | 1) * 4) * 4, states = (size_t)S_STAGES * S_TILE * 4;
+    int rc = allow_smem(gla_prep_kernel, prep);
+    if (!rc) rc = allow_smem(gla_states_kernel, states);
     if (rc) return rc;
-    gla_prep_kernel<<<dim3(n_chunks, a.heads), THREADS, smem, st>>>(a);
-    const int dtiles = (a.dim + 63) / 64;
-    if (a.vdim <= 64) gla_chunk_state_kernel<1><<<dim3(n_chunks, a.heads, dtiles), THREADS, 0, st>>>(a, 1);
-    else {
-        const int vt = (a.vdim + 127) / 128;
-        gla_chunk_state_kernel<2><<<dim3(n_chunks, a.heads, dtiles * vt), THREADS, 0, st>>>(a, vt);
-    }
-    const size_t quads = (size_t)a.heads * a.dim * (v8 / 4);
-    gla_scan_kernel<<<(unsigned)((quads + THREADS - 1) / THREADS), THREADS, 0, st>>>(a, n_chunks);
-    g_b200_launches += 3;
+    gla_prep_kernel<<<dim3(n_chunks, a.heads), THREADS, prep, st>>>(a);
+    gla_states_kernel<<<dim3((a.dim + SD - 1) / SD, (a.vdim + SV - 1) / SV, a.heads), S_THREADS, states, st>>>(a, n_chunks, vec);
+    g_b200_launches += 2;
     if ((rc = (int)cudaGetLastError()) != 0) return rc;
-    if (a.wtype == B200_WT_BF16) return a.vdim <= 64 ? out_rows<1, __nv_bfloat16>(a, n_chunks, st) : out_rows<2, __nv_bfloat16>(a, n_chunks, st);
-    return a.vdim <= 64 ? out_rows<1, float>(a, n_chunks, st) : out_rows<2, float>(a, n_chunks, st);
+    if (a.wtype == B200_WT_BF16) return a.vdim <= 64 ? out_rows<1, __nv_bfloat16>(a, n_chunks, vec, st) : out_rows<2, __nv_bfloat16>(a, n_chunks, vec, st);
+    return a.vdim <= 64 ? out_rows<1, float>(a, n_chunks, vec, st) : out_rows<2, float>(a, n_chunks, vec, st);
 }

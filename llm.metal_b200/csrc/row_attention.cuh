@@ -155,8 +155,17 @@ __device__ __forceinline__ float soft_cap(float s, float two_log2e_over_cap, flo
 {
     return cap - __fdividef(2.0f * cap, ex2(s * two_log2e_over_cap) + 1.0f);
 }
+// Later rows see more keys. Blocks are numbered from the heaviest tile of rows to the lightest; where two of them share
+// an SM and all are resident at once, the second half counts from the light end, so that every SM gets about the same.
+struct Place { int tile, head; };
+__device__ __forceinline__ Place place_of(int id, int n, int heads, int wave)
+{
+    const int r = id < wave || n > 2 * wave ? id : n - 1 - (id - wave);
+    return {n / heads - 1 - r / heads, r % heads};
+}
+
 template <int DV, int NW, bool CAP>
-__global__ void __launch_bounds__(NW * 32, 16 / NW) row_attend_bf16_kernel(const __grid_constant__ RowAttn p, int dqs, int stages)
+__global__ void __launch_bounds__(NW * 32, 16 / NW) row_attend_bf16_kernel(const __grid_constant__ RowAttn p, int dqs, int stages, int wave)
 {
     // dqs: elements of a query / key row in shared memory; its first dqs - 8 are multiples of 16 and hold
     // [unrotated | rotated | zeros]. Rows are 16 bytes off a multiple of 32: ldmatrix is conflict-free.
@@ -168,7 +177,8 @@ __global__ void __launch_bounds__(NW * 32, 16 / NW) row_attend_bf16_kernel(const
     __nv_bfloat16 *ksm = qsm + (size_t)BQ * dqs;             // [stages][BKEY][dqs]
     __nv_bfloat16 *vsm = ksm + (size_t)stages * BKEY * dqs;  // [stages][BKEY][VS]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int h = blockIdx.y, m0 = blockIdx.x * BQ, c0 = blockIdx.z * DV;
+    const Place place = place_of(blockIdx.x, gridDim.x, p.heads, wave);
+    const int h = place.head, m0 = place.tile * BQ, c0 = blockIdx.y * DV;
     const int rows = min(BQ, p.n_rows - m0);
     const __nv_bfloat16 *keys = static_cast<const __nv_bfloat16 *>(p.k) + (h / p.group) * p.k_head;
     const __nv_bfloat16 *values = static_cast<const __nv_bfloat16 *>(p.v) + (h / p.group) * p.v_head;
@@ -353,8 +363,8 @@ int row_attend_bf16(const RowAttn &a, cudaStream_t st)
     if (bytes(2) > 227 * 1024) stages = 1;
     int rc = allow_smem(row_attend_bf16_kernel<DV, NW, CAP>, bytes(stages));
     if (rc) return rc;
-    const dim3 grid((a.n_rows + NW * 16 - 1) / (NW * 16), a.heads, (a.vdim + DV - 1) / DV);
-    row_attend_bf16_kernel<DV, NW, CAP><<<grid, NW * 32, bytes(stages), st>>>(a, dqs, stages);
+    const dim3 grid((a.n_rows + NW * 16 - 1) / (NW * 16) * a.heads, (a.vdim + DV - 1) / DV);
+    row_attend_bf16_kernel<DV, NW, CAP><<<grid, NW * 32, bytes(stages), st>>>(a, dqs, stages, 148);
     ++g_b200_launches;
     return (int)cudaGetLastError();
 }
