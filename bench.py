@@ -535,8 +535,10 @@ def hybrid_kernel_timings(pkg, L, torch, z, M, peaks):
     g.proj_ld = ld
     g.d_k, g.d_v, g.d_gate, g.d_f = (g.d_q + 4 * o for o in (H * d, 2 * H * d, 2 * H * d + H * dv, 2 * H * d + 2 * H * dv))
     g.d_a2, g.d_a2_bias, g.d_norm_gamma, g.d_state = buf(H * d, r4), buf(H * d), buf(dv), buf(2, H, d, up8(dv))
-    g.d_qd, g.d_kd, g.d_decay, g.d_scores = buf(nc * 64, H, up8(d)), buf(nc * 64, H, up8(d)), buf(nc, H, up8(d)), buf(nc, H, 64, 64)
-    g.d_chunk_state, g.d_o, g.d_out_rows, g.out_ld, g.n_rows = buf(nc, H, d, up8(dv)), buf(M, H * dv), buf(M, H * dv, dt=torch.bfloat16), H * dv, M
+    planes = lambda *shape: buf(nc, H, 3, *shape, dt=torch.bfloat16)
+    g.d_qd, g.d_kd, g.d_values, g.d_scores = planes(64, (d + 15) // 16 * 16), planes(64, (d + 15) // 16 * 16), planes(64, up8(dv)), planes(64, 64)
+    g.d_chunk_state, g.d_decay, g.d_o = planes(d, up8(dv)), buf(nc, H, up8(d)), buf(M, H * dv)
+    g.d_out_rows, g.out_ld, g.n_rows = buf(M, H * dv, dt=torch.bfloat16), H * dv, M
     run("linear_attention_rows", L.b200_gla_rows, g, nbytes=M * (4.0 * ld + 2.0 * H * dv))
     s = pkg.RowsStreamsArgs()
     s.streams_in, s.streams_in_stride, s.y, s.y_ld, s.connect, s.n_streams = buf(n, M, D), M * D, buf(M, D), D, buf(n * (n + 2)), n

@@ -348,11 +348,13 @@ typedef struct b200_gla_args {
     /* rows; n_chunks = (n_rows + 63) / 64 */
     int n_rows, pos0;
     long long proj_ld;
-    float *d_qd, *d_kd;                  /* [n_chunks][heads]: queries [up8(dim)][64], keys [64][up8(dim)], times their decays */
-    float *d_decay;                      /* [n_chunks][heads][up8(dim)]: log2 of the decay over a whole chunk */
-    float *d_scores;                     /* [n_chunks][heads][64][64], by key, then query */
-    float *d_chunk_state;                /* [n_chunks][heads][dim][up8(vdim)]: the state before each chunk */
-    float *d_o;                          /* [n_rows][heads * vdim]; vdim > 128 only */
+    /* scratch: three bfloat16 planes (a value as a sum of three) where nothing else is said, 16-byte aligned */
+    void *d_qd, *d_kd;                   /* [n_chunks][heads][3][64][up16(dim)]: queries and keys times their decays */
+    void *d_values;                      /* [n_chunks][heads][3][64][up8(vdim)] */
+    void *d_scores;                      /* [n_chunks][heads][3][64][64] */
+    void *d_chunk_state;                 /* [n_chunks][heads][3][dim][up8(vdim)]: the state before each chunk */
+    float *d_decay;                      /* fp32 [n_chunks][heads][up8(dim)]: log2 of the decay over a whole chunk */
+    float *d_o;                          /* fp32 [n_rows][heads * vdim]; vdim > 128 only */
     void *d_out_rows; long long out_ld;  /* [n_rows] rows of heads * vdim, out_ld elements apart */
 } b200_gla_args;
 int b200_gla_decode(const b200_gla_args *a, void *stream);

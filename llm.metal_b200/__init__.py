@@ -180,7 +180,7 @@ class GlaArgs(C.Structure):
                [(n, C.c_float) for n in ("tau", "q_scale", "eps")] + \
                [(n, C.c_void_p) for n in ("d_q", "d_k", "d_v", "d_gate", "d_f", "d_a2", "d_a2_bias", "d_norm_gamma", "d_state", "d_out", "d_pos")] + \
                [(n, C.c_int) for n in ("use_pdl", "n_rows", "pos0")] + [("proj_ld", C.c_longlong)] + \
-               [(n, C.c_void_p) for n in ("d_qd", "d_kd", "d_decay", "d_scores", "d_chunk_state", "d_o", "d_out_rows")] + [("out_ld", C.c_longlong)]
+               [(n, C.c_void_p) for n in ("d_qd", "d_kd", "d_values", "d_scores", "d_chunk_state", "d_decay", "d_o", "d_out_rows")] + [("out_ld", C.c_longlong)]
 
 
 class RowsStreamsArgs(C.Structure):

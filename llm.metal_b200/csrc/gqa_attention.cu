@@ -589,7 +589,7 @@ __global__ void __launch_bounds__(THREADS) gqa_prep_kernel(const __grid_constant
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
             const int e = lane + 32 * k;
-            held[k] = e < n ? x[e] : 0.0f;
+            held[k] = e < n ? __ldg(x + e) : 0.0f;
             ss = fmaf(held[k], held[k], ss);
         }
         for (int e = lane + 256; e < n; e += 32) ss = fmaf(x[e], x[e], ss);
@@ -605,7 +605,7 @@ __global__ void __launch_bounds__(THREADS) gqa_prep_kernel(const __grid_constant
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
             const int e = lane + 32 * k;
-            if (e < n8) out[e] = (T)(e < n ? gamma[e] * (held[k] * inv) : 0.0f);
+            if (e < n8) out[e] = (T)(e < n ? __ldg(gamma + e) * (held[k] * inv) : 0.0f);
         }
         for (int e = lane + 256; e < n8; e += 32) out[e] = (T)(e < n ? gamma[e] * (x[e] * inv) : 0.0f);
     }

@@ -72,8 +72,8 @@ typedef struct {
     unsigned *tickets;
     /* rows (allocated at the first portion) */
     RowPath rows;
-    float *r_proj, *r_x0, *r_streams[2], *r_u, *r_y, *r_qd, *r_kd, *r_decay, *r_scores, *r_chunk, *r_o;
-    void *r_h, *r_q, *r_attn, *r_act;
+    float *r_proj, *r_x0, *r_streams[2], *r_u, *r_y, *r_decay, *r_o;
+    void *r_h, *r_q, *r_attn, *r_act, *r_qd, *r_kd, *r_values, *r_scores, *r_chunk;
 } Hybrid;
 
 static size_t smax(size_t a, size_t b) { return a > b ? a : b; }
@@ -340,7 +340,7 @@ static void free_model(InferenceState *s)
     for (int i = 0; i < m->n_tables; ++i) cudaFree(m->tables[i]);
     void *b[] = { m->head.w, m->pos, m->emb_w, m->emb_b, m->final_b, m->first_take, m->proj, m->attn, m->act, m->part, m->tickets, m->x0,
                   m->streams[0], m->streams[1], m->u, m->r_proj, m->r_x0, m->r_streams[0], m->r_streams[1], m->r_u, m->r_y, m->r_qd, m->r_kd,
-                  m->r_decay, m->r_scores, m->r_chunk, m->r_o, m->r_h, m->r_q, m->r_attn, m->r_act };
+                  m->r_decay, m->r_values, m->r_scores, m->r_chunk, m->r_o, m->r_h, m->r_q, m->r_attn, m->r_act };
     for (size_t k = 0; k < sizeof(b) / sizeof(b[0]); ++k) cudaFree(b[k]);
     llmb200_row_path_free(&m->rows);
     free(m->layers);
@@ -475,7 +475,7 @@ static int rows_ready(InferenceState *s, Hybrid *m)
 {
     if (m->rows.chunk) return 0;
     const size_t M = llmb200_row_chunk(s), Dp = m->Dp, n = m->n_streams, es = m->es, nc = (M + CHUNK - 1) / CHUNK;
-    size_t proj = 0, q = 0, attn = 0, act = 0, qd = 0, scores = 0, chunk = 0, o = 0;
+    size_t proj = 0, q = 0, attn = 0, act = 0, qd = 0, values = 0, decay = 0, scores = 0, chunk = 0, o = 0;
     for (int i = 0; i < m->n_layers; ++i) {
         const HLayer *y = &m->layers[i];
         const size_t wide = (size_t)y->heads * up8(y->dim);
@@ -484,9 +484,11 @@ static int rows_ready(InferenceState *s, Hybrid *m)
         act = smax(act, y->up.rows);
         if (y->mixer == MIX_ATTENTION) q = smax(q, wide);
         else {
-            qd = smax(qd, wide);
-            scores = smax(scores, (size_t)y->heads * CHUNK * CHUNK);
-            chunk = smax(chunk, (size_t)y->heads * y->dim * up8(y->vdim));
+            decay = smax(decay, wide);
+            qd = smax(qd, (size_t)3 * CHUNK * y->heads * ((y->dim + 15) & ~15));
+            values = smax(values, (size_t)3 * CHUNK * y->heads * up8(y->vdim));
+            scores = smax(scores, (size_t)3 * y->heads * CHUNK * CHUNK);
+            chunk = smax(chunk, (size_t)3 * y->heads * y->dim * up8(y->vdim));
             if (y->vdim > 128) o = smax(o, (size_t)y->heads * y->vdim);
         }
     }
@@ -494,10 +496,11 @@ static int rows_ready(InferenceState *s, Hybrid *m)
     for (int i = 0; i < 2; ++i) m->r_streams[i] = llmb200_dev_zero(n * M * Dp * 4);
     m->r_y = llmb200_dev_zero(M * smax(64, Dp) * 4); m->r_h = llmb200_dev_zero(M * Dp * es);
     m->r_q = llmb200_dev_zero(M * q * es); m->r_attn = llmb200_dev_zero(M * attn * es); m->r_act = llmb200_dev_zero(M * act * es);
-    m->r_qd = llmb200_dev_zero(nc * CHUNK * qd * 4); m->r_kd = llmb200_dev_zero(nc * CHUNK * qd * 4); m->r_decay = llmb200_dev_zero(nc * qd * 4);
-    m->r_scores = llmb200_dev_zero(nc * scores * 4); m->r_chunk = llmb200_dev_zero(nc * chunk * 4); m->r_o = llmb200_dev_zero(M * o * 4);
+    m->r_qd = llmb200_dev_zero(nc * qd * 2); m->r_kd = llmb200_dev_zero(nc * qd * 2); m->r_values = llmb200_dev_zero(nc * values * 2);
+    m->r_scores = llmb200_dev_zero(nc * scores * 2); m->r_chunk = llmb200_dev_zero(nc * chunk * 2); m->r_decay = llmb200_dev_zero(nc * decay * 4);
+    m->r_o = llmb200_dev_zero(M * o * 4);
     if (!m->r_proj || !m->r_x0 || !m->r_u || !m->r_streams[0] || !m->r_streams[1] || !m->r_y || !m->r_h || !m->r_q || !m->r_attn || !m->r_act ||
-        !m->r_qd || !m->r_kd || !m->r_decay || !m->r_scores || !m->r_chunk || !m->r_o)
+        !m->r_qd || !m->r_kd || !m->r_values || !m->r_decay || !m->r_scores || !m->r_chunk || !m->r_o)
         return -1;
     return llmb200_row_path_ready(s, &m->rows, &m->head, m->Dp, (int)M);
 }
@@ -516,7 +519,7 @@ static int mix_rows(InferenceState *s, Hybrid *m, const HLayer *y, const Run *ru
     b200_gla_args at;
     gla_args(s, m, y, run, m->r_proj, &at);
     at.n_rows = M; at.pos0 = pos0; at.proj_ld = y->in.rows;
-    at.d_qd = m->r_qd; at.d_kd = m->r_kd; at.d_decay = m->r_decay; at.d_scores = m->r_scores; at.d_chunk_state = m->r_chunk; at.d_o = m->r_o;
+    at.d_qd = m->r_qd; at.d_kd = m->r_kd; at.d_values = m->r_values; at.d_decay = m->r_decay; at.d_scores = m->r_scores; at.d_chunk_state = m->r_chunk; at.d_o = m->r_o;
     at.d_out_rows = m->r_attn; at.out_ld = y->o.cols;
     K_TRY(b200_gla_rows(&at, g_rt.stream), return -1);
     return 0;

@@ -221,11 +221,27 @@ def test_squared_relu_of_row_products(lib, pkg, M, N, K):
 
 # ------------------------------------------------------------------ attention
 
+_soil = None
+
+
+def soil(lib, pkg):
+    """Leaves NaN in the shared memory of every SM: a kernel that reads what it has not written shows it."""
+    global _soil
+    if _soil is None:
+        w = torch.full((2368, 3072), float("nan"), device="cuda")
+        a = pkg.MatvecArgs()
+        keep = [w, zeros(3072), zeros(2368)]
+        a.d_w, a.row_stride, a.rows, a.cols, a.wtype, a.n_out, a.d_in_vec = w.data_ptr(), 3072 * 4, 2368, 3072, F32, 1, keep[1].data_ptr()
+        a.d_out[0] = keep[2].data_ptr()
+        _soil = (a, keep)
+    assert lib.b200_matvec(C.byref(_soil[0]), None) == 0
+
+
 class Attn:
     """Projections of n tokens, and a kernel state that has not seen any of them. Cache rows not written yet hold NaN."""
 
     def __init__(self, lib, pkg, wtype, H, G, d, dv, n, cap, temp, seed, max_seq=None, far=None, eps=1e-3):
-        self.lib, self.wtype, self.n, self.H, self.G, self.d, self.dv = lib, wtype, n, H, G, d, dv
+        self.lib, self.pkg, self.wtype, self.n, self.H, self.G, self.d, self.dv = lib, pkg, wtype, n, H, G, d, dv
         g, self.scale, self.cap, self.max_seq = rng(seed), 0.9 * d ** -0.5, cap, max_seq or n
         q, k, v = g.standard_normal((n, H, d)), g.standard_normal((n, G, d)), g.standard_normal((n, G, dv))
         if far:                                                       # (query position, key position): that key outweighs the rest
@@ -264,6 +280,7 @@ class Attn:
         out = zeros(m, H * dv + 5, dtype=ttype(self.wtype))
         a.n_rows, a.pos0, a.proj_ld, a.d_q_rows, a.d_out_rows, a.out_ld = m, pos0, self.ld, q.data_ptr(), out.data_ptr(), H * dv + 5
         assert self.lib.b200_gqa_rows_prep(C.byref(a), None) == 0
+        soil(self.lib, self.pkg)
         assert self.lib.b200_gqa_rows_attend(C.byref(a), None) == 0
         got = host(out)
         assert not got[:, H * dv:].any()
@@ -273,6 +290,7 @@ class Attn:
         self.at(pos)
         self.pos.fill_(pos)
         self.out.fill_(float("nan"))
+        soil(self.lib, self.pkg)
         assert self.lib.b200_gqa_decode(C.byref(self.a), None) == 0
         got = host(self.out).reshape(self.H, self.dv)
         assert not host(self.tickets).any()
@@ -348,7 +366,7 @@ def test_attention_ignores_positions_outside_the_cache(lib, pkg):
 class Gla:
     def __init__(self, lib, pkg, H, d, dv, rank, tau, n, seed, slots=3, bias=(2.0, 2.0), wtype=F32, eps=1e-4):
         g = rng(seed)
-        self.lib, self.H, self.dv, self.n, self.wtype, self.slots, self.d = lib, H, dv, n, wtype, slots, d
+        self.lib, self.pkg, self.H, self.dv, self.n, self.wtype, self.slots, self.d = lib, pkg, H, dv, n, wtype, slots, d
         q, k, v, gate, f = (g.standard_normal((n, s)) for s in (H * d, H * d, H * dv, H * dv, rank))
         a2, b, gamma = g.standard_normal((H * d, rank)) * rank ** -0.5, bias[0] + bias[1] * g.standard_normal(H * d), 1 + 0.3 * g.standard_normal(dv)
         a = o.decay(f @ a2.T + b, tau).reshape(n, H, d)
@@ -366,12 +384,14 @@ class Gla:
         self.keep = [dev(padded(a2, R4)), dev(b), dev(gamma)]
         nan = lambda *s: torch.full(s, float("nan"), device="cuda")
         self.st, self.out, self.pos = nan(slots, H, d, up8(dv)), zeros(H * dv), zeros(1, dtype=torch.int32)
-        self.scratch = [nan(nc * 64, H, up8(d)), nan(nc * 64, H, up8(d)), nan(nc, H, up8(d)), nan(nc, H, 64, 64), nan(nc, H, d, up8(dv)), nan(n, H * dv)]
+        planes = lambda *s: nan(nc, H, 3, *s).bfloat16()
+        d16 = (d + 15) // 16 * 16
+        self.scratch = [planes(64, d16), planes(64, d16), planes(64, up8(dv)), planes(64, 64), planes(d, up8(dv)), nan(nc, H, up8(d)), nan(n, H * dv)]
         p = self.p = pkg.GlaArgs()
         p.wtype, p.heads, p.dim, p.vdim, p.rank, p.n_slots, p.tau, p.q_scale, p.eps = wtype, H, d, dv, rank, slots, tau, d ** -0.5, eps
         p.d_a2, p.d_a2_bias, p.d_norm_gamma = (t.data_ptr() for t in self.keep)
         p.d_state, p.d_out, p.d_pos = self.st.data_ptr(), self.out.data_ptr(), self.pos.data_ptr()
-        p.d_qd, p.d_kd, p.d_decay, p.d_scores, p.d_chunk_state, p.d_o = (t.data_ptr() for t in self.scratch)
+        p.d_qd, p.d_kd, p.d_values, p.d_scores, p.d_chunk_state, p.d_decay, p.d_o = (t.data_ptr() for t in self.scratch)
 
     def at(self, row):
         base = self.proj.data_ptr() + 4 * row * self.ld
@@ -381,6 +401,7 @@ class Gla:
         self.at(pos0)
         out = zeros(m, self.H * self.dv + 3, dtype=ttype(self.wtype))
         self.p.n_rows, self.p.pos0, self.p.proj_ld, self.p.d_out_rows, self.p.out_ld = m, pos0, self.ld, out.data_ptr(), self.H * self.dv + 3
+        soil(self.lib, self.pkg)
         assert self.lib.b200_gla_rows(C.byref(self.p), None) == 0
         got = host(out)
         assert not got[:, self.H * self.dv:].any()
@@ -390,6 +411,7 @@ class Gla:
         self.at(pos)
         self.pos.fill_(pos)
         self.out.fill_(float("nan"))
+        soil(self.lib, self.pkg)
         assert self.lib.b200_gla_decode(C.byref(self.p), None) == 0
         return host(self.out)
 
