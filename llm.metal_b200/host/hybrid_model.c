@@ -155,8 +155,8 @@ static int parse(InferenceState *s, Hybrid *m, const json *c)
     m->loop_times = 1;
     if (loop && loop->type != JSON_NULL &&
         (json_int(loop, "start", &m->loop_start) || json_int(loop, "stop", &m->loop_stop) || json_int(loop, "times", &m->loop_times) ||
-         m->loop_start < 0 || m->loop_stop <= m->loop_start || m->loop_stop > m->n_layers || m->loop_times < 1))
-        return llmb200_bad_config("loop", "needs 0 <= start < stop <= layers and times >= 1");
+         m->loop_start < 0 || m->loop_stop < m->loop_start || m->loop_stop > m->n_layers || m->loop_times < 1))
+        return llmb200_bad_config("loop", "needs 0 <= start <= stop <= layers and times >= 1");
     if (s->max_seq > m->max_positions) s->max_seq = m->max_positions;        /* a position past the table does not exist */
     return make_runs(s, m);
 }

@@ -228,6 +228,18 @@ def test_parts_switched_off_by_their_weights(pkg, tmp_path, what):
             good(m, run(m, t, [23, 2]), want)
 
 
+@pytest.mark.parametrize("loop,same", [(None, True), ((1, 1, 3), True), ((0, 3, 1), True), ((2, 3, 2), False), ((0, 1, 3), False)])
+def test_loops_of_every_kind(pkg, tmp_path, loop, same):
+    config, ranks = o.model_config(40, 56, 2, [T.R(2, 8, 12, 24, 4.0, 3), T.A(2, 1, 8, 16, None), T.A(4, 2, 8, 8, 32)], loop=loop)
+    w = o.random_model(config, ranks, 5)
+    t = T.tokens(config, 40, 2)
+    want, _ = o.forward(config, w, t)
+    assert np.array_equal(want, o.forward(dict(config, loop=None), w, t)[0]) == same
+    with pkg.DirModel(o.write_model(str(tmp_path / "m"), config, w), 40, "float32") as m:
+        m.limit = T.LIMIT["float32"]
+        good(m, run(m, t, [25, 2]), want)
+
+
 def test_a_far_key_decides(pkg, tmp_path):
     """One attention layer whose scores rest on the tokens alone: queries of token 1 score the key of token 0 far above all
     others, and token 0 occurs once, hundreds of tokens back. In a prompt, in a later portion, and decoded alone."""
@@ -290,7 +302,7 @@ def edited(tmp_path, change=None, drop=None, reshape=None):
     lambda c: c["layers"][1]["mixer"].__setitem__("q_temp", {"coef": 1.0}), lambda c: c["layers"][1]["mixer"].pop("scale"),
     lambda c: c["layers"][0]["mixer"].pop("tau"), lambda c: c["layers"][0]["mixer"].__setitem__("dim", 0), lambda c: c.pop("streams"),
     lambda c: c.__setitem__("streams", 9), lambda c: c.__setitem__("loop", {"start": 1, "stop": 5, "times": 2}),
-    lambda c: c.__setitem__("loop", {"start": 1, "stop": 1, "times": 2}), lambda c: c.__setitem__("loop", {"start": 0, "stop": 1, "times": 0}),
+    lambda c: c.__setitem__("loop", {"start": 2, "stop": 1, "times": 2}), lambda c: c.__setitem__("loop", {"start": 0, "stop": 1, "times": 0}),
     lambda c: c["norm"].pop("eps"), lambda c: c.__setitem__("max_positions", 511)])
 def test_unusable_configurations_are_refused(lib, tmp_path, change):
     assert not lib.inference_state_create_from_dir(edited(tmp_path, change).encode(), 32, 2)
