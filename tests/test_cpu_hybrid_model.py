@@ -113,7 +113,7 @@ def test_a_planted_mistake_shows_far_above_the_limits(what, monkeypatch):
     if what == "factor step":
         mixers[1]["q_temp"]["every"] = 8
     if what == "cap":
-        mixers[3]["softcap"] = 9.5
+        mixers[3]["softcap"] = None
     if what == "gate":
         monkeypatch.setattr(o, "silu", lambda z: 1.0 / (1.0 + np.exp(-z)))
     if what == "eps":
@@ -124,7 +124,7 @@ def test_a_planted_mistake_shows_far_above_the_limits(what, monkeypatch):
     wrong, _ = o.forward(config, w, t)
     e = T.errors(wrong, right)
     assert np.median(e[45:]) > 20 * T.LIMIT["float32"], e[45:]
-    if what not in ("eps", "tau", "cap"):
+    if what not in ("eps", "tau", "cap", "factor step"):
         assert e.max() > T.LIMIT["bfloat16"], e.max()
 
 
